@@ -73,6 +73,17 @@ class TorchOps:
         if row is not None:
             h += row
 
+    def stream_join(self, h, delta, delta_scale, rows, row, *, out_dtype):
+        """[h (+ delta (* delta_scale)) | rows] in out_dtype, and a new stream that holds row (zeros without one)."""
+        if isinstance(delta, PendingProduct):
+            delta = delta.take(self)
+        x = h
+        if delta is not None:
+            d = delta.float().sum(0) if delta.dim() == 3 else delta.float()
+            x = h + (d if delta_scale is None else d * delta_scale)
+        new = torch.zeros_like(h) if row is None else row.expand_as(h).clone()
+        return torch.cat([x, rows], dim=1).to(out_dtype), new
+
     def norm_add(self, h, delta, weight, eps, out_dtype, then_weight=None, then_eps=0.0):
         """h += delta / sqrt(mean(delta^2) + eps) * weight (in place, float32); the new rows in out_dtype,
         or, with then_weight, their RMS norm under that weight."""
@@ -104,6 +115,8 @@ class TorchOps:
             return x * torch.sigmoid(x)
         if kind == "gelu_tanh":
             return 0.5 * x * (1.0 + torch.tanh(math.sqrt(2.0 / math.pi) * (x + 0.044715 * x ** 3)))
+        if kind == "gelu":
+            return 0.5 * x * (1.0 + torch.erf(x / math.sqrt(2.0)))
         raise ValueError(kind)
 
     def activation(self, x, kind, out_dtype=None):
@@ -153,6 +166,35 @@ class TorchOps:
             page, slot = sm // page_size, sm % page_size
             k_pages[page, :, slot] = turn(k, n_k_heads).to(k_pages.dtype)
             v_pages[page, :, slot] = v.reshape(T, n_v_heads, v_head_dim).to(v_pages.dtype)
+        return q.to(out_dtype).contiguous(), (torch.sigmoid(e).to(out_dtype).contiguous() if n_extra else None)
+
+    def norm_rope_store(self, proj, positions, table, *, n_q_heads, n_k_heads, head_dim, v_head_dim, rot_dims, interleaved, n_extra,
+                        k_pages, v_pages, slot_mapping, page_size, out_dtype, bias=None, values_are_keys=False, q_norm=None,
+                        k_norm=None, qk_head_norm=False, v_head_norm=False, eps=0.0):
+        """A row of proj is [q heads | k heads | v heads (unless values are keys) | extra], bias added first.  q and k each
+        RMS-normed over all their heads at once (with a weight), rotated, then every head divided by its root mean square
+        (qk_head_norm); a value is a v head or the k head as projected, divided by its root mean square (v_head_norm)."""
+        x = proj.float().sum(0) if proj.dim() == 3 else proj.float()
+        if bias is not None:
+            x = x + bias
+        T = x.shape[0]
+        nq, nk, nv = n_q_heads * head_dim, n_k_heads * head_dim, 0 if values_are_keys else n_k_heads * v_head_dim
+        q, k, v, e = x.split([nq, nk, nv, n_extra], dim=1)
+        v = (k if values_are_keys else v).reshape(T, n_k_heads, v_head_dim)
+        rms = lambda y: y * torch.rsqrt(y.pow(2).mean(-1, keepdim=True) + eps)
+        if q_norm is not None:
+            q = rms(q) * q_norm
+        if k_norm is not None:
+            k = rms(k) * k_norm
+        q = self._turn(q.reshape(T, n_q_heads, head_dim), positions, table, rot_dims, interleaved)
+        k = self._turn(k.reshape(T, n_k_heads, head_dim), positions, table, rot_dims, interleaved)
+        if qk_head_norm:
+            q, k = rms(q), rms(k)
+        if v_head_norm:
+            v = rms(v)
+        sm = slot_mapping.long()
+        k_pages[sm // page_size, :, sm % page_size] = k.to(k_pages.dtype)
+        v_pages[sm // page_size, :, sm % page_size] = v.to(v_pages.dtype)
         return q.to(out_dtype).contiguous(), (torch.sigmoid(e).to(out_dtype).contiguous() if n_extra else None)
 
     def differential_combine(self, maps, lam, *, eps, out_scale, gate, out_dtype):
@@ -460,11 +502,13 @@ class TorchOps:
             state[slot] = S
         return out.to(out_dtype)
 
-    def rmsnorm(self, h, delta, weight, eps, out_dtype, rows=None, deferred=False):
+    def rmsnorm(self, h, delta, weight, eps, out_dtype, rows=None, deferred=False, groups=1, delta_scale=None):
         if isinstance(delta, PendingProduct):
             delta = delta.take(self)
         if delta is not None and delta.dim() == 3:
             delta = delta.float().sum(0)
+        if delta is not None and delta_scale is not None:
+            delta = delta.float() * delta_scale
         x = h if delta is None else h + delta.float()
         if rows is None:
             if delta is not None:
@@ -474,7 +518,8 @@ class TorchOps:
         if deferred:
             assert rows is None
             return RowScaled((x * weight).to(out_dtype), x.pow(2).sum(-1, keepdim=True), x.shape[1], float(eps))
-        y = x * torch.rsqrt(x.pow(2).mean(-1, keepdim=True) + eps) * weight
+        parts = x.unflatten(-1, (groups, -1))
+        y = (parts * torch.rsqrt(parts.pow(2).mean(-1, keepdim=True) + eps)).flatten(-2) * weight
         return y.to(out_dtype)
 
     fuse_residual = True      # tests switch it off to compare the two ways
@@ -559,16 +604,17 @@ class TorchOps:
     def paged_attention(self, q, k_pages, v_pages, block_table, q_start, kv_len, *, n_seqs, max_q_len,
                         max_kv_len, scale, window, page_size, allow_split=True, impl="auto", n_tokens=None, out=None,
                         keep_first=0, distance_bias=None, distance_buckets=None, gate=None, n_v_heads=None,
-                        out_dtype=None, softcap=0.0, sinks=None, value_dim=None):
+                        out_dtype=None, softcap=0.0, sinks=None, value_dim=None, chunk=None, weights="softmax", score_bias=None):
         T, H, hd = q.shape
         KV = k_pages.shape[1]
         group = H // KV
         if keep_first or distance_bias is not None or gate is not None or v_pages.shape[3] != hd \
-                or v_pages.shape[1] != KV or out_dtype not in (None, q.dtype) or softcap or sinks is not None or value_dim:
+                or v_pages.shape[1] != KV or out_dtype not in (None, q.dtype) or softcap or sinks is not None or value_dim \
+                or chunk or weights != "softmax":
             assert out is None and n_tokens is None and (n_v_heads or KV) == v_pages.shape[1]
             return self._attention_general(q, k_pages, v_pages, block_table, q_start, kv_len, n_seqs, scale, window,
                                            page_size, keep_first, distance_bias, distance_buckets, gate, out_dtype,
-                                           softcap, sinks, value_dim)
+                                           softcap, sinks, value_dim, chunk, weights, score_bias)
         # the same contract as the kernels' front end: the step's bounds cover its requests and fit the table
         assert block_table.shape[1] * page_size >= max_kv_len, "block_table is too narrow for max_kv_len"
         assert int(kv_len[:n_seqs].max()) <= max_kv_len and n_seqs <= block_table.shape[0]
@@ -598,9 +644,9 @@ class TorchOps:
 
     def _attention_general(self, q, k_pages, v_pages, block_table, q_start, kv_len, n_seqs, scale, window, page_size,
                            keep_first, distance_bias, distance_buckets, gate, out_dtype=None, softcap=0.0, sinks=None,
-                           value_dim=None):
+                           value_dim=None, chunk=None, weights="softmax", score_bias=None):
         """Everything the general kernel can do, key by visible key: kept first tokens behind a
-        window, a bias by bucketed distance, values of another size, an output gate per head
+        window, chunks, softmax or sigmoid weights, a bias by bucketed distance, values of another size, an output gate per head
         ([T, H]) or per element ([T, H * dv])."""
         T, H, hd = q.shape
         KV, dv, VH = k_pages.shape[1], v_pages.shape[3], v_pages.shape[1]
@@ -612,7 +658,7 @@ class TorchOps:
         for b in range(n_seqs):
             ql, L = qs[b + 1] - qs[b], kl[b]
             qpos = torch.arange(L - ql, L, device=q.device)
-            lo = max(0, (L - ql) - window + 1) if window else 0
+            lo = max(0, (L - ql) - window + 1) if window else (L - ql) // chunk * chunk if chunk else 0
             pos = torch.cat([torch.arange(0, min(keep_first, lo), device=q.device), torch.arange(lo, L, device=q.device)])
             pages = block_table[b].long()[pos // page_size]
             assert (pages >= 0).all(), "attention would read a page that was given back"
@@ -623,6 +669,8 @@ class TorchOps:
             hidden = dist < 0
             if window:
                 hidden = hidden | ((dist >= window) & (pos[None, :] >= keep_first))
+            if chunk:
+                hidden = hidden | (pos[None, :] // chunk != qpos[:, None] // chunk)
             for h in range(H):
                 s = (qq[:, h] @ k[:, h // group].T) * scale
                 if distance_bias is not None:
@@ -630,7 +678,9 @@ class TorchOps:
                 if softcap:
                     s = np.float32(softcap) * torch.tanh(s / np.float32(softcap))
                 s = s.masked_fill(hidden, float("-inf"))
-                if sinks is not None:        # one more term in the denominator, without a value
+                if weights == "sigmoid":
+                    o = torch.sigmoid(s if score_bias is None else s + score_bias[h]) @ v[:, (h // group) % VH]
+                elif sinks is not None:        # one more term in the denominator, without a value
                     s = torch.cat([s, sinks[h].expand(ql, 1)], dim=1)
                     o = torch.softmax(s, -1)[:, :-1] @ v[:, (h // group) % VH]
                 else:

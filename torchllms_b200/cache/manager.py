@@ -7,9 +7,9 @@ page (:225), a block table and a length per live request (:230-231) with
 ``len(pages) == ceil(length / page_size)`` (:129-130), lazy growth (:332-350),
 handles that are never used twice (:271-281) and an invariant checker
 (:797-843).  Different from it: growth is all-or-nothing over a whole batch;
-runs of layers are sorted into *groups* by what they need (all keys, or a
-window of them), each group with pages and block tables of its own, a window
-group giving pages back once the window has passed them (all but the pages of
+runs of layers are sorted into *groups* by what they need (all keys, a window
+of them, or those of the current chunk), each group with pages and block tables
+of its own, a window or chunk group giving pages back once no query can see them (all but the pages of
 the first tokens, where the need says that those are read for ever); values may
 have another size than keys, or not be stored at all; and every live
 request also owns a dense *slot* that indexes fixed-size state rows and the
@@ -123,8 +123,9 @@ class CacheGroup:
         v_shape = (len(runs), n_pages, need.value_heads, page_size, need.value_dim)
         self.v_pages = torch.zeros(v_shape, dtype=dtype, device=device) if need.value_dim else None
         self.run_index = {run: i for i, run in enumerate(self.runs)}
+        self.gives_back = need.kind != "full"      # pages that no later query can read go back while the request lives
         # blocks that hold the first tokens a window keeps: never given back while the request lives
-        self.kept_blocks = -(-need.keep_first // page_size) if need.kind == "window" else 0
+        self.kept_blocks = -(-need.keep_first // page_size) if self.gives_back else 0
 
     def bytes(self) -> int:
         return sum(t.numel() * t.element_size() for t in (self.k_pages, self.v_pages) if t is not None)
@@ -174,7 +175,7 @@ class CacheManager:
             by_need.setdefault(need, []).append(i)
         for need, runs in by_need.items():
             n_pages = full_pages
-            if need.kind == "window":
+            if need.kind != "full":
                 step = max_step_tokens if max_step_tokens is not None else self.max_len
                 per_req = -(-(need.window + step) // self.page_size) + 1 + -(-need.keep_first // self.page_size)
                 n_pages = min(full_pages, self.max_num_seqs * per_req)
@@ -328,18 +329,17 @@ class CacheManager:
         return starts
 
     def pass_window(self, handle: int) -> int:
-        """After a step: give back the pages of window groups that no later query can see.
+        """After a step: give back the pages of window and chunk groups that no later query can see.
 
         A query at position ``p`` of a window ``w`` reads keys ``p - w + 1 .. p`` (and the
-        first ``keep_first`` keys, whose blocks stay); the next query sits at ``length``.
-        Returns how many pages were freed."""
+        first ``keep_first`` keys, whose blocks stay), one of a chunk the keys from the chunk's first
+        to ``p``; the next query sits at ``length``.  Returns how many pages were freed."""
         req = self._req(handle)
         freed = 0
         for gi, g in enumerate(self.groups):
-            if g.need.kind != "window":
+            if not g.gives_back:
                 continue
-            first_needed = req.length - g.need.window + 1
-            last_dead_block = first_needed // self.page_size if first_needed > 0 else 0
+            last_dead_block = g.need.first_needed(req.length) // self.page_size
             for b in range(max(req.first_block[gi], g.kept_blocks), min(last_dead_block, len(req.blocks[gi]))):
                 p = req.blocks[gi][b]
                 if p != FREED:
@@ -357,8 +357,8 @@ class CacheManager:
             raise CacheError(f"request {handle}: cannot truncate {req.length} tokens to {new_length}")
         keep = -(-new_length // self.page_size)
         for gi, g in enumerate(self.groups):       # check every group before touching any
-            if g.need.kind == "window" and req.first_block[gi] > g.kept_blocks:
-                first_needed = new_length - g.need.window + 1
+            if g.gives_back and req.first_block[gi] > g.kept_blocks:
+                first_needed = g.need.first_needed(new_length)
                 if first_needed < req.first_block[gi] * self.page_size:
                     raise CacheError(
                         f"request {handle}: truncating to {new_length} would need keys that window "
@@ -411,7 +411,7 @@ class CacheManager:
                         f"group {gi} request {req.handle}: {len(blocks)} blocks for {req.length} tokens")
                 for b, p in enumerate(blocks):
                     if p == FREED:
-                        if g.need.kind != "window" or b >= req.first_block[gi] or b < g.kept_blocks:
+                        if not g.gives_back or b >= req.first_block[gi] or b < g.kept_blocks:
                             raise AssertionError(f"group {gi} request {req.handle}: block {b} has no page")
                         continue
                     if g.kept_blocks <= b < req.first_block[gi]:

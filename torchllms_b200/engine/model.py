@@ -42,7 +42,8 @@ class Model:
         self.position_table: Optional[torch.Tensor] = None
         self.head: Optional[torch.Tensor] = None
         self.row_tensors: Dict[str, torch.Tensor] = {}
-        self.keeps_embedding = any(run.add_embedding for run in spec.run_order)
+        self.join_tensors: Dict[str, torch.Tensor] = {}
+        self.keeps_embedding = any(run.add_embedding or run.join_embedding is not None for run in spec.run_order)
 
     # ----------------------------------------------------------------- weights
     def expected_tensors(self) -> Dict[str, ExpectedTensor]:
@@ -62,6 +63,8 @@ class Model:
             out[spec.head_tensor] = ExpectedTensor((spec.vocab_size, spec.dim))
         for name, rows in spec.row_tensors:
             out[name] = ExpectedTensor((rows, spec.dim))
+        for name in spec.join_tensors:
+            out[name] = ExpectedTensor((spec.dim, 2 * spec.dim))
         return out
 
     def load(self, tensors: Mapping[str, torch.Tensor]) -> None:
@@ -81,12 +84,14 @@ class Model:
         # rows that runs add to the stream: kept in 32-bit, as the stream is
         self.row_tensors = {name: tensors[name].to(device=self.device, dtype=torch.float32).contiguous()
                             for name, _rows in spec.row_tensors}
+        self.join_tensors = {name: as_compute(tensors[name], self.env) for name in spec.join_tensors}
 
     def weight_bytes(self) -> int:
         """Bytes of weights a step has to read: every layer's matrices and the head once
         (of the embedding table a step reads only the rows of its tokens)."""
         return sum(blk.weight_bytes() for blk in self.blocks) + self.final_norm.weight_bytes() \
-            + self.head.numel() * self.head.element_size()
+            + self.head.numel() * self.head.element_size() \
+            + sum(t.numel() * t.element_size() for t in self.join_tensors.values())
 
     # ------------------------------------------------------------------- cache
     def run_needs(self) -> List[Tuple[Optional[CacheNeed], Optional[StateNeed], Optional[int]]]:
@@ -117,7 +122,19 @@ class Model:
         residual.h, residual.rows = nxt, None
 
     def _add_before_run(self, residual: Residual, run, embedding_output: Optional[torch.Tensor]) -> None:
-        """``h += embedding output + row`` (either may be absent), in 32-bit, before a run that asks for it."""
+        """``h += embedding output + row`` (either may be absent), in 32-bit, before a run that asks for it; or, for a
+        run that joins the two, ``h <- W [h; embedding output] + row``: a kernel takes the pending sum and lays the
+        product's input out, and the product is left pending on a stream that holds the row."""
+        if run.join_embedding is not None:
+            if residual.normed is not None or residual.history is not None:
+                raise RuntimeError("a product in front of a run needs a stream without a norm taken ahead and no kept history")
+            row = None if run.add_row is None else self.row_tensors[run.add_row[0]][run.add_row[1]]
+            both, residual.h = self.ops.stream_join(residual.h, residual.delta, residual.delta_scale, embedding_output, row,
+                                                    out_dtype=self.dtype)
+            # (the stream is 32-bit, so the product that makes it leaves in 32-bit too)
+            residual.delta = self.ops.linear(both, self.join_tensors[run.join_embedding], out_dtype=torch.float32, partials_ok=True)
+            residual.delta_scale = residual.rows = None
+            return
         if residual.delta is not None or residual.normed is not None or residual.history is not None:
             raise RuntimeError("a sum in front of a run needs a stream with nothing pending and no kept history")
         row = None
@@ -148,14 +165,18 @@ class Model:
             residual = Residual(self.ops.rmsnorm(residual.h, None, self.embedding_norm.weight, self.embedding_norm.eps,
                                                  out_dtype=torch.float32))
         order = self.spec.run_order
-        embedding_output = residual.h.clone() if self.keeps_embedding else None
+        embedding_output = None
+        if self.keeps_embedding:
+            # (a first run that joins writes a new stream and leaves this one as it is)
+            embedding_output = residual.h if order[0].join_embedding is not None else residual.h.clone()
         for i, run in enumerate(order):
-            if run.add_embedding or run.add_row is not None:
+            if run.add_embedding or run.add_row is not None or run.join_embedding is not None:
                 self._add_before_run(residual, run, embedding_output)
             follows = order[i + 1] if i + 1 < len(order) else None
             # (a run that starts with a sum onto the stream takes its own input norm afterwards)
             residual.next_norm = (self.blocks[follows.layer].input_norm
-                                  if follows is not None and not (follows.add_embedding or follows.add_row is not None) else None)
+                                  if follows is not None and not (follows.add_embedding or follows.add_row is not None
+                                                                  or follows.join_embedding is not None) else None)
             self.blocks[run.layer].forward(residual, ctx, views[i])
             if residual.history is not None and residual.level != i + 1:
                 self._next_level(residual)      # a block that reads no earlier results: the stream passes as it is

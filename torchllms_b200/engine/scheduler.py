@@ -125,15 +125,15 @@ class Scheduler:
 
     def _most_cached_tokens(self, need: int) -> int:
         """How long a request that has the pool to itself may grow, given that it wants ``need``.
-        A group that keeps every key holds its page count times the page size.  A window group
-        gives pages back as the request grows: it only has to hold the window and the portion
+        A group that keeps every key holds its page count times the page size.  A window or chunk group
+        gives pages back as the request grows: it only has to hold the window (the chunk) and the portion
         being fed (plus a page for where they start and end), however long the request gets."""
         cache = self.engine.cache
         page = cache.page_size
         most = need
         for g in cache.groups:
             held = g.allocator.n_pages * page
-            if g.need.kind == "window":
+            if g.gives_back:
                 portion = min(self.prefill_chunk, self.max_num_batched_tokens)
                 if (-(-(g.need.window + portion) // page) + 1) * page <= held:
                     continue                      # it never holds more than that: no limit from this group

@@ -162,7 +162,7 @@ class Engine:
                                   max_num_seqs=max_num_seqs, max_len=self.max_len, dtype=model.dtype,
                                   device=self.device, max_step_tokens=self.max_step_tokens)
         self._buf = _StepBuffers(self.cache, self.max_step_tokens, self.device)
-        self._has_window = any(g.need.kind == "window" for g in self.cache.groups)
+        self._has_window = any(g.gives_back for g in self.cache.groups)
         self.vocab_size = model.spec.vocab_size
         self.steps_run = 0
         self.tokens_run = 0

@@ -338,26 +338,37 @@ class RotaryGatedAttention(Mixer):
     switches of the spec:
 
     * projections ``wq, wk, wv`` (and ``wo``) with optional biases (``qkv_bias``, ``out_bias``), keys and
-      values of sizes of their own (``head_dim``, ``v_head_dim``);
+      values of sizes of their own (``head_dim``, ``v_head_dim``); with ``values_are_keys`` there is no ``wv`` and a
+      value is the key as projected (biases included), before any norm or rotation;
+    * with ``qk_row_norm`` an RMS norm over all of q at once and over all of k at once, before they are cut into heads
+      (plain weights ``q_norm.weight``, ``k_norm.weight``), ahead of the rotation;
     * rotation of the first ``rot_dims`` coordinates of every q and k head by ``p * rot_base^(-2i/rot_dims)``
-      (``rot_pairing`` ``"interleaved"``: coordinate ``2i`` with ``2i + 1``; ``"half"``: ``i`` with ``i + rot_dims / 2``);
+      (``rot_pairing`` ``"interleaved"``: coordinate ``2i`` with ``2i + 1``; ``"half"``: ``i`` with ``i + rot_dims / 2``), the
+      frequencies optionally rescaled by band (``rot_band``, see :func:`~torchllms_b200.parts.rope.band_scaled`);
+    * with ``qk_head_norm`` every rotated head of q and k, and with ``v_head_norm`` every head's value, is divided by its
+      root mean square (no weight); keys and values are stored so;
     * score ``= q . k * scale``, then, with ``softcap = c > 0``, ``c * tanh(score / c)``;
-    * causal, optionally behind a sliding ``window``;
-    * softmax whose denominator, with ``sinks``, also holds ``exp(sinks[h])``: a learned number per head
-      (tensor ``sinks``) that stands for a key without a value and is neither scaled nor capped;
+    * causal, optionally behind a sliding ``window`` or inside chunks (a query sees keys of its own run of ``chunk``
+      positions, counted from the request's first token);
+    * ``weights="softmax"``: softmax whose denominator, with ``sinks``, also holds ``exp(sinks[h])``: a learned number per
+      head (tensor ``sinks``) that stands for a key without a value and is neither scaled nor capped, or, with
+      ``sinks="zero"``, ``exp(0)`` and no tensor; ``weights="sigmoid"``: a visible key's weight is ``sigmoid(score +
+      score_bias[h])`` (tensor ``score_bias``, a number per head), not normalised over the keys;
     * an output gate ``sigmoid(wg x)``, one number per head (``gate="head"``) or per element
       (``"element"``), ahead of ``wo``.
 
-    One stacked product gives q, k, v and the gate's logits; one kernel adds the biases, rotates,
-    stores keys and values and takes the gate's sigmoid; cap, sink and gate live in the attention
+    One stacked product gives q, k, v and the gate's logits; one kernel adds the biases, norms, rotates,
+    stores keys and values and takes the gate's sigmoid; mask, cap, sink, sigmoid and gate live in the attention
     kernel; the output bias is added where the output product is added up."""
 
     graph_safe = True
 
     def __init__(self, env: BuildEnv, *, dim: int, n_heads: int, n_kv_heads: int, head_dim: int,
-                 v_head_dim: Optional[int] = None, scale: float, softcap: float = 0.0, sinks: bool = False,
+                 v_head_dim: Optional[int] = None, scale: float, softcap: float = 0.0, sinks=False,
                  rot_dims: int = 0, rot_base: float = 10000.0, rot_pairing: str = "interleaved", window: Optional[int] = None,
-                 qkv_bias: bool = False, out_bias: bool = False, gate: Optional[str] = None):
+                 qkv_bias: bool = False, out_bias: bool = False, gate: Optional[str] = None, rot_band: Optional[Mapping[str, float]] = None,
+                 chunk: Optional[int] = None, values_are_keys: bool = False, qk_row_norm: bool = False, qk_head_norm: bool = False,
+                 v_head_norm: bool = False, norm_eps: float = 1e-6, weights: str = "softmax", score_bias: bool = False):
         if n_heads % n_kv_heads != 0:
             raise ValueError(f"n_heads ({n_heads}) must be a multiple of n_kv_heads ({n_kv_heads})")
         if rot_dims < 0 or rot_dims % 2 or rot_dims > head_dim:
@@ -368,32 +379,53 @@ class RotaryGatedAttention(Mixer):
             raise ValueError(f"gate must be None, 'element' or 'head', got {gate!r}")
         if softcap < 0:
             raise ValueError(f"softcap must not be negative, got {softcap}")
+        if window is not None and chunk is not None:
+            raise ValueError("attention looks back through a window or inside chunks, not both")
+        if weights not in ("softmax", "sigmoid"):
+            raise ValueError(f"attention weights are 'softmax' or 'sigmoid', got {weights!r}")
+        if sinks not in (False, True, "zero") or (sinks and weights != "softmax") or (score_bias and weights != "sigmoid"):
+            raise ValueError("sinks (True or 'zero') go with softmax weights, a score bias with sigmoid weights")
+        if values_are_keys and v_head_dim not in (None, head_dim):
+            raise ValueError(f"values that are keys have the keys' size ({head_dim}), got v_head_dim {v_head_dim}")
         self.env = env
         self.dim, self.n_heads, self.n_kv_heads = int(dim), int(n_heads), int(n_kv_heads)
         self.head_dim = int(head_dim)
         self.v_head_dim = int(v_head_dim if v_head_dim is not None else head_dim)
         self.scale, self.softcap = float(scale), float(softcap)
-        self.has_sinks, self.qkv_bias, self.out_bias, self.gate = bool(sinks), bool(qkv_bias), bool(out_bias), gate
+        self.zero_sink = sinks == "zero"
+        self.has_sinks, self.qkv_bias, self.out_bias, self.gate = sinks is True, bool(qkv_bias), bool(out_bias), gate
         self.rot_dims, self.interleaved = int(rot_dims), rot_pairing == "interleaved"
         self.window = None if window is None else int(window)
-        self.n_q, self.n_k, self.n_v = self.n_heads * self.head_dim, self.n_kv_heads * self.head_dim, self.n_kv_heads * self.v_head_dim
+        self.chunk = None if chunk is None else int(chunk)
+        if min(x for x in (self.window, self.chunk, 1) if x is not None) < 1:
+            raise ValueError(f"a window or a chunk holds at least one key, got {window or chunk}")
+        self.values_are_keys, self.qk_row_norm = bool(values_are_keys), bool(qk_row_norm)
+        self.qk_head_norm, self.v_head_norm, self.norm_eps = bool(qk_head_norm), bool(v_head_norm), float(norm_eps)
+        self.weights, self.has_score_bias = weights, bool(score_bias)
+        self.n_q, self.n_k = self.n_heads * self.head_dim, self.n_kv_heads * self.head_dim
+        self.n_v = 0 if self.values_are_keys else self.n_kv_heads * self.v_head_dim
         self.n_g = {None: 0, "head": self.n_heads, "element": self.n_heads * self.v_head_dim}[gate]
         env.ops.check_attention_sizes(self.n_heads, self.n_kv_heads, self.head_dim, env.dtype, v_head_dim=self.v_head_dim)
-        self.table = precise_rotary_table(max(self.rot_dims, 2), rot_base, 1.0, env.max_positions, env.device)
-        self.w_in = self.b_in = self.sinks = self.wo = self.bo = None
+        self.table = precise_rotary_table(max(self.rot_dims, 2), rot_base, 1.0, env.max_positions, env.device, band=rot_band)
+        self.w_in = self.b_in = self.sinks = self.wo = self.bo = self.q_norm_w = self.k_norm_w = self.score_bias = None
 
     def cache_need(self) -> CacheNeed:
+        if self.chunk is not None:
+            return CacheNeed("chunk", self.n_kv_heads, self.head_dim, self.chunk, self.v_head_dim)
         if self.window is None:
             return CacheNeed("full", self.n_kv_heads, self.head_dim, None, self.v_head_dim)
         return CacheNeed("window", self.n_kv_heads, self.head_dim, self.window, self.v_head_dim)
 
     def expected_tensors(self) -> Dict[str, ExpectedTensor]:
-        out = {"wq.weight": ExpectedTensor((self.n_q, self.dim)), "wk.weight": ExpectedTensor((self.n_k, self.dim)),
-               "wv.weight": ExpectedTensor((self.n_v, self.dim)),
-               "wo.weight": ExpectedTensor((self.dim, self.n_heads * self.v_head_dim))}
-        if self.qkv_bias:
-            out.update({"wq.bias": ExpectedTensor((self.n_q,)), "wk.bias": ExpectedTensor((self.n_k,)),
-                        "wv.bias": ExpectedTensor((self.n_v,))})
+        out = {"wo.weight": ExpectedTensor((self.dim, self.n_heads * self.v_head_dim))}
+        for name, rows in self._projected():
+            out[f"{name}.weight"] = ExpectedTensor((rows, self.dim))
+            if self.qkv_bias:
+                out[f"{name}.bias"] = ExpectedTensor((rows,))
+        if self.qk_row_norm:
+            out.update({"q_norm.weight": ExpectedTensor((self.n_q,)), "k_norm.weight": ExpectedTensor((self.n_k,))})
+        if self.has_score_bias:
+            out["score_bias"] = ExpectedTensor((self.n_heads,))
         if self.out_bias:
             out["wo.bias"] = ExpectedTensor((self.dim,))
         if self.has_sinks:
@@ -402,13 +434,24 @@ class RotaryGatedAttention(Mixer):
             out["wg.weight"] = ExpectedTensor((self.n_g, self.dim))
         return out
 
+    def _projected(self):
+        """``(name, rows)`` of the stacked projections of q, k and v, in order."""
+        return [("wq", self.n_q), ("wk", self.n_k)] + ([] if self.values_are_keys else [("wv", self.n_v)])
+
     def load(self, tensors: Mapping[str, torch.Tensor]) -> None:
         f32 = dict(device=self.env.device, dtype=torch.float32)
-        names = ["wq.weight", "wk.weight", "wv.weight"] + (["wg.weight"] if self.gate else [])
+        names = [f"{n}.weight" for n, _rows in self._projected()] + (["wg.weight"] if self.gate else [])
         self.w_in = torch.cat([as_compute(tensors[n], self.env) for n in names])       # rows [wq; wk; wv; wg]
         if self.qkv_bias:
-            self.b_in = torch.cat([tensors[n].to(**f32) for n in ("wq.bias", "wk.bias", "wv.bias")]
+            self.b_in = torch.cat([tensors[f"{n}.bias"].to(**f32) for n, _rows in self._projected()]
                                   + [torch.zeros(self.n_g, **f32)]).contiguous()
+        if self.qk_row_norm:
+            self.q_norm_w = tensors["q_norm.weight"].to(**f32).contiguous()
+            self.k_norm_w = tensors["k_norm.weight"].to(**f32).contiguous()
+        if self.has_score_bias:
+            self.score_bias = tensors["score_bias"].to(**f32).contiguous()
+        if self.zero_sink:
+            self.sinks = torch.zeros(self.n_heads, **f32)
         if self.out_bias:
             self.bo = tensors["wo.bias"].to(**f32).contiguous()
         if self.has_sinks:
@@ -421,13 +464,19 @@ class RotaryGatedAttention(Mixer):
     def forward(self, x: torch.Tensor, ctx, cache) -> PendingProduct:
         ops = self.env.ops
         proj = ops.linear(x, self.w_in, partials_ok=True)
-        q, gate = ops.rope_store(
-            proj, ctx.positions, self.table, n_q_heads=self.n_heads, n_k_heads=self.n_kv_heads, n_v_heads=self.n_kv_heads,
-            head_dim=self.head_dim, v_head_dim=self.v_head_dim, rot_dims=self.rot_dims, interleaved=self.interleaved,
-            n_extra=self.n_g, k_pages=cache.k_pages, v_pages=cache.v_pages, slot_mapping=cache.slot_mapping,
-            page_size=cache.page_size, out_dtype=self.env.dtype, bias=self.b_in)
+        store = dict(n_q_heads=self.n_heads, n_k_heads=self.n_kv_heads, head_dim=self.head_dim, v_head_dim=self.v_head_dim,
+                     rot_dims=self.rot_dims, interleaved=self.interleaved, n_extra=self.n_g, k_pages=cache.k_pages,
+                     v_pages=cache.v_pages, slot_mapping=cache.slot_mapping, page_size=cache.page_size, out_dtype=self.env.dtype,
+                     bias=self.b_in)
+        if self.qk_row_norm or self.qk_head_norm or self.v_head_norm or self.values_are_keys:
+            q, gate = ops.norm_rope_store(proj, ctx.positions, self.table, values_are_keys=self.values_are_keys,
+                                          q_norm=self.q_norm_w, k_norm=self.k_norm_w, qk_head_norm=self.qk_head_norm,
+                                          v_head_norm=self.v_head_norm, eps=self.norm_eps, **store)
+        else:
+            q, gate = ops.rope_store(proj, ctx.positions, self.table, n_v_heads=self.n_kv_heads, **store)
         o = ops.paged_attention(
             q, cache.k_pages, cache.v_pages, cache.block_table, ctx.q_start, ctx.kv_len, n_seqs=ctx.n_seqs,
-            max_q_len=ctx.max_q_len, max_kv_len=ctx.max_kv_len, scale=self.scale, window=self.window,
-            page_size=cache.page_size, gate=gate, softcap=self.softcap, sinks=self.sinks, impl="auto")
+            max_q_len=ctx.max_q_len, max_kv_len=ctx.max_kv_len, scale=self.scale, window=self.window, chunk=self.chunk,
+            page_size=cache.page_size, gate=gate, softcap=self.softcap, sinks=self.sinks, weights=self.weights,
+            score_bias=self.score_bias, impl="auto")
         return PendingProduct(o.view(o.shape[0], self.n_heads * self.v_head_dim), self.wo, bias=self.bo)

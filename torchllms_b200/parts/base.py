@@ -47,10 +47,12 @@ class BuildEnv:
 class CacheNeed:
     """Paged key/value storage a mixer wants for every token of a request.
 
-    ``kind`` is ``"full"`` (all keys stay) or ``"window"`` (only the last
+    ``kind`` is ``"full"`` (all keys stay), ``"window"`` (only the last
     ``window`` keys are ever read, so older pages may be given back; with
     ``keep_first`` the first so many tokens of a request are read for ever and
-    their pages stay).  ``v_head_dim`` is the size of a stored value when it
+    their pages stay) or ``"chunk"`` (a request's positions fall into chunks of ``window``, counted from its
+    first token, and a query reads keys of its own chunk only: when a request enters a new chunk, the
+    pages of all earlier ones may be given back).  ``v_head_dim`` is the size of a stored value when it
     differs from a key's; 0 means that nothing but keys is stored (a mixer
     that derives keys and values from one stored vector).  ``n_v_heads`` is the number of value
     heads when it differs from the number of key heads (key head ``j`` then goes with value head
@@ -67,10 +69,10 @@ class CacheNeed:
     n_v_heads: Optional[int] = None
 
     def __post_init__(self):
-        if self.kind not in ("full", "window"):
-            raise ValueError(f"cache kind must be 'full' or 'window', got {self.kind!r}")
-        if (self.kind == "window") != (self.window is not None):
-            raise ValueError("a window size goes with kind 'window' and only with it")
+        if self.kind not in ("full", "window", "chunk"):
+            raise ValueError(f"cache kind must be 'full', 'window' or 'chunk', got {self.kind!r}")
+        if (self.kind != "full") != (self.window is not None):
+            raise ValueError("a window size goes with kinds 'window' and 'chunk' and only with them")
         if self.keep_first < 0 or (self.keep_first and self.kind != "window"):
             raise ValueError("keep_first is a count of tokens and goes with kind 'window' only")
         if self.v_head_dim is not None and self.v_head_dim == self.head_dim:
@@ -91,6 +93,14 @@ class CacheNeed:
         """How many heads a stored value has."""
         return self.n_kv_heads if self.n_v_heads is None else self.n_v_heads
 
+    def first_needed(self, position: int) -> int:
+        """The first key that a query at ``position`` or any later place reads (apart from ``keep_first``)."""
+        if self.kind == "window":
+            return max(0, position - self.window + 1)
+        if self.kind == "chunk":
+            return position // self.window * self.window
+        return 0
+
     def covering(self, other: "CacheNeed") -> "CacheNeed":
         """The need that keeps what both this one and ``other`` (a run that reads this run's cache
         through a mask of its own) will read."""
@@ -99,6 +109,9 @@ class CacheNeed:
             raise ValueError("a run can read another run's cache only if both store the same vectors")
         if self.kind == "full" or other.kind == "full":
             return CacheNeed("full", self.n_kv_heads, self.head_dim, None, self.v_head_dim, 0, self.n_v_heads)
+        if self == other:
+            return self
+        # (a chunk never reaches further back than a window of its size)
         return CacheNeed("window", self.n_kv_heads, self.head_dim, max(self.window, other.window), self.v_head_dim,
                          max(self.keep_first, other.keep_first), self.n_v_heads)
 
@@ -277,6 +290,9 @@ class Residual:
     ``h`` left such a copy (a block whose sublayers read the stream itself, without a norm in
     front, takes its input from there); whoever changes ``h`` afterwards sets it to ``None``.
 
+    ``delta_scale`` (float32 ``[dim]``, or ``None``): what the pending delta is multiplied by, element by element, when
+    it is added (a layer scale).
+
     ``history`` is there for models whose layers read earlier layers' results
     (``ModelSpec.keeps_history``): ``[levels, T, dim]`` float32, level 0 the embedding output,
     level ``j`` the result of the ``j``-th layer run; ``level`` counts the finished ones, and ``h``
@@ -288,12 +304,13 @@ class Residual:
     instead of running its norm.
     """
 
-    __slots__ = ("h", "delta", "rows", "history", "level", "next_norm", "normed")
+    __slots__ = ("h", "delta", "delta_scale", "rows", "history", "level", "next_norm", "normed")
 
     def __init__(self, h: torch.Tensor, delta: Optional[torch.Tensor] = None, rows: Optional[torch.Tensor] = None,
                  history: Optional[torch.Tensor] = None):
         self.h = h
         self.delta = delta
+        self.delta_scale: Optional[torch.Tensor] = None
         self.rows = rows
         self.history = history
         self.level = 0

@@ -24,19 +24,29 @@ from .spec import PartSpec
 
 @register_block("prenorm")
 class PreNormBlock(Block):
-    """Sub-part tensor prefixes are parameters, so the block does not know whose names they are."""
+    """Sub-part tensor prefixes are parameters, so the block does not know whose names they are.  A layer may
+    have no feed-forward (``feed_forward=None``), and then has no second norm either.
 
-    def __init__(self, env: BuildEnv, *, mixer: PartSpec, feed_forward: PartSpec,
-                 mixer_norm: PartSpec, ffn_norm: PartSpec,
-                 mixer_prefix: str, ffn_prefix: str, mixer_norm_prefix: str, ffn_norm_prefix: str):
+    ``mixer_scale`` / ``ffn_scale``: names of stored ``[dim]`` vectors (layer scales) by which a sublayer's result is
+    multiplied, element by element, before it is added; the norm that takes the sum multiplies, in 32-bit."""
+
+    def __init__(self, env: BuildEnv, *, mixer: PartSpec, feed_forward: Optional[PartSpec],
+                 mixer_norm: PartSpec, ffn_norm: Optional[PartSpec],
+                 mixer_prefix: str, ffn_prefix: str, mixer_norm_prefix: str, ffn_norm_prefix: str,
+                 mixer_scale: Optional[str] = None, ffn_scale: Optional[str] = None):
         self.env = env
         self.mixer = MIXERS.build(mixer, env)
-        self.feed_forward = FEED_FORWARDS.build(feed_forward, env)
         self.mixer_norm = NORMS.build(mixer_norm, env)
-        self.ffn_norm = NORMS.build(ffn_norm, env)
-        self.graph_safe = all(x.graph_safe for x in (self.mixer, self.feed_forward, self.mixer_norm, self.ffn_norm))
-        self._subparts = ((mixer_prefix, self.mixer), (ffn_prefix, self.feed_forward),
-                          (mixer_norm_prefix, self.mixer_norm), (ffn_norm_prefix, self.ffn_norm))
+        self._subparts = [(mixer_prefix, self.mixer), (mixer_norm_prefix, self.mixer_norm)]
+        self.feed_forward = self.ffn_norm = None
+        if feed_forward is not None:
+            self.feed_forward = FEED_FORWARDS.build(feed_forward, env)
+            self.ffn_norm = NORMS.build(ffn_norm, env)
+            self._subparts += [(ffn_prefix, self.feed_forward), (ffn_norm_prefix, self.ffn_norm)]
+        self.graph_safe = all(sub.graph_safe for _p, sub in self._subparts)
+        self.mixer_scale, self.ffn_scale = mixer_scale, (ffn_scale if feed_forward is not None else None)
+        self.mixer_ls: Optional[torch.Tensor] = None
+        self.ffn_ls: Optional[torch.Tensor] = None
 
     def cache_need(self):
         return self.mixer.cache_need()
@@ -49,17 +59,24 @@ class PreNormBlock(Block):
         for prefix, sub in self._subparts:
             for name, e in sub.expected_tensors().items():
                 out[f"{prefix}.{name}"] = e
+        for name in (self.mixer_scale, self.ffn_scale):
+            if name is not None:
+                out[name] = ExpectedTensor((self.env.dim,))
         return out
 
     def load(self, tensors: Mapping[str, torch.Tensor]) -> None:
         for prefix, sub in self._subparts:
             sub.load({name: tensors[f"{prefix}.{name}"] for name in sub.expected_tensors()})
+        f32 = dict(device=self.env.device, dtype=torch.float32)
+        self.mixer_ls = None if self.mixer_scale is None else tensors[self.mixer_scale].to(**f32).contiguous()
+        self.ffn_ls = None if self.ffn_scale is None else tensors[self.ffn_scale].to(**f32).contiguous()
 
     def forward(self, residual: Residual, ctx, cache) -> None:
         x = self._normed(self.mixer_norm, self.mixer, residual)
-        residual.delta = self.mixer.forward(x, ctx, cache)
-        x = self._normed(self.ffn_norm, self.feed_forward, residual)
-        residual.delta = self.feed_forward.forward(x, ctx)
+        residual.delta, residual.delta_scale = self.mixer.forward(x, ctx, cache), self.mixer_ls
+        if self.feed_forward is not None:
+            x = self._normed(self.ffn_norm, self.feed_forward, residual)
+            residual.delta, residual.delta_scale = self.feed_forward.forward(x, ctx), self.ffn_ls
 
     @staticmethod
     def _normed(norm, reader, residual: Residual):
@@ -209,7 +226,7 @@ class SandwichBlock(Block):
                                    f"but {'there is none' if history is None else f'{level + 2} exist'}")
             nxt = history[level + 2]
             follow = residual.next_norm
-            if isinstance(follow, RMSNorm):
+            if isinstance(follow, RMSNorm) and follow.groups == 1:
                 # the average and the next layer's input norm of it in one kernel
                 rows = self.env.ops.depth_mix(history, self.depth_coef, self.depth_inputs, nxt, then_weight=follow.weight,
                                               then_eps=follow.eps, out_dtype=self.env.dtype)
@@ -328,7 +345,7 @@ class ParallelBlock(Block):
         u = ops.linear(rows, self.side_gate_w, partials_ok=True)
         g = ops.side_gate(u, ctx.token_ids, self.side_table, out_dtype=self.env.dtype)
         follow = residual.next_norm
-        if isinstance(follow, RMSNorm):
+        if isinstance(follow, RMSNorm) and follow.groups == 1:
             residual.normed = (follow, self.side_norm.fold_normed(residual, PendingProduct(g, self.side_proj_w), then=follow))
         else:
             self.side_norm.fold_normed(residual, PendingProduct(g, self.side_proj_w), want_rows=False)

@@ -19,7 +19,7 @@ from ..kernels.lazy import PendingProduct
 from ..weights.loader import ExpectedTensor
 from .base import BuildEnv, FeedForward, as_compute, register_feed_forward
 
-EXPERT_ACTIVATIONS = ("relu2", "silu", "gelu_tanh", "clamped_swish")
+EXPERT_ACTIVATIONS = ("relu2", "silu", "gelu_tanh", "gelu", "clamped_swish")      # ("gelu" is the exact form, with erf)
 
 
 @register_feed_forward("routed_experts")

@@ -33,9 +33,15 @@ class RMSNorm(Norm):
     graph_safe = True
     can_defer = True
 
-    def __init__(self, env: BuildEnv, *, dim: int, eps: float, offset: float = 0.0, scalar: bool = False):
+    def __init__(self, env: BuildEnv, *, dim: int, eps: float, offset: float = 0.0, scalar: bool = False, groups: int = 1):
         """``offset``: what is added to the stored weight (1 for a weight that is kept around zero).
-        ``scalar``: the stored weight is one number for all coordinates (a tensor without axes)."""
+        ``scalar``: the stored weight is one number for all coordinates (a tensor without axes).
+        ``groups``: the row is cut into so many equal runs of neighbouring coordinates, each divided by a root
+        mean square of its own (one scale per row is not enough then, so nothing is deferred)."""
+        if groups < 1 or dim % groups:
+            raise ValueError(f"a norm over {dim} coordinates cannot have {groups} equal groups")
+        self.groups = int(groups)
+        self.can_defer = self.groups == 1
         self.env = env
         self.scalar = bool(scalar)
         self.dim = int(dim)
@@ -55,7 +61,13 @@ class RMSNorm(Norm):
         ops = self.env.ops
         # 32-bit mode keeps the reference's order of operations to the letter
         deferred = bool(deferred_ok and rows is None and self.env.dtype == torch.bfloat16)
-        delta = residual.delta
+        delta, scale = residual.delta, residual.delta_scale
+        if self.groups > 1 or scale is not None:
+            out = ops.rmsnorm(residual.h, delta, self.weight, self.eps, out_dtype=self.env.dtype, rows=rows, groups=self.groups,
+                              delta_scale=scale)
+            if rows is None:
+                residual.delta = residual.delta_scale = residual.rows = None
+            return out
         if deferred and isinstance(delta, PendingProduct) and ops.can_fuse_residual(delta, residual.h):
             out = ops.linear_residual_norm(delta, residual.h, self.weight, self.eps)   # h += product, in the product's kernel
             residual.delta = None
@@ -78,6 +90,8 @@ class RMSNorm(Norm):
         :class:`~torchllms_b200.kernels.lazy.PendingProduct`.  With ``then`` (the norm in front of
         the next reader) the same kernel also returns ``then(h)`` in the activation dtype."""
         ops = self.env.ops
+        if self.groups > 1 or (then is not None and then.groups > 1):
+            raise RuntimeError("a norm with groups stands in front of a sublayer, not on its output")
         residual.delta = None
         if then is not None:
             residual.rows = None

@@ -57,15 +57,30 @@ def rotary_table(freq: torch.Tensor, max_positions: int) -> torch.Tensor:
 _precise_tables: dict = {}
 
 
-def precise_rotary_table(dims: int, theta: float, factor: float, max_positions: int, device="cpu") -> torch.Tensor:
+def band_scaled(freq: torch.Tensor, factor: float, low: float, high: float, original: float) -> torch.Tensor:
+    """Frequencies rescaled by band (the llama3 rule) in ``freq``'s own precision: with wavelength
+    ``l = 2 pi / f``, ``f`` stays where ``l < original / high``, becomes ``f / factor`` where ``l > original / low``,
+    and between the two is blended by ``s = (original / l - low) / (high - low)``."""
+    wavelen = 2.0 * math.pi / freq
+    s = (original / wavelen - low) / (high - low) if high != low else torch.ones_like(freq)
+    blended = (1.0 - s) * freq / factor + s * freq
+    return torch.where(wavelen < original / high, freq, torch.where(wavelen > original / low, freq / factor, blended))
+
+
+def precise_rotary_table(dims: int, theta: float, factor: float, max_positions: int, device="cpu",
+                         band: Optional[Mapping[str, float]] = None) -> torch.Tensor:
     """``[max_positions, dims / 2, 2]`` float32 (cos, sin) of the angles ``p * theta^(-2i/dims) / factor``,
     the angles taken in 64-bit so that the table is exact to float32 rounding at any position.
+    ``band`` (``factor``, ``low``, ``high``, ``original``) rescales the frequencies by :func:`band_scaled`.
     Layers with the same numbers on the same device share one table."""
-    key = (int(dims), float(theta), float(factor), int(max_positions), str(device))
+    bands = None if band is None else tuple(float(band[k]) for k in ("factor", "low", "high", "original"))
+    key = (int(dims), float(theta), float(factor), int(max_positions), str(device), bands)
     table = _precise_tables.get(key)
     if table is None:
         i = torch.arange(dims // 2, dtype=torch.float64)
         freq = float(theta) ** (-2.0 * i / dims) / float(factor)
+        if bands is not None:
+            freq = band_scaled(freq, *bands)
         angles = torch.arange(max_positions, dtype=torch.float64)[:, None] * freq[None, :]
         table = torch.stack([torch.cos(angles), torch.sin(angles)], dim=-1).to(torch.float32).contiguous().to(device)
         if len(_precise_tables) >= 8:

@@ -59,12 +59,15 @@ class RunEntry:
     What may be added to the stream right before the run (a model that runs a span of layers
     several times starts every pass this way): ``add_embedding`` adds the embedding output (the
     stream as it was before the first run), ``add_row = (tensor, i)`` adds row ``i`` of a model-level
-    ``[rows, dim]`` tensor (``ModelSpec.row_tensors``) to every token.  Both sums are 32-bit."""
+    ``[rows, dim]`` tensor (``ModelSpec.row_tensors``) to every token.  Both sums are 32-bit.
+    ``join_embedding = tensor`` replaces the stream by a product first: with ``W`` the model-level ``[dim, 2 dim]``
+    matrix of that name (``ModelSpec.join_tensors``), ``h <- W [h; embedding output]``; a row is added after it."""
 
     layer: int
     cache_of: Optional[int] = None
     add_embedding: bool = False
     add_row: Optional[Tuple[str, int]] = None
+    join_embedding: Optional[str] = None
 
 
 @dataclass(frozen=True)
@@ -86,6 +89,7 @@ class ModelSpec:
     embedding_norm_prefix: str = "embedding_norm"    # prefix of that norm's tensors
     logit_scale: float = 1.0         # the head's products leave multiplied by this
     row_tensors: Tuple[Tuple[str, int], ...] = ()    # model-level (name, rows) tensors [rows, dim] whose rows runs add to the stream (RunEntry.add_row)
+    join_tensors: Tuple[str, ...] = ()               # model-level [dim, 2 dim] matrices that join the stream and the embedding output (RunEntry.join_embedding)
 
     def __post_init__(self):
         n = len(self.layers)
@@ -93,6 +97,9 @@ class ModelSpec:
         for i, run in enumerate(self.run_order):
             if run.add_row is not None and not (run.add_row[0] in rows and 0 <= run.add_row[1] < rows[run.add_row[0]]):
                 raise ValueError(f"run {i} adds row {run.add_row[1]} of '{run.add_row[0]}', which the model does not have")
+            if run.join_embedding is not None and (run.join_embedding not in self.join_tensors or run.add_embedding):
+                raise ValueError(f"run {i} joins the embedding output through '{run.join_embedding}', which the model does not have, "
+                                 "or adds it as well")
             if not 0 <= run.layer < n:
                 raise ValueError(f"run {i} names layer {run.layer}, but there are {n} layers")
             if run.cache_of is not None:
