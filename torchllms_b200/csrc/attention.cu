@@ -18,6 +18,10 @@
 //                exp(sinks[h]); it stands for a key without a value, counts once, and is neither scaled nor capped
 //   v_stride     elements from one stored value to the next when that is not v_head_dim: with v_pages being
 //                k_pages and v_stride = head_dim, a value is the first v_head_dim coordinates of a stored key
+//   chunk        a request's positions fall into chunks of this size (counted from its first token), and a query sees
+//                keys of its own chunk only
+//   sigmoid      the weight of a visible key is sigmoid(score + score_bias[h]) ([n_heads] float32, or none) and the
+//                weights are not divided by their sum
 //
 // What it computes, per query token at absolute position p of request b and query head h
 // (kv head h / (H / KV)):   o = softmax_k( q . k_k * scale ) v_k   over keys k <= p
@@ -61,6 +65,9 @@ struct AttnParams {
     int v_stride;        // elements between stored values (v_head_dim unless values are parts of wider vectors)
     float softcap;       // 0: none
     const float* sinks;  // [n_heads] or null
+    int chunk;           // 0: none
+    int sigmoid;
+    const float* score_bias;   // [n_heads] or null
     int table_stride;
     int n_heads, n_kv_heads, head_dim, v_head_dim, page_size;
     int group, gchunk, n_gchunks, tokens_per_tile;
@@ -120,7 +127,8 @@ __global__ void __launch_bounds__(NT) paged_attention_kernel(const AttnParams p)
     // The keys this tile's queries can see: the window's (or all up to the last query), and ahead of
     // them the kept first keys that the window has passed.  They are walked as one run u = 0 .. n_vis - 1,
     // u < n_kept being key u and the rest key win_lo + (u - n_kept).
-    const int win_lo = p.window > 0 ? max(0, qpos_min - p.window + 1) : 0;
+    const int win_lo = p.window > 0 ? max(0, qpos_min - p.window + 1) : p.chunk > 0 ? qpos_min / p.chunk * p.chunk : 0;
+    const int my_lo = p.window > 0 ? my_qpos - p.window + 1 : p.chunk > 0 ? my_qpos / p.chunk * p.chunk : 0;      // this row's first key
     const int n_kept = min(p.keep_first, win_lo);
     const int n_vis = n_kept + max(qpos_max + 1 - win_lo, 0);
     int k_lo = 0, k_hi = n_vis;
@@ -198,7 +206,7 @@ __global__ void __launch_bounds__(NT) paged_attention_kernel(const AttnParams p)
         for (int jj = 0; jj < 4; ++jj) {
             const int u = k0 + c + 8 * jj;
             const int kpos = u < n_kept ? u : win_lo + (u - n_kept);
-            ok[jj] = u < k_hi && kpos <= my_qpos && (p.window <= 0 || kpos > my_qpos - p.window || kpos < p.keep_first);
+            ok[jj] = u < k_hi && kpos <= my_qpos && (kpos >= my_lo || kpos < p.keep_first);
             s[jj] *= p.scale;
             if (p.softcap > 0.f) s[jj] = p.softcap * tanhf(s[jj] / p.softcap);
             if (ok[jj] && p.rel != nullptr) s[jj] += p.rel[(size_t)p.bucket[min(my_qpos - kpos, p.n_bucket - 1)] * p.n_heads + my_head];
@@ -209,7 +217,12 @@ __global__ void __launch_bounds__(NT) paged_attention_kernel(const AttnParams p)
         const float m_new = fmaxf(m, tile_max);
         float alpha = 1.f, row_sum = 0.f;
         float pr[4] = {0.f, 0.f, 0.f, 0.f};
-        if (m_new != -INFINITY) {
+        if (p.sigmoid) {
+            // no maximum and no sum: every visible key's weight by itself
+            const float sb = p.score_bias != nullptr ? p.score_bias[my_head] : 0.f;
+#pragma unroll
+            for (int jj = 0; jj < 4; ++jj) pr[jj] = ok[jj] ? 1.f / (1.f + expf(-(s[jj] + sb))) : 0.f;
+        } else if (m_new != -INFINITY) {
             alpha = expf(m - m_new);  // m = -inf gives 0
 #pragma unroll
             for (int jj = 0; jj < 4; ++jj) {
@@ -254,7 +267,7 @@ __global__ void __launch_bounds__(NT) paged_attention_kernel(const AttnParams p)
 #pragma unroll
             for (int jd = 0; jd < HD_MAX / 8; ++jd) acc[jd] *= a;
         }
-        float inv = l > 0.f ? 1.f / l : 0.f;
+        float inv = p.sigmoid ? 1.f : l > 0.f ? 1.f / l : 0.f;
         const T* gate = reinterpret_cast<const T*>(p.gate);
         if (p.gate_mode == 1) inv *= to_float(gate[row]);
 #pragma unroll
@@ -271,8 +284,8 @@ __global__ void __launch_bounds__(NT) paged_attention_kernel(const AttnParams p)
             if (c + jd * 8 < dv) o[c + jd * 8] = acc[jd];
         if (c == 0) {
             float* ml = p.part_ml + (row * p.n_splits + split) * 2;
-            ml[0] = m;
-            ml[1] = l;
+            ml[0] = p.sigmoid ? 0.f : m;
+            ml[1] = p.sigmoid ? 0.f : l;
         }
     }
 }
@@ -282,7 +295,7 @@ template <typename T>
 __global__ void attention_merge_kernel(const float* __restrict__ part_o, const float* __restrict__ part_ml,
                                        T* __restrict__ out, int n_splits, int head_dim,
                                        const T* __restrict__ gate, int gate_mode, int out_f32,
-                                       const float* __restrict__ sinks, int n_heads) {
+                                       const float* __restrict__ sinks, int n_heads, int sigmoid) {
     const size_t row = blockIdx.x;
     const float* ml = part_ml + row * n_splits * 2;
     float M = -INFINITY;
@@ -299,7 +312,7 @@ __global__ void attention_merge_kernel(const float* __restrict__ part_o, const f
             den = fmaf(w, ml[2 * i + 1], den);
         }
         if (sinks != nullptr) den += expf(sink - M);
-        float o = den > 0.f ? num / den : 0.f;
+        float o = sigmoid ? num : den > 0.f ? num / den : 0.f;       // (without a sum to divide by the partial results just add up)
         if (gate_mode == 1) o *= to_float(gate[row]);
         else if (gate_mode == 2) o *= to_float(gate[row * head_dim + d]);
         if (out_f32) reinterpret_cast<float*>(out)[row * head_dim + d] = o;
@@ -375,6 +388,9 @@ struct TlAttentionOptions {
     float softcap;          // 0: none
     const float* sinks;     // [n_heads] or null
     int v_stride;           // 0: as v_head_dim
+    int chunk;              // 0: none; not together with a window
+    int sigmoid;            // 1: sigmoid weights without a sum over the keys; not together with sinks
+    const float* score_bias;   // [n_heads] or null; sigmoid only
 };
 
 // How many key splits the general kernel would use for this batch, and how many float32 words of
@@ -401,7 +417,8 @@ extern "C" int tl_attention_plan(int n_tokens, int n_seqs, int n_heads, int n_kv
 // q: [n_tokens, n_heads, head_dim]; out: [n_tokens, n_heads, v_head_dim]; k_pages: [n_pages, n_kv_heads,
 // page_size, head_dim]; v_pages: the same with v_head_dim; block_table: [n_seqs, table_stride]; q_start:
 // [n_seqs + 1]; kv_len: [n_seqs] (length after this step's tokens were appended).  workspace: float32, as
-// large as tl_attention_plan_ex said for the same window and keep_first (may be null when it said 0).
+// large as tl_attention_plan_ex said for the same window (with chunks: for a window of a chunk's size) and keep_first
+// (may be null when it said 0).
 // window <= 0 means no window.
 extern "C" int tl_paged_attention_ex(const void* q, const void* k_pages, const void* v_pages, void* out,
                                      const int* block_table, int table_stride, const int* q_start,
@@ -423,9 +440,11 @@ extern "C" int tl_paged_attention_ex(const void* q, const void* k_pages, const v
     if (o.n_v_heads <= 0) o.n_v_heads = n_kv_heads;
     if (o.v_stride <= 0) o.v_stride = o.v_head_dim;
     if (o.v_stride < o.v_head_dim || o.softcap < 0.f) return TL_BAD_SIZE;
+    if (o.chunk < 0 || (o.chunk > 0 && window > 0) || (o.sigmoid && o.sinks != nullptr) || (o.score_bias != nullptr && !o.sigmoid)) return TL_BAD_SIZE;
     if (n_kv_heads % o.n_v_heads != 0 || (o.n_v_heads != n_kv_heads && v_pages == k_pages)) return TL_BAD_SIZE;
     if (!aligned16(q) || !aligned16(k_pages) || !aligned16(v_pages) || !aligned16(out)) return TL_BAD_ALIGN;
-    const Plan pl = make_plan(n_seqs, n_heads, n_kv_heads, max_q_len, max_kv_len, allow_split, window, o.keep_first);
+    // (a query sees no further back inside a chunk than behind a window of that size)
+    const Plan pl = make_plan(n_seqs, n_heads, n_kv_heads, max_q_len, max_kv_len, allow_split, window > 0 ? window : o.chunk, o.keep_first);
     if (pl.n_splits > 1 && workspace == nullptr) return TL_BAD_SIZE;
     if (n_seqs > 65535 || (long long)n_kv_heads * pl.n_gchunks > 65535) return TL_BAD_SIZE;
     if (smem_bytes(head_dim, o.v_head_dim) > 200 * 1024) return TL_TOO_LARGE;
@@ -444,6 +463,7 @@ extern "C" int tl_paged_attention_ex(const void* q, const void* k_pages, const v
     p.gate = o.gate; p.gate_mode = o.gate_mode;
     p.n_v_heads = o.n_v_heads; p.out_f32 = o.out_f32;
     p.v_stride = o.v_stride; p.softcap = o.softcap; p.sinks = o.sinks;
+    p.chunk = o.chunk; p.sigmoid = o.sigmoid; p.score_bias = o.score_bias;
     p.n_splits = pl.n_splits;
     p.scale = scale;
     p.part_o = workspace;
@@ -461,11 +481,11 @@ extern "C" int tl_paged_attention_ex(const void* q, const void* k_pages, const v
         const unsigned rows = (unsigned)n_tokens * n_heads;
         if (dtype == TL_F32)
             attention_merge_kernel<float><<<rows, threads, 0, s>>>(p.part_o, p.part_ml, (float*)out, pl.n_splits, o.v_head_dim,
-                                                                    (const float*)o.gate, o.gate_mode, o.out_f32, o.sinks, n_heads);
+                                                                    (const float*)o.gate, o.gate_mode, o.out_f32, o.sinks, n_heads, o.sigmoid);
         else
             attention_merge_kernel<__nv_bfloat16><<<rows, threads, 0, s>>>(p.part_o, p.part_ml, (__nv_bfloat16*)out, pl.n_splits,
                                                                             o.v_head_dim, (const __nv_bfloat16*)o.gate, o.gate_mode, o.out_f32,
-                                                                            o.sinks, n_heads);
+                                                                            o.sinks, n_heads, o.sigmoid);
         TL_LAUNCH_CHECK();
     }
     return TL_OK;

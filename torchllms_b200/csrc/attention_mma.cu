@@ -22,8 +22,9 @@
 // value (the value tile is the key tile), a window that keeps a request's first keys visible (they
 // are walked as tiles of their own ahead of the window's), a bias by bucketed distance added to the
 // scaled score, an output gate per head or per element, a cap on the scaled score (c * tanh(s / c)), a learned
-// sink per head in the softmax's denominator, and values that are the first coordinates of the stored keys; and
-// it multiplies probabilities as three bfloat16 terms, which add up to the float32 probability exactly.
+// sink per head in the softmax's denominator, values that are the first coordinates of the stored keys, chunks (a
+// query sees keys of its own run of so many positions), and (template flag SIG) sigmoid weights that are not divided
+// by their sum; and it multiplies probabilities as three bfloat16 terms, which add up to the float32 probability exactly.
 #include "common.cuh"
 #include <limits.h>
 #include <math.h>
@@ -71,6 +72,8 @@ struct MmaParams {
     float cap_log2;             // softcap * log2(e); 0: scores are not capped
     float scale_over_cap;       // scale / softcap
     const float* sinks;         // [n_heads] or null (natural-log scale, as stored)
+    int chunk;                  // 0: none
+    const float* score_bias;    // SIG: a key's weight is sigmoid(score + score_bias[head]), not normalised; [n_heads] or null
 };
 
 __device__ __forceinline__ unsigned smem_addr(const void* p) { return (unsigned)__cvta_generic_to_shared(p); }
@@ -104,7 +107,7 @@ __device__ __forceinline__ unsigned pack_bf16(float lo, float hi) {
     return *reinterpret_cast<unsigned*>(&v);
 }
 
-template <int HD, bool KEY_SPLIT, bool EXT>
+template <int HD, bool KEY_SPLIT, bool EXT, bool SIG>
 __global__ void __launch_bounds__(NT, KEY_SPLIT ? 4 : 2) attention_mma_kernel(const MmaParams p) {
     const int hd = EXT ? p.hd : HD, dv = EXT ? p.dv : HD;
     constexpr int PITCH = HD + 8;                 // bf16 elements per shared-memory row
@@ -165,7 +168,8 @@ __global__ void __launch_bounds__(NT, KEY_SPLIT ? 4 : 2) attention_mma_kernel(co
     // The window's keys start at win_lo; ahead of them, in tiles of their own, the kept first keys
     // that the window of the CTA's earliest query has passed (none unless EXT).  Tile i of the walk
     // starts at key tile_k0(i) and ends before tile_hi(i).
-    const int win_lo = p.window > 0 ? max(0, qpos_base + tok0 - p.window + 1) : 0;
+    const int win_lo = p.window > 0 ? max(0, qpos_base + tok0 - p.window + 1)
+                       : (EXT && p.chunk > 0) ? (qpos_base + tok0) / p.chunk * p.chunk : 0;
     const int win_hi = qpos_base + cta_tok_hi;                           // last query's position + 1
     const int n_kept = EXT ? min(p.keep_first, win_lo) : 0;
     const int kept_tiles = (n_kept + BN - 1) / BN;
@@ -192,6 +196,14 @@ __global__ void __launch_bounds__(NT, KEY_SPLIT ? 4 : 2) attention_mma_kernel(co
     const int warp_qmax = __reduce_max_sync(0xffffffffu, max(qpos[0], qpos[1]));
     // smallest position among the warp's real rows (rows without a query are never stored)
     const int warp_qmin = __reduce_min_sync(0xffffffffu, min(qpos[0] < 0 ? INT_MAX : qpos[0], qpos[1] < 0 ? INT_MAX : qpos[1]));
+
+    // the first key that the warp's last query sees: none of the warp's queries starts later
+    const int warp_lo = p.window > 0 ? warp_qmax - p.window + 1 : (EXT && p.chunk > 0 && warp_qmax > 0) ? warp_qmax / p.chunk * p.chunk : 0;
+    float sig_bias[2] = {0.f, 0.f};
+    if (SIG && p.score_bias != nullptr) {
+#pragma unroll
+        for (int i = 0; i < 2; ++i) sig_bias[i] = __ldg(p.score_bias + kvh * p.group + g0 + (g + 8 * i) % ng) * LOG2E;
+    }
 
     const int* table = p.block_table + (size_t)b * p.table_stride;
     // A thread always copies the same 16-byte column of a row: chunk c = tid + i * NT covers key
@@ -283,7 +295,7 @@ __global__ void __launch_bounds__(NT, KEY_SPLIT ? 4 : 2) attention_mma_kernel(co
             // ---- mask, streaming softmax (base 2; the scale is folded into the exponent)
             float mx[2] = {-INFINITY, -INFINITY};
             const int share_lo = k0 + key_off, share_hi = share_lo + 16 * KG;   // this warp's keys of the tile
-            const bool biased = EXT && p.rel != nullptr;
+            const bool biased = EXT && !SIG && p.rel != nullptr;
             const bool capped = EXT && p.cap_log2 > 0.f;        // (never together with a bias: the host sends those elsewhere)
             if (capped) {
                 // c * tanh(score * scale / c), on the base-2 scale; hidden keys are masked below as usual
@@ -293,8 +305,7 @@ __global__ void __launch_bounds__(NT, KEY_SPLIT ? 4 : 2) attention_mma_kernel(co
                     for (int e = 0; e < 4; ++e) s[nt][e] = p.cap_log2 * tanhf(s[nt][e] * p.scale_over_cap);
             }
             const float sl = (biased || capped) ? 1.f : p.scale_log2;       // biased and capped scores are on the base-2 scale already
-            const bool all_visible = share_hi <= k_hi && share_hi - 1 <= warp_qmin &&
-                                     (p.window <= 0 || share_lo > warp_qmax - p.window);
+            const bool all_visible = share_hi <= k_hi && share_hi - 1 <= warp_qmin && share_lo >= warp_lo;
             if (biased && all_visible && warp_qmax - share_lo < bias_cols) {
                 // every key of the share counts for every row and every distance is in the table
                 const float* brow[2] = {Bs + (g % ng) * bias_cols + (qpos[0] - share_lo - 2 * t),
@@ -336,6 +347,10 @@ __global__ void __launch_bounds__(NT, KEY_SPLIT ? 4 : 2) attention_mma_kernel(co
                     }
                 }
             } else if (!all_visible) {      // else every key counts for every row: no per-element tests
+                int row_lo[2];              // the first key of each row's window or chunk
+#pragma unroll
+                for (int i = 0; i < 2; ++i)
+                    row_lo[i] = p.window > 0 ? qpos[i] - p.window + 1 : (EXT && p.chunk > 0 && qpos[i] > 0) ? qpos[i] / p.chunk * p.chunk : 0;
 #pragma unroll
                 for (int nt = 0; nt < 2 * KG; ++nt) {
 #pragma unroll
@@ -343,11 +358,19 @@ __global__ void __launch_bounds__(NT, KEY_SPLIT ? 4 : 2) attention_mma_kernel(co
                         const int i = e >> 1;
                         const int kpos = share_lo + nt * 8 + 2 * t + (e & 1);
                         const bool ok = kpos <= qpos[i] && kpos < k_hi &&
-                                        (p.window <= 0 || kpos > qpos[i] - p.window || (EXT && kpos < p.keep_first));
+                                        (kpos >= row_lo[i] || (EXT && kpos < p.keep_first));
                         if (!ok) s[nt][e] = -INFINITY;
                     }
                 }
             }
+            if (SIG) {
+                // 1 / (1 + 2^-x) of the score with its bias on the base-2 scale; a hidden key's -inf gives 0.  Nothing is
+                // rescaled and no sum is kept
+#pragma unroll
+                for (int nt = 0; nt < 2 * KG; ++nt)
+#pragma unroll
+                    for (int e = 0; e < 4; ++e) s[nt][e] = __fdividef(1.f, 1.f + ex2(-fmaf(s[nt][e], sl, sig_bias[e >> 1])));
+            } else {
 #pragma unroll
             for (int nt = 0; nt < 2 * KG; ++nt)
 #pragma unroll
@@ -378,6 +401,7 @@ __global__ void __launch_bounds__(NT, KEY_SPLIT ? 4 : 2) attention_mma_kernel(co
                     o[i][0] *= alpha[0]; o[i][1] *= alpha[0];
                     o[i][2] *= alpha[1]; o[i][3] *= alpha[1];
                 }
+            }
             }
             // ---- accumulate probabilities times values.  A probability is split into two bfloat16
             // numbers (value and remainder) and multiplied twice, so the product keeps 16 bits of
@@ -440,7 +464,7 @@ __global__ void __launch_bounds__(NT, KEY_SPLIT ? 4 : 2) attention_mma_kernel(co
             const int head = kvh * p.group + g0 + rr % ng;
             const size_t row = (size_t)tok * p.n_heads + head;
             __nv_bfloat16* dst = p.out + row * dv;
-            if (EXT && p.sinks != nullptr) {
+            if (EXT && !SIG && p.sinks != nullptr) {
                 // one more term of the denominator, without a value: everything is rescaled to max(m, sink)
                 const float sink2 = p.sinks[head] * LOG2E;
                 const float M = fmaxf(m[i], sink2);
@@ -449,7 +473,7 @@ __global__ void __launch_bounds__(NT, KEY_SPLIT ? 4 : 2) attention_mma_kernel(co
 #pragma unroll
                 for (int nt = 0; nt < HD / 8; ++nt) { o[nt][2 * i] *= a; o[nt][2 * i + 1] *= a; }
             }
-            float inv = l[i] > 0.f ? 1.f / l[i] : 0.f;
+            float inv = SIG ? 1.f : l[i] > 0.f ? 1.f / l[i] : 0.f;
             if (EXT && p.gate_mode == 1) inv *= __bfloat162float(p.gate[row]);
 #pragma unroll
             for (int nt = 0; nt < HD / 8; ++nt) {
@@ -481,7 +505,7 @@ __global__ void __launch_bounds__(NT, KEY_SPLIT ? 4 : 2) attention_mma_kernel(co
             Om[(warp * 16 + rr) * HD + nt * 8 + 2 * t + 1] = o[nt][2 * i + 1];
         }
         if (t == 0) {
-            Mm[warp * 16 + rr] = m[i];
+            Mm[warp * 16 + rr] = SIG ? 0.f : m[i];      // (sigmoid weights have no maximum: partial results just add up)
             Lm[warp * 16 + rr] = l[i];
         }
     }
@@ -506,14 +530,14 @@ __global__ void __launch_bounds__(NT, KEY_SPLIT ? 4 : 2) attention_mma_kernel(co
         const size_t row = (size_t)tok * p.n_heads + head;
         if (EXT && d >= dv) continue;
         if (p.n_splits == 1) {
-            if (EXT && p.sinks != nullptr) {
+            if (EXT && !SIG && p.sinks != nullptr) {
                 const float sink2 = p.sinks[head] * LOG2E;
                 const float M2 = fmaxf(M, sink2);
                 const float f = exp2f(M - M2);          // M = -inf (no key seen) gives 0
                 num *= f;
                 den = den * f + exp2f(sink2 - M2);
             }
-            float v = den > 0.f ? num / den : 0.f;
+            float v = SIG ? num : den > 0.f ? num / den : 0.f;
             if (EXT && p.gate_mode == 1) v *= __bfloat162float(p.gate[row]);
             else if (EXT && p.gate_mode == 2) v *= __bfloat162float(p.gate[row * dv + d]);
             if (EXT && p.out_f32) reinterpret_cast<float*>(p.out)[row * dv + d] = v;
@@ -535,7 +559,7 @@ constexpr int MERGE_MAX_SPLITS = 256;
 __global__ void merge_partials_kernel(const float* __restrict__ part_o, const float* __restrict__ part_ml,
                                       __nv_bfloat16* __restrict__ out, int n_splits, int head_dim,
                                       const __nv_bfloat16* __restrict__ gate = nullptr, int gate_mode = 0, int out_f32 = 0,
-                                      const float* __restrict__ sinks = nullptr, int n_heads = 1) {
+                                      const float* __restrict__ sinks = nullptr, int n_heads = 1, int sigmoid = 0) {
     __shared__ float wgt[MERGE_MAX_SPLITS];
     __shared__ float red[2];
     const size_t row = blockIdx.x;
@@ -558,7 +582,7 @@ __global__ void merge_partials_kernel(const float* __restrict__ part_o, const fl
     }
     __syncthreads();
     const float den = red[0];
-    const float inv = den > 0.f ? 1.f / den : 0.f;
+    const float inv = sigmoid ? 1.f : den > 0.f ? 1.f / den : 0.f;
     for (int d = threadIdx.x; d < head_dim; d += blockDim.x) {
         float num = 0.f;
         for (int i = 0; i < n_splits; ++i) num = fmaf(wgt[i], part_o[(row * n_splits + i) * head_dim + d], num);
@@ -609,7 +633,7 @@ Plan make_plan(int n_seqs, int n_heads, int n_kv_heads, int max_q_len, int max_k
     return pl;
 }
 
-template <int HD, bool KEY_SPLIT, bool EXT = false>
+template <int HD, bool KEY_SPLIT, bool EXT = false, bool SIG = false>
 int launch(const MmaParams& p, dim3 grid, cudaStream_t s) {
     constexpr int PITCH = HD + 8;
     constexpr int QROWS = KEY_SPLIT ? 16 : 16 * NW;
@@ -617,7 +641,7 @@ int launch(const MmaParams& p, dim3 grid, cudaStream_t s) {
     if (EXT && !KEY_SPLIT && p.rel != nullptr) smem += (size_t)p.ng * p.bias_cols * sizeof(float);
     const size_t merge = KEY_SPLIT ? (size_t)(NW * 16 * (HD + 2)) * sizeof(float) : 0;
     if (merge > smem) smem = merge;
-    auto kern = attention_mma_kernel<HD, KEY_SPLIT, EXT>;
+    auto kern = attention_mma_kernel<HD, KEY_SPLIT, EXT, SIG>;
     static size_t raised = 48 * 1024;    // per instantiation: the largest limit set so far (one device per process)
     if (smem > raised) {
         cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
@@ -635,7 +659,8 @@ int launch_mode(const MmaParams& p, dim3 grid, bool key_split, cudaStream_t s) {
 }
 
 template <int HD>
-int launch_mode_ext(const MmaParams& p, dim3 grid, bool key_split, cudaStream_t s) {
+int launch_mode_ext(const MmaParams& p, dim3 grid, bool key_split, bool sigmoid, cudaStream_t s) {
+    if (sigmoid) return key_split ? launch<HD, true, true, true>(p, grid, s) : launch<HD, false, true, true>(p, grid, s);
     return key_split ? launch<HD, true, true>(p, grid, s) : launch<HD, false, true>(p, grid, s);
 }
 
@@ -693,6 +718,7 @@ extern "C" int tl_paged_attention_mma(const void* q, const void* k_pages, const 
     p.part_ml = workspace ? workspace + (size_t)n_tokens * n_heads * pl.n_splits * head_dim : nullptr;
     p.hd = p.dv = head_dim; p.shared_kv = 0; p.keep_first = 0; p.rel = nullptr; p.bucket = nullptr; p.n_bucket = 0; p.n_v_heads = n_kv_heads; p.out_f32 = 0;
     p.gate = nullptr; p.gate_mode = 0; p.bias_cols = 0; p.cap_log2 = 0.f; p.scale_over_cap = 0.f; p.sinks = nullptr;
+    p.chunk = 0; p.score_bias = nullptr;
 
     cudaStream_t s = (cudaStream_t)stream;
     dim3 grid(pl.n_q_tiles * pl.n_splits, n_kv_heads * pl.n_gchunks, n_seqs);
@@ -727,6 +753,9 @@ struct TlAttentionOptions {
     float softcap;          // c > 0: the scaled score s becomes c * tanh(s / c); not together with rel
     const float* sinks;     // [n_heads] or null: exp(sinks[h]) joins the softmax's denominator
     int v_stride;           // 0, or head_dim with v_pages == k_pages: a value is the first v_head_dim coordinates of a key
+    int chunk;              // 0: none; a query sees keys of its own run of so many positions; not together with a window
+    int sigmoid;            // 1: weights are sigmoid(score + score_bias[head]), not normalised; not together with sinks or rel
+    const float* score_bias;   // [n_heads] or null; sigmoid only
 };
 
 // 1 if the extended form takes keys of head_dim and values of v_head_dim elements, else 0.
@@ -764,10 +793,14 @@ extern "C" int tl_paged_attention_mma_ex(const void* q, const void* k_pages, con
     if (v_pages == k_pages && dv > head_dim) return TL_BAD_SIZE;
     if (o.v_stride != 0 && !(v_pages == k_pages && o.v_stride == head_dim)) return TL_BAD_SIZE;
     if (o.softcap < 0.f || (o.softcap > 0.f && o.rel != nullptr)) return TL_BAD_SIZE;
+    if (o.chunk < 0 || (o.chunk > 0 && (window > 0 || o.rel != nullptr)) || (o.sigmoid && (o.sinks != nullptr || o.rel != nullptr)) ||
+        (o.score_bias != nullptr && !o.sigmoid))
+        return TL_BAD_SIZE;
     const int n_v_heads = o.n_v_heads > 0 ? o.n_v_heads : n_kv_heads;
     if (n_kv_heads % n_v_heads != 0 || (n_v_heads != n_kv_heads && v_pages == k_pages)) return TL_BAD_SIZE;
     if (!aligned16(q) || !aligned16(k_pages) || !aligned16(v_pages) || !aligned16(out)) return TL_BAD_ALIGN;
-    const Plan pl = make_plan(n_seqs, n_heads, n_kv_heads, max_q_len, max_kv_len, allow_split, window, o.keep_first);
+    // (a query sees no further back inside a chunk than behind a window of that size)
+    const Plan pl = make_plan(n_seqs, n_heads, n_kv_heads, max_q_len, max_kv_len, allow_split, window > 0 ? window : o.chunk, o.keep_first);
     if (pl.n_splits > 1 && workspace == nullptr) return TL_BAD_SIZE;
     if (n_seqs > 65535 || (long long)n_kv_heads * pl.n_gchunks > 65535) return TL_BAD_SIZE;
 
@@ -792,6 +825,7 @@ extern "C" int tl_paged_attention_mma_ex(const void* q, const void* k_pages, con
     p.cap_log2 = o.softcap > 0.f ? o.softcap * LOG2E : 0.f;
     p.scale_over_cap = o.softcap > 0.f ? scale / o.softcap : 0.f;
     p.sinks = o.sinks;
+    p.chunk = o.chunk; p.score_bias = o.score_bias;
     // distances a row-split CTA meets inside its window (all of them when there is no window), as far as
     // 20 KB of shared memory hold them for the heads of a tile
     p.bias_cols = 0;
@@ -806,15 +840,15 @@ extern "C" int tl_paged_attention_mma_ex(const void* q, const void* k_pages, con
     dim3 grid(pl.n_q_tiles * pl.n_splits, n_kv_heads * pl.n_gchunks, n_seqs);
     int rc;
     switch (size) {
-        case 16: rc = launch_mode_ext<16>(p, grid, pl.key_split, s); break;
-        case 32: rc = launch_mode_ext<32>(p, grid, pl.key_split, s); break;
-        case 64: rc = launch_mode_ext<64>(p, grid, pl.key_split, s); break;
-        default: rc = launch_mode_ext<128>(p, grid, pl.key_split, s); break;
+        case 16: rc = launch_mode_ext<16>(p, grid, pl.key_split, o.sigmoid != 0, s); break;
+        case 32: rc = launch_mode_ext<32>(p, grid, pl.key_split, o.sigmoid != 0, s); break;
+        case 64: rc = launch_mode_ext<64>(p, grid, pl.key_split, o.sigmoid != 0, s); break;
+        default: rc = launch_mode_ext<128>(p, grid, pl.key_split, o.sigmoid != 0, s); break;
     }
     if (rc != TL_OK) return rc;
     if (pl.n_splits > 1) {
         merge_partials_kernel<<<dim3((unsigned)n_tokens * (unsigned)n_heads), dim3(dv >= 128 ? 128u : 64u), 0, s>>>(
-            p.part_o, p.part_ml, p.out, pl.n_splits, dv, p.gate, p.gate_mode, p.out_f32, p.sinks, n_heads);
+            p.part_o, p.part_ml, p.out, pl.n_splits, dv, p.gate, p.gate_mode, p.out_f32, p.sinks, n_heads, o.sigmoid);
         TL_LAUNCH_CHECK();
     }
     return TL_OK;

@@ -20,7 +20,7 @@
 
 namespace {
 
-enum : int { ACT_NONE = -1, ACT_SILU = 0, ACT_GELU_TANH = 1, ACT_RELU2 = 2, ACT_CLAMPED_SWISH = 3 };
+enum : int { ACT_NONE = -1, ACT_SILU = 0, ACT_GELU_TANH = 1, ACT_RELU2 = 2, ACT_CLAMPED_SWISH = 3, ACT_GELU = 4 };
 
 // the gated forms: act(gate) * up, or, clamped: g * sigmoid(alpha g) * (u + offset) with g = min(gate, limit), u = clamp(up, +-limit)
 struct GateParams { float limit, alpha, up_offset; };
@@ -29,6 +29,7 @@ __device__ __forceinline__ float act_apply(float x, int act) {
     if (act == ACT_NONE) return x;
     if (act == ACT_SILU) return x / (1.f + expf(-x));
     if (act == ACT_GELU_TANH) return 0.5f * x * (1.f + tanhf(0.7978845608028654f * (x + 0.044715f * x * x * x)));
+    if (act == ACT_GELU) return 0.5f * x * (1.f + erff(0.7071067811865476f * x));
     const float r = fmaxf(x, 0.f);
     return r * r;
 }
@@ -455,7 +456,7 @@ extern "C" int tl_moe_scale_act(const void* u, int in_dtype, int splits, long lo
                                 int top, int act, int gated, float limit, float alpha, float up_offset, float extra_limit,
                                 void* stream) {
     if (n_tokens <= 0) return TL_OK;
-    if (n_experts <= 0 || hidden <= 0 || extra < 0 || top <= 0 || top > 1024 || splits < 1 || act < -1 || act > 3) return TL_BAD_SIZE;
+    if (n_experts <= 0 || hidden <= 0 || extra < 0 || top <= 0 || top > 1024 || splits < 1 || act < -1 || act > 4) return TL_BAD_SIZE;
     if (act == ACT_CLAMPED_SWISH && !gated) return TL_BAD_SIZE;
     const GateParams gp = {limit, alpha, up_offset}, gp_extra = {extra_limit, alpha, up_offset};
     const size_t smem = (size_t)n_experts * sizeof(float);
@@ -535,12 +536,12 @@ extern "C" int tl_moe_plan(const int* chosen, int n_pairs, int n_experts, int* o
 // The experts' products over the sorted rows.  A: [rows][K]; with gather_div > 0 row r of the sorted order
 // reads A[order[r] / gather_div] (a token's row for each of its choices), else A[r].  W: expert e's [N][K]
 // matrix starts w_expert elements after expert e - 1's and its rows lie ldw elements apart;
-// C: [n_pairs][N] in sorted order.  act: -1 none, 0 silu, 1 gelu (tanh form), 2 squared relu.
+// C: [n_pairs][N] in sorted order.  act: -1 none, 0 silu, 1 gelu (tanh form), 2 squared relu, 4 gelu (exact).
 extern "C" int tl_moe_gemm(const void* A, const void* W, void* C, int dtype, const int* tiles, const int* order,
                            int gather_div, int n_pairs, int n_experts, int N, int K, int act, long long w_expert,
                            long long ldw, void* stream) {
     if (n_pairs <= 0 || N <= 0) return TL_OK;
-    if (K <= 0 || act < -1 || act > 2) return TL_BAD_SIZE;
+    if (K <= 0 || act < -1 || act > 4 || act == ACT_CLAMPED_SWISH) return TL_BAD_SIZE;
     const int max_tiles = tl_moe_max_tiles(n_pairs, n_experts);
     if (max_tiles > 65535) return TL_BAD_SIZE;
     const dim3 grid((N + BN - 1) / BN, max_tiles), block(NT);

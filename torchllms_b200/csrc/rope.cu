@@ -481,3 +481,275 @@ extern "C" int tl_rope_segment(const void* x, long long ldx, long long hsx, void
                               hsx, (__nv_bfloat16*)out, ldo, hso, positions, table, table_rows, total, n_heads, rot, interleaved);
     return TL_BAD_DTYPE;
 }
+
+// ---------------------------------------------------------------------------------------------
+// What follows the stacked projection [q heads | k heads | v heads | extra] of an attention mixer with norms
+// around its rotation (no v columns where values are the keys as projected):
+//
+//   x = row + bias;   q, k <- x / sqrt(mean over all heads' coordinates + eps) * w     (where q_norm / k_norm is given)
+//   the first rot coordinates of every q and k head rotated by the position
+//   q, k heads <- head / sqrt(mean(head^2) + eps)                                      (head_norm)
+//   v <- v columns, or the k columns of x (before norm and rotation); / its root mean square per head   (v_norm)
+//
+// k and v go to their pages, q and sigmoid(extra) leave as tensors; everything is float32 until it leaves.  A
+// rotation keeps a head's sum of squares, so the head norm's sum is taken on the way in.  A CTA per token with the
+// row in shared memory, a warp per head; without a norm over whole rows the heads of a token may be spread over CTAs.
+namespace {
+
+struct NormStoreParams {
+    const void* proj;          // [splits][T][width]
+    int splits;
+    long long plane;
+    const float* bias;         // [width] or null
+    const int* positions;
+    const float* table;        // [table_rows][rot / 2][2]
+    const int* slot_mapping;
+    const float* q_norm;       // [n_q * hd] or null
+    const float* k_norm;       // [n_k * hd] or null
+    void* q_out;               // [T][n_q][hd]
+    void* extra_out;           // [T][n_extra]
+    void* k_pages;             // [pages][n_k][page_size][hd]
+    void* v_pages;             // [pages][n_k][page_size][dv]
+    float eps;
+    int n_q, n_k, hd, dv, rot, n_extra, page_size, table_rows;
+    int interleaved, values_are_keys, head_norm, v_norm;
+    int heads_per_cta;
+};
+
+__device__ __forceinline__ float4 get4(const float* p) { return *reinterpret_cast<const float4*>(p); }
+__device__ __forceinline__ float4 get4(const __nv_bfloat16* p) {
+    const uint2 raw = *reinterpret_cast<const uint2*>(p);
+    const float2 a = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&raw.x));
+    const float2 b = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&raw.y));
+    return make_float4(a.x, a.y, b.x, b.y);
+}
+__device__ __forceinline__ void put4(float* p, float4 v) { *reinterpret_cast<float4*>(p) = v; }
+__device__ __forceinline__ void put4(__nv_bfloat16* p, float4 v) {
+    const __nv_bfloat162 a = __floats2bfloat162_rn(v.x, v.y), b = __floats2bfloat162_rn(v.z, v.w);
+    uint2 raw;
+    raw.x = *reinterpret_cast<const unsigned*>(&a);
+    raw.y = *reinterpret_cast<const unsigned*>(&b);
+    *reinterpret_cast<uint2*>(p) = raw;
+}
+__device__ __forceinline__ float4 scale4(float4 x, float s) { return make_float4(x.x * s, x.y * s, x.z * s, x.w * s); }
+__device__ __forceinline__ float4 mul4(float4 x, float4 y) { return make_float4(x.x * y.x, x.y * y.y, x.z * y.z, x.w * y.w); }
+__device__ __forceinline__ float dot4(float4 x) { return x.x * x.x + x.y * x.y + x.z * x.z + x.w * x.w; }
+
+// VEC: four columns at a time (head sizes, the rotated part and its half, and the extra columns' start are multiples of 4)
+template <typename TI, typename T, bool VEC>
+__global__ void norm_rope_store_kernel(const NormStoreParams p) {
+    extern __shared__ __align__(16) float row_s[];
+    __shared__ float part[2][33];
+    grid_launch_dependents();
+    const int t = blockIdx.x, lane = threadIdx.x & 31, warp = threadIdx.x >> 5, n_warps = blockDim.x >> 5;
+    const int qk = p.n_q + p.n_k, n_heads = qk + (p.values_are_keys ? 0 : p.n_k);
+    const int h_lo = blockIdx.y * p.heads_per_cta, h_hi = min(n_heads, h_lo + p.heads_per_cta);
+    auto head_col = [&](int h) { return h <= qk ? h * p.hd : qk * p.hd + (h - qk) * p.dv; };
+    const int c_lo = head_col(min(h_lo, n_heads)), c_hi = head_col(max(h_hi, h_lo));
+    const int width = head_col(n_heads) + p.n_extra;
+    const int nq_cols = p.n_q * p.hd, nqk_cols = qk * p.hd;
+    int pos = p.positions[t];
+    (void)TL_CHECK(pos >= 0 && pos < p.table_rows, TL_DBG_POSITION);
+    pos = pos < 0 ? 0 : (pos >= p.table_rows ? p.table_rows - 1 : pos);
+    const int half = p.rot >> 1;
+    const float* cs = p.table + (size_t)pos * p.rot;
+    const int sm = p.slot_mapping[t];
+    const int page = sm / p.page_size, slot = sm - page * p.page_size;
+    const bool write = TL_CHECK(sm >= 0, TL_DBG_SLOT) && tl_check_page(page);
+    grid_dependency_wait();
+    const TI* src = reinterpret_cast<const TI*>(p.proj) + (size_t)t * width;
+
+    // ---- this CTA's columns: planes summed, bias added
+    float ssq_q = 0.f, ssq_k = 0.f;
+    if (VEC) {
+        for (int c = c_lo + threadIdx.x * 4; c < c_hi; c += blockDim.x * 4) {
+            float4 x = get4(src + c);
+#pragma unroll 4
+            for (int s = 1; s < p.splits; ++s) {
+                const float4 y = get4(src + (size_t)s * p.plane + c);
+                x.x += y.x; x.y += y.y; x.z += y.z; x.w += y.w;
+            }
+            if (p.bias != nullptr) {
+                const float4 b = get4(p.bias + c);
+                x.x += b.x; x.y += b.y; x.z += b.z; x.w += b.w;
+            }
+            put4(row_s + (c - c_lo), x);
+            if (c < nq_cols) ssq_q += dot4(x);
+            else if (c < nqk_cols) ssq_k += dot4(x);
+        }
+    } else {
+        for (int c = c_lo + threadIdx.x; c < c_hi; c += blockDim.x) {
+            float x = to_float(src[c]);
+            for (int s = 1; s < p.splits; ++s) x += to_float(src[(size_t)s * p.plane + c]);
+            if (p.bias != nullptr) x += p.bias[c];
+            row_s[c - c_lo] = x;
+            if (c < nq_cols) ssq_q = fmaf(x, x, ssq_q);
+            else if (c < nqk_cols) ssq_k = fmaf(x, x, ssq_k);
+        }
+    }
+    float rq = 1.f, rk = 1.f;
+    if (p.q_norm != nullptr || p.k_norm != nullptr) {        // (one CTA has the whole row then)
+        ssq_q = warp_sum(ssq_q);
+        ssq_k = warp_sum(ssq_k);
+        if (lane == 0) { part[0][warp] = ssq_q; part[1][warp] = ssq_k; }
+        __syncthreads();
+        if (warp < 2) {
+            float v = lane < n_warps ? part[warp][lane] : 0.f;
+            v = warp_sum(v);
+            if (lane == 0) part[warp][32] = v;
+        }
+        __syncthreads();
+        rq = rsqrtf(part[0][32] / (float)nq_cols + p.eps);
+        rk = rsqrtf(part[1][32] / (float)(nqk_cols - nq_cols) + p.eps);
+    }
+    __syncthreads();
+
+    // ---- a warp per head
+    for (int h = h_lo + warp; h < h_hi; h += n_warps) {
+        const float* x = row_s + (head_col(h) - c_lo);
+        if (h < qk) {
+            const bool is_q = h < p.n_q;
+            const float* w = is_q ? p.q_norm : p.k_norm;
+            if (w != nullptr) w += (is_q ? h : h - p.n_q) * p.hd;
+            float sc = w == nullptr ? 1.f : (is_q ? rq : rk);
+            T* dst = is_q ? reinterpret_cast<T*>(p.q_out) + ((size_t)t * p.n_q + h) * p.hd
+                          : reinterpret_cast<T*>(p.k_pages) + (((size_t)page * p.n_k + (h - p.n_q)) * p.page_size + slot) * p.hd;
+            const bool put = is_q || write;
+            if (p.head_norm) {
+                float ssq = 0.f;
+                for (int d = lane; d < p.hd; d += 32) {
+                    const float v = x[d] * (w != nullptr ? sc * w[d] : 1.f);
+                    ssq = fmaf(v, v, ssq);
+                }
+                sc *= rsqrtf(warp_sum(ssq) / (float)p.hd + p.eps);
+            }
+            if (VEC) {
+                for (int i = lane * 4; i < p.hd - half; i += 128) {
+                    if (i >= half) {                                  // passes unrotated (or, interleaved, is the rest of the pairs)
+                        const int d = i + half;
+                        float4 v = scale4(get4(x + d), sc);
+                        if (w != nullptr) v = mul4(v, get4(w + d));
+                        if (put) put4(dst + d, v);
+                    } else if (!p.interleaved) {
+                        float4 u = scale4(get4(x + i), sc), v = scale4(get4(x + i + half), sc);
+                        if (w != nullptr) { u = mul4(u, get4(w + i)); v = mul4(v, get4(w + i + half)); }
+                        const float4 a = get4(cs + 2 * i), b = get4(cs + 2 * i + 4);      // (cos, sin) of pairs i, i + 1 and i + 2, i + 3
+                        const float4 u2 = make_float4(u.x * a.x - v.x * a.y, u.y * a.z - v.y * a.w, u.z * b.x - v.z * b.y, u.w * b.z - v.w * b.w);
+                        const float4 v2 = make_float4(v.x * a.x + u.x * a.y, v.y * a.z + u.y * a.w, v.z * b.x + u.z * b.y, v.w * b.z + u.w * b.w);
+                        if (put) { put4(dst + i, u2); put4(dst + i + half, v2); }
+                    } else {
+                        // four pairs are the eight coordinates from 2 i on
+                        float4 u = scale4(get4(x + 2 * i), sc), v = scale4(get4(x + 2 * i + 4), sc);
+                        if (w != nullptr) { u = mul4(u, get4(w + 2 * i)); v = mul4(v, get4(w + 2 * i + 4)); }
+                        const float4 a = get4(cs + 2 * i), b = get4(cs + 2 * i + 4);
+                        const float4 u2 = make_float4(u.x * a.x - u.y * a.y, u.y * a.x + u.x * a.y, u.z * a.z - u.w * a.w, u.w * a.z + u.z * a.w);
+                        const float4 v2 = make_float4(v.x * b.x - v.y * b.y, v.y * b.x + v.x * b.y, v.z * b.z - v.w * b.w, v.w * b.z + v.z * b.w);
+                        if (put) { put4(dst + 2 * i, u2); put4(dst + 2 * i + 4, v2); }
+                    }
+                }
+            } else {
+                for (int i = lane; i < p.hd - half; i += 32) {
+                    if (i >= half) {
+                        const int d = i + half;
+                        const float v = x[d] * sc * (w != nullptr ? w[d] : 1.f);
+                        if (put) dst[d] = from_float<T>(v);
+                    } else {
+                        const int l0 = p.interleaved ? 2 * i : i, l1 = p.interleaved ? 2 * i + 1 : i + half;
+                        const float u = x[l0] * sc * (w != nullptr ? w[l0] : 1.f), v = x[l1] * sc * (w != nullptr ? w[l1] : 1.f);
+                        const float c = cs[2 * i], s = cs[2 * i + 1];
+                        if (put) {
+                            dst[l0] = from_float<T>(u * c - v * s);
+                            dst[l1] = from_float<T>(v * c + u * s);
+                        }
+                    }
+                }
+            }
+            if (is_q || !p.values_are_keys) continue;
+        }
+        // ---- a value: a v head, or the key head just stored as it was projected
+        const int vh = p.values_are_keys ? h - p.n_q : h - qk;
+        float rv = 1.f;
+        if (p.v_norm) {
+            float ssq = 0.f;
+            for (int d = lane; d < p.dv; d += 32) ssq = fmaf(x[d], x[d], ssq);
+            rv = rsqrtf(warp_sum(ssq) / (float)p.dv + p.eps);
+        }
+        if (!write) continue;
+        T* dst = reinterpret_cast<T*>(p.v_pages) + (((size_t)page * p.n_k + vh) * p.page_size + slot) * p.dv;
+        if (VEC) {
+            for (int d = lane * 4; d < p.dv; d += 128) put4(dst + d, scale4(get4(x + d), rv));
+        } else {
+            for (int d = lane; d < p.dv; d += 32) dst[d] = from_float<T>(x[d] * rv);
+        }
+    }
+    // ---- gates that ride in the same projection
+    if (p.n_extra > 0 && blockIdx.y == gridDim.y - 1) {
+        const int e0 = width - p.n_extra;
+        for (int c = threadIdx.x; c < p.n_extra; c += blockDim.x) {
+            float x = p.bias != nullptr ? p.bias[e0 + c] : 0.f;
+            for (int s = 0; s < p.splits; ++s) x += to_float(src[(size_t)s * p.plane + e0 + c]);
+            reinterpret_cast<T*>(p.extra_out)[(size_t)t * p.n_extra + c] = from_float<T>(1.f / (1.f + expf(-x)));
+        }
+    }
+}
+
+}  // namespace
+
+// proj: [splits, n_tokens, width] of in_dtype, width = (n_q_heads + n_k_heads) * head_dim (+ n_k_heads * v_head_dim unless
+// values_are_keys, which wants v_head_dim == head_dim) + n_extra; bias float32 [width] or null; q_norm float32
+// [n_q_heads * head_dim] and k_norm [n_k_heads * head_dim], each or null; table float32 [table_rows, rot_dims / 2, 2];
+// q_out [n_tokens, n_q_heads, head_dim], extra_out [n_tokens, n_extra] and the pages in dtype.
+extern "C" int tl_norm_rope_store(const void* proj, int in_dtype, int splits, const float* bias, const int* positions, const float* table,
+                                  const int* slot_mapping, const float* q_norm, const float* k_norm, float eps, void* q_out,
+                                  void* extra_out, void* k_pages, void* v_pages, int dtype, int n_tokens, int n_q_heads, int n_k_heads,
+                                  int head_dim, int v_head_dim, int rot_dims, int n_extra, int page_size, int table_rows,
+                                  int interleaved, int values_are_keys, int head_norm, int v_norm, void* stream) {
+    if (n_tokens <= 0) return TL_OK;
+    if (head_dim <= 0 || v_head_dim <= 0 || n_q_heads <= 0 || n_k_heads <= 0 || n_extra < 0 || splits < 1 || rot_dims < 0 ||
+        (rot_dims & 1) || rot_dims > head_dim || page_size <= 0 || table_rows <= 0 || slot_mapping == nullptr ||
+        k_pages == nullptr || v_pages == nullptr || (values_are_keys && v_head_dim != head_dim) || (n_extra > 0 && extra_out == nullptr))
+        return TL_BAD_SIZE;
+    const int heads = n_q_heads + n_k_heads + (values_are_keys ? 0 : n_k_heads);
+    const int cols = (n_q_heads + n_k_heads) * head_dim + (values_are_keys ? 0 : n_k_heads * v_head_dim);
+    const int width = cols + n_extra;
+    NormStoreParams p = {};
+    p.proj = proj; p.splits = splits; p.plane = (long long)n_tokens * width; p.bias = bias; p.positions = positions; p.table = table;
+    p.slot_mapping = slot_mapping; p.q_norm = q_norm; p.k_norm = k_norm; p.q_out = q_out; p.extra_out = extra_out;
+    p.k_pages = k_pages; p.v_pages = v_pages; p.eps = eps; p.n_q = n_q_heads; p.n_k = n_k_heads; p.hd = head_dim; p.dv = v_head_dim;
+    p.rot = rot_dims; p.n_extra = n_extra; p.page_size = page_size; p.table_rows = table_rows; p.interleaved = interleaved;
+    p.values_are_keys = values_are_keys; p.head_norm = head_norm; p.v_norm = v_norm;
+    // few tokens (decoding) and no norm over whole rows: a token's heads are spread over CTAs
+    int per = heads;
+    if (n_tokens < 256 && q_norm == nullptr && k_norm == nullptr) {
+        per = heads < 4 ? heads : 4;
+        while ((heads + per - 1) / per > 16) ++per;
+    }
+    p.heads_per_cta = per;
+    const int by = (heads + per - 1) / per;
+    const int widest = head_dim > v_head_dim ? head_dim : v_head_dim;
+    const size_t smem = (size_t)(by == 1 ? cols : per * widest) * sizeof(float);
+    if (smem > 200 * 1024) return TL_TOO_LARGE;
+    const bool vec = head_dim % 4 == 0 && v_head_dim % 4 == 0 && rot_dims % 8 == 0 && width % 4 == 0 && aligned16(proj) && aligned16(bias) &&
+                     aligned16(table) && aligned16(q_norm) && aligned16(k_norm) && aligned16(q_out) && aligned16(k_pages) && aligned16(v_pages);
+    int threads = ((by == 1 ? cols : per * widest) / (vec ? 4 : 1) + 31) / 32 * 32;
+    const int most = n_tokens > 256 ? 256 : 1024;
+    threads = threads < 64 ? 64 : (threads > most ? most : threads);
+    cudaStream_t s = (cudaStream_t)stream;
+#define TL_NRS(TI, T, V)                                                                                                          \
+    do {                                                                                                                          \
+        static int raised = 0;                                                                                                    \
+        if (smem > 48 * 1024 && (int)smem > raised) {                                                                             \
+            cudaError_t e = cudaFuncSetAttribute(norm_rope_store_kernel<TI, T, V>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem); \
+            if (e != cudaSuccess) return (int)e;                                                                                  \
+            raised = (int)smem;                                                                                                   \
+        }                                                                                                                         \
+        return (int)tl_launch(norm_rope_store_kernel<TI, T, V>, dim3(n_tokens, by), dim3(threads), smem, s, p);                   \
+    } while (0)
+#define TL_NRS_PICK(TI, T) do { if (vec) TL_NRS(TI, T, true); else TL_NRS(TI, T, false); } while (0)
+    if (in_dtype == TL_F32 && dtype == TL_F32) TL_NRS_PICK(float, float);
+    if (in_dtype == TL_F32 && dtype == TL_BF16) TL_NRS_PICK(float, __nv_bfloat16);
+    if (in_dtype == TL_BF16 && dtype == TL_BF16) TL_NRS_PICK(__nv_bfloat16, __nv_bfloat16);
+#undef TL_NRS_PICK
+#undef TL_NRS
+    return TL_BAD_DTYPE;
+}

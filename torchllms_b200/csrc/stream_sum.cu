@@ -9,6 +9,12 @@
 //
 // stream_inject: h[t] += e[t] + r: a second stream and one row for all tokens (either may be absent), float32.
 //
+// stream_join:   out[t] = [h[t] + c * d | e[t]], the input of a product that makes the next stream from this one (its pending sum
+//                included) and another; the next stream starts as a row shared by all tokens.
+//
+// group_norm:    x = h[t] + c * d;  every one of `groups` equal runs of neighbouring columns is divided by its own
+//                sqrt(mean(x^2) + eps), the row is multiplied by w, and x replaces h[t] (c: a vector, or ones).
+//
 // sum_partials: the planes of a split-K product added up and rounded once (for readers that take no partial sums).
 //
 // Sums, norms and the stream are float32 whatever the terms' dtype.  Every term may arrive as float32 partial sums
@@ -152,6 +158,136 @@ __global__ void stream_inject_kernel(float* __restrict__ h, const float* __restr
     }
 }
 
+// VEC: four columns per thread and turn (columns and planes are multiples of 4)
+template <int VEC>
+struct Cols { float v[VEC]; };
+template <int VEC> __device__ __forceinline__ Cols<VEC> load_cols(const float* p) {
+    Cols<VEC> c;
+    if (VEC == 4) {
+        const float4 x = *reinterpret_cast<const float4*>(p);
+        c.v[0] = x.x; c.v[VEC > 1 ? 1 : 0] = x.y; c.v[VEC > 2 ? 2 : 0] = x.z; c.v[VEC > 3 ? 3 : 0] = x.w;
+    } else c.v[0] = *p;
+    return c;
+}
+template <int VEC> __device__ __forceinline__ Cols<VEC> load_cols(const __nv_bfloat16* p) {
+    Cols<VEC> c;
+    if (VEC == 4) {
+        const uint2 raw = *reinterpret_cast<const uint2*>(p);
+        const float2 a = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&raw.x));
+        const float2 b = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&raw.y));
+        c.v[0] = a.x; c.v[VEC > 1 ? 1 : 0] = a.y; c.v[VEC > 2 ? 2 : 0] = b.x; c.v[VEC > 3 ? 3 : 0] = b.y;
+    } else c.v[0] = __bfloat162float(*p);
+    return c;
+}
+template <int VEC> __device__ __forceinline__ void store_cols(float* p, const Cols<VEC>& c) {
+    if (VEC == 4) *reinterpret_cast<float4*>(p) = make_float4(c.v[0], c.v[VEC > 1 ? 1 : 0], c.v[VEC > 2 ? 2 : 0], c.v[VEC > 3 ? 3 : 0]);
+    else *p = c.v[0];
+}
+template <int VEC> __device__ __forceinline__ void store_cols(__nv_bfloat16* p, const Cols<VEC>& c) {
+    if (VEC == 4) {
+        const __nv_bfloat162 a = __floats2bfloat162_rn(c.v[0], c.v[VEC > 1 ? 1 : 0]), b = __floats2bfloat162_rn(c.v[VEC > 2 ? 2 : 0], c.v[VEC > 3 ? 3 : 0]);
+        uint2 raw;
+        raw.x = *reinterpret_cast<const unsigned*>(&a);
+        raw.y = *reinterpret_cast<const unsigned*>(&b);
+        *reinterpret_cast<uint2*>(p) = raw;
+    } else *p = __float2bfloat16_rn(c.v[0]);
+}
+
+// the stream with its pending sum: h + scale * (sum of delta's planes); delta and scale may be null
+template <int VEC, typename TD>
+__device__ __forceinline__ Cols<VEC> summed(const float* h, const TD* delta, int splits, long long plane, const float* scale, size_t at, int d) {
+    Cols<VEC> x = load_cols<VEC>(h + at);
+    if (delta != nullptr) {
+        Cols<VEC> y = load_cols<VEC>(delta + at);
+#pragma unroll 4
+        for (int s = 1; s < splits; ++s) {
+            const Cols<VEC> z = load_cols<VEC>(delta + (size_t)s * plane + at);
+#pragma unroll
+            for (int i = 0; i < VEC; ++i) y.v[i] += z.v[i];
+        }
+        if (scale != nullptr) {
+            const Cols<VEC> c = load_cols<VEC>(scale + d);
+#pragma unroll
+            for (int i = 0; i < VEC; ++i) y.v[i] *= c.v[i];
+        }
+#pragma unroll
+        for (int i = 0; i < VEC; ++i) x.v[i] += y.v[i];
+    }
+    return x;
+}
+
+template <int VEC, typename TD, typename TO>
+__global__ void stream_join_kernel(const float* __restrict__ h, const TD* __restrict__ delta, int splits, long long plane,
+                                   const float* __restrict__ scale, const float* __restrict__ rows, const float* __restrict__ row,
+                                   TO* __restrict__ out, float* __restrict__ h_next, long long n_chunks, int width) {
+    grid_launch_dependents();
+    grid_dependency_wait();
+    const int per_row = width / VEC;
+    for (long long i = (long long)blockIdx.x * blockDim.x + threadIdx.x; i < n_chunks; i += (long long)gridDim.x * blockDim.x) {
+        const long long t = i / per_row;
+        const int d = (int)(i - t * per_row) * VEC;
+        const size_t at = (size_t)t * width + d;
+        store_cols<VEC>(out + (size_t)t * 2 * width + d, summed<VEC>(h, delta, splits, plane, scale, at, d));
+        store_cols<VEC>(out + (size_t)t * 2 * width + width + d, load_cols<VEC>(rows + at));
+        Cols<VEC> r;
+#pragma unroll
+        for (int e = 0; e < VEC; ++e) r.v[e] = 0.f;
+        if (row != nullptr) r = load_cols<VEC>(row + d);
+        store_cols<VEC>(h_next + at, r);
+    }
+}
+
+// A CTA per row.  The warps form teams, one per group where there are warps enough, and a team walks its groups
+// (all teams the same number of times); a thread reads back only what it kept in shared memory itself.
+template <int VEC, typename TD, typename TO>
+__global__ void group_norm_kernel(float* __restrict__ h, const TD* __restrict__ delta, int splits, long long plane,
+                                  const float* __restrict__ scale, const float* __restrict__ weight, TO* __restrict__ out,
+                                  const int* __restrict__ pick, int dim, int groups, int teams, float eps, int write_back) {
+    extern __shared__ __align__(16) float row_buf[];
+    __shared__ float part[32];
+    grid_launch_dependents();
+    int r = pick != nullptr ? pick[blockIdx.x] : (int)blockIdx.x;
+    if (!tl_check_row(r)) r = 0;
+    grid_dependency_wait();
+    const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, n_warps = blockDim.x >> 5;
+    const int per_team = n_warps / teams, team = warp / per_team;
+    const int in_team = (warp - team * per_team) * 32 + lane, size = dim / groups;
+    const size_t base = (size_t)r * dim;
+    TO* o = out + (size_t)blockIdx.x * dim;
+    const int rounds = (groups + teams - 1) / teams;
+    for (int k = 0; k < rounds; ++k) {
+        const int g = k * teams + team;
+        const bool mine = team < teams && g < groups;
+        float ssq = 0.f;
+        if (mine) {
+            for (int c = in_team * VEC; c < size; c += per_team * 32 * VEC) {
+                const int d = g * size + c;
+                const Cols<VEC> x = summed<VEC>(h, delta, splits, plane, scale, base + d, d);
+                store_cols<VEC>(row_buf + d, x);
+                if (write_back) store_cols<VEC>(h + base + d, x);
+#pragma unroll
+                for (int i = 0; i < VEC; ++i) ssq = fmaf(x.v[i], x.v[i], ssq);
+            }
+        }
+        ssq = warp_sum(ssq);
+        if (k > 0) __syncthreads();            // part[] of the round before is read
+        if (lane == 0) part[warp] = ssq;
+        __syncthreads();
+        if (!mine) continue;
+        float total = 0.f;
+        for (int w = 0; w < per_team; ++w) total += part[team * per_team + w];
+        const float rs = rsqrtf(total / (float)size + eps);
+        for (int c = in_team * VEC; c < size; c += per_team * 32 * VEC) {
+            const int d = g * size + c;
+            Cols<VEC> x = load_cols<VEC>(row_buf + d);
+            const Cols<VEC> w = load_cols<VEC>(weight + d);
+#pragma unroll
+            for (int i = 0; i < VEC; ++i) x.v[i] *= rs * w.v[i];
+            store_cols<VEC>(o + d, x);
+        }
+    }
+}
+
 template <typename TO>
 __global__ void sum_partials_kernel(const float* __restrict__ parts, int splits, long long plane, TO* __restrict__ out, long long total) {
     grid_launch_dependents();
@@ -259,4 +395,71 @@ extern "C" int tl_stream_inject(float* h, const float* rows, const float* row, i
     long long blocks = (total + 255) / 256;
     if (blocks > 148 * 8) blocks = 148 * 8;
     return (int)tl_launch(stream_inject_kernel, dim3((unsigned)blocks), dim3(256), 0, (cudaStream_t)stream, h, rows, row, total, width);
+}
+
+// h: float32 [n_tokens][width] (left as it is); delta: [splits][n_tokens][width] of delta_dtype (float32 where splits > 1) or
+// null, planes `plane` elements apart; scale: float32 [width] or null; rows: float32 [n_tokens][width]; row: float32
+// [width] or null; out: [n_tokens][2 * width] of out_dtype; h_next: float32 [n_tokens][width], row (or zeros) in every token.
+extern "C" int tl_stream_join(const float* h, const void* delta, int delta_dtype, int splits, long long plane, const float* scale,
+                              const float* rows, const float* row, void* out, int out_dtype, float* h_next, int n_tokens, int width,
+                              void* stream) {
+    if (n_tokens <= 0) return TL_OK;
+    if (width <= 0 || splits < 1 || rows == nullptr || h_next == h || (splits > 1 && delta_dtype != TL_F32)) return TL_BAD_SIZE;
+    const bool vec = width % 4 == 0 && plane % 4 == 0 && aligned16(h) && aligned16(delta) && aligned16(scale) && aligned16(rows) &&
+                     aligned16(row) && aligned16(out) && aligned16(h_next);
+    const long long n_chunks = (long long)n_tokens * (vec ? width / 4 : width);
+    long long blocks = (n_chunks + 255) / 256;
+    if (blocks > 148 * 16) blocks = 148 * 16;
+    const dim3 grid((unsigned)blocks), block(256);
+    cudaStream_t s = (cudaStream_t)stream;
+#define TL_JOIN(TD, TO)                                                                                                            \
+    return (int)(vec ? tl_launch(stream_join_kernel<4, TD, TO>, grid, block, 0, s, h, (const TD*)delta, splits, plane, scale, rows, row, \
+                                 (TO*)out, h_next, n_chunks, width)                                                                \
+                     : tl_launch(stream_join_kernel<1, TD, TO>, grid, block, 0, s, h, (const TD*)delta, splits, plane, scale, rows, row, \
+                                 (TO*)out, h_next, n_chunks, width))
+    if (delta_dtype == TL_F32 && out_dtype == TL_F32) TL_JOIN(float, float);
+    if (delta_dtype == TL_F32 && out_dtype == TL_BF16) TL_JOIN(float, __nv_bfloat16);
+    if (delta_dtype == TL_BF16 && out_dtype == TL_BF16) TL_JOIN(__nv_bfloat16, __nv_bfloat16);
+    if (delta_dtype == TL_BF16 && out_dtype == TL_F32) TL_JOIN(__nv_bfloat16, float);
+#undef TL_JOIN
+    return TL_BAD_DTYPE;
+}
+
+// h: float32 [rows of the stream][dim], replaced by the sum where write_back; delta, scale as above (delta rows are h's); weight:
+// float32 [dim]; pick: int32 [n_out] rows of h, or null (row o is row o of h); out: [n_out][dim] of out_dtype.
+extern "C" int tl_group_norm(float* h, const void* delta, int delta_dtype, int splits, long long plane, const float* scale,
+                             const float* weight, void* out, int out_dtype, const int* pick, int n_out, int dim, int groups, float eps,
+                             int write_back, void* stream) {
+    if (n_out <= 0) return TL_OK;
+    if (dim <= 0 || groups <= 0 || dim % groups != 0 || splits < 1 || (splits > 1 && delta_dtype != TL_F32)) return TL_BAD_SIZE;
+    const size_t smem = (size_t)dim * sizeof(float);
+    if (smem > 200 * 1024) return TL_TOO_LARGE;
+    const bool vec = (dim / groups) % 4 == 0 && plane % 4 == 0 && aligned16(h) && aligned16(delta) && aligned16(scale) &&
+                     aligned16(weight) && aligned16(out);
+    int warps = (dim / (vec ? 4 : 1) + 31) / 32;
+    const int most = n_out >= 512 ? 8 : 32;              // many rows: smaller CTAs, more of them resident
+    warps = warps < 2 ? 2 : (warps > most ? most : warps);
+    const int teams = groups < warps ? groups : warps;
+    warps = warps / teams * teams;
+    const dim3 grid(n_out), block(warps * 32);
+    cudaStream_t s = (cudaStream_t)stream;
+#define TL_GN(V, TD, TO)                                                                                                          \
+    do {                                                                                                                          \
+        static int raised = 0;                                                                                                    \
+        if (smem > 48 * 1024 && (int)smem > raised) {                                                                             \
+            cudaError_t e = cudaFuncSetAttribute(group_norm_kernel<V, TD, TO>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem); \
+            if (e != cudaSuccess) return (int)e;                                                                                  \
+            raised = (int)smem;                                                                                                   \
+        }                                                                                                                         \
+        return (int)tl_launch(group_norm_kernel<V, TD, TO>, grid, block, smem, s, h, (const TD*)delta, splits, plane, scale, weight, \
+                              (TO*)out, pick, dim, groups, teams, eps, write_back);                                               \
+    } while (0)
+#define TL_GN_PICK(TD, TO) do { if (vec) TL_GN(4, TD, TO); else TL_GN(1, TD, TO); } while (0)
+    if (delta_dtype == TL_F32 && out_dtype == TL_F32) TL_GN_PICK(float, float);
+    if (delta_dtype == TL_F32 && out_dtype == TL_BF16) TL_GN_PICK(float, __nv_bfloat16);
+    if (delta_dtype == TL_BF16 && out_dtype == TL_BF16) TL_GN_PICK(__nv_bfloat16, __nv_bfloat16);
+    if (delta_dtype == TL_BF16 && out_dtype == TL_F32) TL_GN_PICK(__nv_bfloat16, float);
+#undef TL_GN_PICK
+#undef TL_GN
+    return TL_BAD_DTYPE;
 }

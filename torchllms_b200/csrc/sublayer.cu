@@ -577,11 +577,12 @@ extern "C" int tl_project_store(const void* proj, int in_dtype, int splits, long
 //                  o / sqrt(mean(o^2) + eps) * out_scale * gate[token, head]
 namespace {
 
-enum : int { ACT_SILU = 0, ACT_GELU_TANH = 1, ACT_RELU2 = 2 };
+enum : int { ACT_SILU = 0, ACT_GELU_TANH = 1, ACT_RELU2 = 2, ACT_GELU = 4 };      // (3 names a gated form of the experts' kernels)
 
 __device__ __forceinline__ float act_apply(float x, int act) {
     if (act == ACT_SILU) return x / (1.f + expf(-x));
     if (act == ACT_GELU_TANH) return 0.5f * x * (1.f + tanhf(0.7978845608028654f * (x + 0.044715f * x * x * x)));
+    if (act == ACT_GELU) return 0.5f * x * (1.f + erff(0.7071067811865476f * x));
     const float r = fmaxf(x, 0.f);
     return r * r;
 }
@@ -828,11 +829,11 @@ extern "C" int tl_depth_mix_norm(const float* levels, long long level_stride, co
 }
 
 // gated: in is [splits][n_tokens][2 * hidden] (gate columns first) and out = act(gate) * up; else in is
-// [splits][n_tokens][hidden] and out = act(in).  act: 0 silu, 1 gelu (tanh form), 2 squared relu.
+// [splits][n_tokens][hidden] and out = act(in).  act: 0 silu, 1 gelu (tanh form), 2 squared relu, 4 gelu (exact).
 extern "C" int tl_act(const void* in, int in_dtype, int splits, long long plane, void* out, int out_dtype, int n_tokens,
                       int hidden, int act, int gated, void* stream) {
     if ((long long)n_tokens * hidden <= 0) return TL_OK;
-    if (splits < 1 || act < 0 || act > 2) return TL_BAD_SIZE;
+    if (splits < 1 || act < 0 || act > 4 || act == 3) return TL_BAD_SIZE;
     cudaStream_t s = (cudaStream_t)stream;
     long long blocks = ((long long)n_tokens * hidden + 255) / 256;
     if (blocks > 148 * 16) blocks = 148 * 16;

@@ -232,10 +232,13 @@ class NativeOps:
 
     @_timed
     def rmsnorm(self, h: torch.Tensor, delta, weight: torch.Tensor, eps: float,
-                out_dtype: torch.dtype, rows: Optional[torch.Tensor] = None, deferred: bool = False):
+                out_dtype: torch.dtype, rows: Optional[torch.Tensor] = None, deferred: bool = False, groups: int = 1,
+               delta_scale: Optional[torch.Tensor] = None):
         """``delta`` may be a tensor, float32 partial sums ``[splits, T, dim]``, or a
         :class:`PendingProduct` (taken here the ordinary way).  ``deferred``: return the rows
-        weighted but not normalised, as a :class:`RowScaled` (not with ``rows``)."""
+        weighted but not normalised, as a :class:`RowScaled` (not with ``rows``).  ``groups``: the row is cut into so
+        many equal runs of neighbouring columns, each with a root mean square of its own; ``delta_scale`` (float32
+        ``[dim]``): the delta is multiplied by it, element by element, as it is added."""
         if isinstance(delta, PendingProduct):
             delta = delta.take(self)
         _cuda_contig(h, "residual stream", torch.float32)
@@ -259,6 +262,19 @@ class NativeOps:
             _cuda_contig(rows, "rows", torch.int32)
         n_out = h.shape[0] if rows is None else rows.numel()
         out = torch.empty((n_out, dim), dtype=out_dtype, device=h.device)
+        if groups > 1 or delta_scale is not None:
+            _need(not deferred and groups >= 1 and dim % groups == 0, f"a norm over {dim} columns cannot have {groups} groups, or be deferred with them")
+            if delta_scale is not None:
+                _cuda_contig(delta_scale, "delta scale", torch.float32)
+                _need(delta_scale.numel() == dim, "the delta's scale must match the stream's width")
+            self._debug_limit("stream_sum", 1, h.shape[0])
+            rc = self._lib("stream_sum").tl_group_norm(
+                _ptr(h), _ptr(delta), _DT[delta.dtype] if delta is not None else 0, splits, ctypes.c_longlong(plane), _ptr(delta_scale),
+                _ptr(weight), _ptr(out), _DT[out_dtype], _ptr(rows), n_out, dim, int(groups), ctypes.c_float(eps),
+                1 if (delta is not None and rows is None) else 0, _stream())
+            _check(rc, "group_norm")
+            self.launches += 1
+            return out
         ssq = torch.empty((n_out, 1), dtype=torch.float32, device=h.device) if deferred else None
         write_back = 1 if (delta is not None and rows is None) else 0
         self._debug_limit("elementwise", 1, h.shape[0])
@@ -555,6 +571,39 @@ class NativeOps:
         self.launches += 1
 
     @_timed
+    def stream_join(self, h: torch.Tensor, delta, delta_scale: Optional[torch.Tensor], rows: torch.Tensor, row: Optional[torch.Tensor], *,
+                    out_dtype: torch.dtype):
+        """The input of a product that makes a new stream from this one and another: ``[h + delta * delta_scale | rows]`` in
+        ``out_dtype`` (``delta`` a tensor, float32 partial sums, a :class:`PendingProduct` or ``None``; ``delta_scale`` float32
+        ``[dim]`` or ``None``; ``rows`` float32 ``[T, dim]``), and the stream that product is to be added to, which holds
+        ``row`` (float32 ``[dim]``, zeros without one) for every token.  ``h`` is left as it is."""
+        if isinstance(delta, PendingProduct):
+            delta = delta.take(self)
+        _cuda_contig(h, "residual stream", torch.float32)
+        _cuda_contig(rows, "joined stream", torch.float32)
+        _need(h.dim() == 2 and rows.shape == h.shape and out_dtype in _DT, "stream_join: two streams of one shape, float32 or bfloat16 out")
+        T, dim = h.shape
+        splits, plane = 1, 0
+        if delta is not None:
+            _cuda_contig(delta, "delta")
+            _need(delta.dtype in _DT and delta.shape[-2:] == h.shape and (delta.dim() == 2 or (delta.dim() == 3 and delta.dtype == torch.float32)),
+                  "the pending sum has the stream's shape, or is float32 partial sums of it")
+            if delta.dim() == 3:
+                splits, plane = delta.shape[0], delta.stride(0)
+        for t, name in ((delta_scale, "delta scale"), (row, "row of the new stream")):
+            if t is not None:
+                _cuda_contig(t, name, torch.float32)
+                _need(t.numel() == dim, f"the {name} must have the stream's width")
+        out = torch.empty((T, 2 * dim), dtype=out_dtype, device=h.device)
+        new = torch.empty_like(h)
+        rc = self._lib("stream_sum").tl_stream_join(
+            _ptr(h), _ptr(delta), _DT[delta.dtype] if delta is not None else 0, splits, ctypes.c_longlong(plane), _ptr(delta_scale),
+            _ptr(rows), _ptr(row), _ptr(out), _DT[out_dtype], _ptr(new), T, dim, _stream())
+        _check(rc, "stream_join")
+        self.launches += 1
+        return out, new
+
+    @_timed
     def selective_scan(self, x: torch.Tensor, dt: torch.Tensor, B: torch.Tensor, C: torch.Tensor, z: torch.Tensor, A: torch.Tensor,
                        D: torch.Tensor, dt_bias: torch.Tensor, state: torch.Tensor, q_start: torch.Tensor, state_slot: torch.Tensor,
                        fresh: torch.Tensor, *, n_seqs: int, max_q_len: int, out_dtype: torch.dtype) -> torch.Tensor:
@@ -587,7 +636,7 @@ class NativeOps:
         return out
 
     # ------------------------------------------- activations by name, depth average, map combination
-    _ACTS = {"silu": 0, "gelu_tanh": 1, "relu2": 2, "clamped_swish": 3}      # (the last one: gated forms of the experts' kernels only)
+    _ACTS = {"silu": 0, "gelu_tanh": 1, "relu2": 2, "clamped_swish": 3, "gelu": 4}      # (clamped_swish: gated forms of the experts' kernels only; gelu: the exact form)
 
     @_timed
     def depth_mix(self, history: torch.Tensor, coef: torch.Tensor, n: int, out: torch.Tensor,
@@ -640,7 +689,7 @@ class NativeOps:
 
     @_timed
     def activation(self, x: torch.Tensor, kind: str, out_dtype: Optional[torch.dtype] = None) -> torch.Tensor:
-        """``act(x)`` by name (``silu``, ``gelu_tanh``, ``relu2``: the square of relu), float32 arithmetic;
+        """``act(x)`` by name (``silu``, ``gelu_tanh``, ``gelu``: with erf, ``relu2``: the square of relu), float32 arithmetic;
         ``x`` is ``[tokens, width]`` or float32 partial sums of it."""
         return self._act(x, kind, out_dtype, False)
 
@@ -746,6 +795,54 @@ class NativeOps:
             _ptr(q), _ptr(extra), _ptr(k_pages), _ptr(v_pages), _DT[out_dtype], T, n_q_heads, n_k_heads, n_v_heads, head_dim,
             v_head_dim, rot_dims, n_extra, page_size, table.shape[0], 1 if interleaved else 0, _stream())
         _check(rc, "rope_store")
+        self.launches += 1
+        return q, extra
+
+    @_timed
+    def norm_rope_store(self, proj: torch.Tensor, positions: torch.Tensor, table: torch.Tensor, *, n_q_heads: int, n_k_heads: int,
+                        head_dim: int, v_head_dim: int, rot_dims: int, interleaved: bool, n_extra: int, k_pages: torch.Tensor,
+                        v_pages: torch.Tensor, slot_mapping: torch.Tensor, page_size: int, out_dtype: torch.dtype,
+                        bias: Optional[torch.Tensor] = None, values_are_keys: bool = False, q_norm: Optional[torch.Tensor] = None,
+                        k_norm: Optional[torch.Tensor] = None, qk_head_norm: bool = False, v_head_norm: bool = False, eps: float = 0.0):
+        """What :meth:`rope_store` does, with norms around the rotation: after the bias, q over all its heads at once and k
+        likewise are RMS-normed where a weight is given (``q_norm`` float32 ``[n_q_heads * head_dim]``, ``k_norm``); q and k are
+        rotated; with ``qk_head_norm`` every head of both is divided by its root mean square.  Rows are ``[q heads | k heads | v
+        heads | extra]``, as many v heads as k heads, or, with ``values_are_keys``, ``[q heads | k heads | extra]`` and a value
+        is the key as projected (bias included).  With ``v_head_norm`` every head's value is divided by its root mean square."""
+        _cuda_contig(proj, "projection")
+        _cuda_contig(positions, "positions", torch.int32)
+        _cuda_contig(table, "rotary table", torch.float32)
+        _cuda_contig(slot_mapping, "slot_mapping", torch.int32)
+        _cuda_contig(k_pages, "k_pages", out_dtype)
+        _cuda_contig(v_pages, "v_pages", out_dtype)
+        cols = (n_q_heads + n_k_heads) * head_dim + (0 if values_are_keys else n_k_heads * v_head_dim)
+        width = cols + n_extra
+        _need(proj.dim() in (2, 3) and proj.shape[-1] == width and proj.dtype in _DT, "projection rows must be [q | k | v | extra]")
+        splits = proj.shape[0] if proj.dim() == 3 else 1
+        _need(splits == 1 or proj.dtype == torch.float32, "partial sums must be float32")
+        _need(out_dtype in _DT and (out_dtype == proj.dtype or proj.dtype == torch.float32), "norm_rope_store cannot widen bfloat16 input")
+        _need(0 <= rot_dims <= head_dim and rot_dims % 2 == 0, "rot_dims must be even and at most head_dim")
+        _need(not values_are_keys or v_head_dim == head_dim, "values that are keys have the keys' size")
+        _need(table.dim() == 3 and table.shape[2] == 2 and (rot_dims == 0 or table.shape[1] == rot_dims // 2),
+              "rotary table must be [positions, rot_dims / 2, 2]")
+        _need(cols * 4 <= 200 * 1024, f"norm_rope_store keeps a row in shared memory: {cols} columns exceed 51200")
+        T = proj.shape[-2]
+        _need(positions.numel() == T and slot_mapping.numel() == T, "one position and one cache slot per token")
+        for t, n, name in ((bias, width, "bias"), (q_norm, n_q_heads * head_dim, "q_norm"), (k_norm, n_k_heads * head_dim, "k_norm")):
+            if t is not None:
+                _cuda_contig(t, name, torch.float32)
+                _need(t.numel() == n, f"{name} must have {n} elements")
+        _need(k_pages.shape[1:] == (n_k_heads, page_size, head_dim) and v_pages.shape[1:] == (n_k_heads, page_size, v_head_dim)
+              and v_pages.shape[0] == k_pages.shape[0], "pages must be [pages, heads, page_size, size] for keys and for values")
+        self._debug_limit("rope", 0, k_pages.shape[0])
+        q = torch.empty((T, n_q_heads, head_dim), dtype=out_dtype, device=proj.device)
+        extra = torch.empty((T, n_extra), dtype=out_dtype, device=proj.device) if n_extra else None
+        rc = self._lib("rope").tl_norm_rope_store(
+            _ptr(proj), _DT[proj.dtype], splits, _ptr(bias), _ptr(positions), _ptr(table), _ptr(slot_mapping), _ptr(q_norm), _ptr(k_norm),
+            ctypes.c_float(eps), _ptr(q), _ptr(extra), _ptr(k_pages), _ptr(v_pages), _DT[out_dtype], T, n_q_heads, n_k_heads, head_dim,
+            v_head_dim, rot_dims, n_extra, page_size, table.shape[0], 1 if interleaved else 0, 1 if values_are_keys else 0,
+            1 if qk_head_norm else 0, 1 if v_head_norm else 0, _stream())
+        _check(rc, "norm_rope_store")
         self.launches += 1
         return q, extra
 
@@ -1476,7 +1573,8 @@ class NativeOps:
                         distance_bias: Optional[torch.Tensor] = None, distance_buckets: Optional[torch.Tensor] = None,
                         gate: Optional[torch.Tensor] = None, n_v_heads: Optional[int] = None,
                         out_dtype: Optional[torch.dtype] = None, softcap: float = 0.0, sinks: Optional[torch.Tensor] = None,
-                        value_dim: Optional[int] = None) -> torch.Tensor:
+                        value_dim: Optional[int] = None, chunk: Optional[int] = None, weights: str = "softmax",
+                        score_bias: Optional[torch.Tensor] = None) -> torch.Tensor:
         """``impl``: ``"general"`` (CUDA cores, any supported size, both dtypes), ``"mma"`` (tensor
         cores, bfloat16, head_dim 16/32/64/128), ``"decode"`` (tensor cores fed by TMA, bfloat16,
         head_dim 64/128, steps whose requests bring one token or very few), ``"prefill"``
@@ -1501,15 +1599,17 @@ class NativeOps:
         leaves unrounded whatever q's dtype); ``softcap = c > 0`` (the scaled score ``s`` becomes ``c * tanh(s / c)``),
         ``sinks`` (float32 ``[H]``: ``exp(sinks[h])`` joins the softmax's denominator, a key without a value that is neither
         scaled nor capped) and ``value_dim`` (``v_pages`` is ``k_pages`` and a value is the first ``value_dim`` coordinates
-        of a stored key; the result is ``[T, H, value_dim]``)."""
+        of a stored key; the result is ``[T, H, value_dim]``); ``chunk`` (instead of a window: a query sees keys of its own run
+        of ``chunk`` positions, counted from the request's first token) and ``weights="sigmoid"`` (a visible key's weight is
+        ``sigmoid(score + score_bias[h])``, ``score_bias`` float32 ``[H]`` or ``None``, not divided by the weights' sum)."""
         if keep_first or distance_bias is not None or gate is not None or v_pages.shape[-1] != q.shape[-1] \
                 or q.shape[-1] % 16 != 0 or v_pages.shape[1] != k_pages.shape[1] or out_dtype not in (None, q.dtype) \
-                or softcap or sinks is not None or value_dim:
+                or softcap or sinks is not None or value_dim or chunk or weights != "softmax":
             _need(impl in ("auto", "general", "mma"), "only the general and the mma.sync attention kernels take these options")
             return self._paged_attention_general(q, k_pages, v_pages, block_table, q_start, kv_len, n_seqs, max_q_len,
                                                  max_kv_len, scale, window, page_size, allow_split, n_tokens, out,
                                                  keep_first, distance_bias, distance_buckets, gate, impl, n_v_heads, out_dtype,
-                                                 softcap, sinks, value_dim)
+                                                 softcap, sinks, value_dim, chunk, weights, score_bias)
         _cuda_contig(q, "q")
         _cuda_contig(k_pages, "k_pages", q.dtype)
         _cuda_contig(v_pages, "v_pages", q.dtype)
@@ -1601,13 +1701,15 @@ class NativeOps:
         _fields_ = [("v_head_dim", ctypes.c_int), ("keep_first", ctypes.c_int), ("rel", ctypes.c_void_p),
                     ("bucket", ctypes.c_void_p), ("n_bucket", ctypes.c_int), ("gate", ctypes.c_void_p),
                     ("gate_mode", ctypes.c_int), ("n_v_heads", ctypes.c_int), ("out_f32", ctypes.c_int),
-                    ("softcap", ctypes.c_float), ("sinks", ctypes.c_void_p), ("v_stride", ctypes.c_int)]
+                    ("softcap", ctypes.c_float), ("sinks", ctypes.c_void_p), ("v_stride", ctypes.c_int), ("chunk", ctypes.c_int),
+                    ("sigmoid", ctypes.c_int), ("score_bias", ctypes.c_void_p)]
 
     def _paged_attention_general(self, q, k_pages, v_pages, block_table, q_start, kv_len, n_seqs, max_q_len, max_kv_len,
                                  scale, window, page_size, allow_split, n_tokens, out, keep_first, distance_bias,
                                  distance_buckets, gate, impl: str = "general", n_v_heads: Optional[int] = None,
                                  out_dtype: Optional[torch.dtype] = None, softcap: float = 0.0,
-                                 sinks: Optional[torch.Tensor] = None, value_dim: Optional[int] = None) -> torch.Tensor:
+                                 sinks: Optional[torch.Tensor] = None, value_dim: Optional[int] = None, chunk: Optional[int] = None,
+                                 weights: str = "softmax", score_bias: Optional[torch.Tensor] = None) -> torch.Tensor:
         """The CUDA-core kernel with everything it can do (see :meth:`paged_attention`), or, with
         ``impl`` "auto" or "mma", in bfloat16 and for sizes it takes (keys and values multiples of 8
         up to 128), the extended form of the mma.sync kernel, which does the same."""
@@ -1646,7 +1748,15 @@ class NativeOps:
             _need(out.shape == (T_all, n_heads, v_dim), "out must be [tokens, heads, v_dim]")
         opt = self._AttentionOptions(v_dim, int(keep_first), None, None, 0, None, 0, v_heads,
                                      1 if (out_dtype == torch.float32 and q.dtype != torch.float32) else 0,
-                                     float(softcap or 0.0), None, v_stride)
+                                     float(softcap or 0.0), None, v_stride, int(chunk or 0), 1 if weights == "sigmoid" else 0, None)
+        _need(not (chunk and window) and (chunk is None or chunk > 0), "attention looks back through a window or inside chunks of at least one position")
+        _need(weights in ("softmax", "sigmoid") and not (weights == "sigmoid" and (sinks is not None or distance_bias is not None)),
+              "attention weights are 'softmax' or 'sigmoid'; sinks and a distance bias go with softmax")
+        if score_bias is not None:
+            _cuda_contig(score_bias, "score_bias", torch.float32)
+            _need(score_bias.numel() == n_heads and weights == "sigmoid", "score_bias: one number per query head, with sigmoid weights")
+            opt.score_bias = score_bias.data_ptr()
+        span = int(window or chunk or 0)          # how far back a query sees at most
         _need(opt.softcap >= 0.0, "softcap must not be negative")
         if sinks is not None:
             _cuda_contig(sinks, "sinks", torch.float32)
@@ -1667,12 +1777,12 @@ class NativeOps:
         n_splits, floats = ctypes.c_int(0), ctypes.c_longlong(0)
         mma_ok = (q.dtype == torch.bfloat16 and impl in ("auto", "mma") and self.use_mma_options
                   and self._lib("attention_mma").tl_attention_mma_ex_supports(head_dim, v_dim) == 1
-                  and not (softcap and distance_bias is not None))
+                  and not ((softcap or chunk) and distance_bias is not None))
         _need(impl != "mma" or mma_ok, "the mma.sync kernel takes bfloat16 and keys and values that are multiples of 8 up to 128")
         if mma_ok:
             lib = self._lib("attention_mma")
             rc = lib.tl_attention_mma_plan_ex(T, n_seqs, n_heads, n_kv_heads, head_dim, v_dim, max_q_len, max_kv_len,
-                                              int(window or 0), int(keep_first), 1 if allow_split else 0,
+                                              span, int(keep_first), 1 if allow_split else 0,
                                               ctypes.byref(n_splits), ctypes.byref(floats))
             _check(rc, "attention_mma_plan")
             ws = self._scratch(q.device, floats.value)
@@ -1687,7 +1797,7 @@ class NativeOps:
             return out
         lib = self._lib("attention")
         rc = lib.tl_attention_plan_ex(T, n_seqs, n_heads, n_kv_heads, head_dim, v_dim, max_q_len, max_kv_len,
-                                      int(window or 0), int(keep_first), 1 if allow_split else 0,
+                                      span, int(keep_first), 1 if allow_split else 0,
                                       ctypes.byref(n_splits), ctypes.byref(floats))
         _check(rc, "attention_plan")
         ws = self._scratch(q.device, floats.value)
