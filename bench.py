@@ -361,10 +361,40 @@ def _zusitar_config(z, vocab, max_len):
                          max_seq_len=max_len)
 
 
+# Lagusun at the same widths: window attention with sigmoid weights and chunked attention with a zero sink in turn, every
+# layer with experts, the middle layers run twice; beside it a Zusitar of the same shape whose layers are all capped
+# attention with sinks over (gated) experts, with the same loop
+LAGUSUN_SIZES = {name: dict(z, window=1024, chunk=1024, groups=4, keep_groups=2, norm_groups=4, loop=(1, 3, 2)) for name, z in RAKUVIK_SIZES.items()}
+
+
+def _lagusun_config(z, vocab, max_len):
+    from torchllms_b200.models.lagusun import AttentionConfig, BandScaling, LagusunConfig, LayerConfig, MlpConfig
+    hd = z["head_dim"]
+    common = dict(heads=z["heads"], kv_heads=z["kv_heads"], dim=hd, vdim=hd, scale=hd ** -0.5, rot_dims=z["rot_dims"], rot_base=500000.0)
+    win = AttentionConfig("attention_2", mask_size=z["window"], scaling=BandScaling(8.0, 1.0, 4.0, 8192.0), softcap=30.0, **common)
+    chunk = AttentionConfig("attention", mask_size=z["chunk"], **common)
+    moe = MlpConfig(z["expert_ff"], experts=z["experts"], top=z["top"], router_scale=2.0, shared_ff=z["shared_ff"])
+    return LagusunConfig("Lagusun", vocab, z["dim"], 1e-6, z["norm_groups"], 1.0,
+                         tuple(LayerConfig((win, chunk)[i % 2], moe) for i in range(z["layers"])),
+                         loop_start=z["loop"][0], loop_stop=z["loop"][1], loop_times=z["loop"][2], max_seq_len=max_len)
+
+
+def _looped_zusitar_config(z, vocab, max_len):
+    from torchllms_b200.models.zusitar import AttentionConfig, LayerConfig, MlpConfig, ZusitarConfig
+    hd = z["head_dim"]
+    att = AttentionConfig(heads=z["heads"], kv_heads=z["kv_heads"], dim=hd, vdim=hd, scale=hd ** -0.5, softcap=30.0, rot_dims=z["rot_dims"],
+                          rot_base=500000.0)
+    moe = MlpConfig("moe", z["expert_ff"], limit=7.0, experts=z["experts"], top=z["top"], router_scale=2.0, groups=z["groups"],
+                    keep_groups=z["keep_groups"], shared_ff=z["shared_ff"], shared_limit=7.0)
+    return ZusitarConfig("Zusitar", vocab, z["dim"], 1e-6, 1.0, tuple(LayerConfig(att, moe) for _ in range(z["layers"])),
+                         loop_start=z["loop"][0], loop_stop=z["loop"][1], loop_times=z["loop"][2], max_seq_len=max_len)
+
+
 # design -> (its name, the table of sizes, how its configuration is made, the model it stands beside)
 DESIGNS = {"nagolix": ("Nagolix", DESIGN_SIZES, _nagolix_config, "llama"), "rakuvik": ("Rakuvik", RAKUVIK_SIZES, _rakuvik_config, "llama"),
            "nunosun": ("Nunosun", NUNOSUN_SIZES, _nunosun_config, "rakuvik"),
-           "zusitar": ("Zusitar", ZUSITAR_SIZES, _zusitar_config, "rakuvik")}
+           "zusitar": ("Zusitar", ZUSITAR_SIZES, _zusitar_config, "rakuvik"),
+           "lagusun": ("Lagusun", LAGUSUN_SIZES, _lagusun_config, "zusitar")}
 
 
 def design_workload(args, peaks, design="nagolix"):
@@ -375,7 +405,8 @@ def design_workload(args, peaks, design="nagolix"):
     attention, attention, latent attention reading the first one's latents, attention; Rakuvik layers
     alternate minGRU with a dense feed-forward, differential attention with experts, minGRU with experts,
     differential attention reading the first one's keys and values with experts.  Nunosun and Zusitar stand beside
-    Rakuvik, the closest model (recurrent layers, attention, experts), at the same sizes."""
+    Rakuvik, the closest model (recurrent layers, attention, experts), at the same sizes; Lagusun beside a Zusitar
+    whose layers are all attention with experts, with the same loop."""
     import torch
     from torchllms_b200.engine.step import StepEntry
     from torchllms_b200.inference import LLM
@@ -391,8 +422,8 @@ def design_workload(args, peaks, design="nagolix"):
         hd = z["head_dim"]
         configs = {
             design: make_config(z, vocab, max_len),
-            "rakuvik": _rakuvik_config(z, vocab, max_len),
-        } if beside == "rakuvik" else {
+            beside: {"rakuvik": _rakuvik_config, "zusitar": _looped_zusitar_config}[beside](z, vocab, max_len),
+        } if beside != "llama" else {
             design: make_config(z, vocab, max_len),
             "llama": LlamaConfig(architecture="LlamaForCausalLM", n_layers=z["layers"], dim=z["dim"], n_heads=z["heads"],
                                  n_kv_heads=z["kv_heads"], head_dim=hd, ffn_hidden=z["ff"], vocab_size=vocab, norm_eps=1e-5,
@@ -472,10 +503,11 @@ def main():
     ap.add_argument("--layers", type=int, default=SHAPE_8B["n_layers"], help="fewer layers than the shape has (named in config)")
     ap.add_argument("--batch", type=int, default=8)
     ap.add_argument("--skip-points", action="store_true", help="only the headline batch and the prefill")
-    ap.add_argument("--workload", default="decode_8b", choices=["decode_8b", "design_nagolix", "design_rakuvik", "design_nunosun", "design_zusitar"] + sorted(SERVE),
+    ap.add_argument("--workload", default="decode_8b", choices=["decode_8b", "design_nagolix", "design_rakuvik", "design_nunosun", "design_zusitar", "design_lagusun"] + sorted(SERVE),
                     help="decode_8b: the headline (default); serve_1b, long_3b: whole serving runs through LLM.generate; "
                          "design_nagolix, design_rakuvik: that design beside the Llama decoder at equal sizes; "
-                         "design_nunosun, design_zusitar: that design beside Rakuvik at equal sizes")
+                         "design_nunosun, design_zusitar: that design beside Rakuvik at equal sizes; "
+                         "design_lagusun: Lagusun beside a Zusitar of attention layers")
     ap.add_argument("--context-len", type=int, default=PROMPT_LEN,
                     help="prompt length of the decode measurements (the headline is 2,048; the prefill figure stays at 2,048)")
     ap.add_argument("--long-contexts", type=lambda t: [int(x) for x in t.split(",") if x], default=[8192, 32768],
