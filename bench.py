@@ -457,7 +457,7 @@ def design_workload(args, peaks, design="nagolix"):
             handles = [engine.claim() for _ in range(batch)]
             for h in handles:
                 engine.step([StepEntry(h, torch.randint(0, vocab, (prompt_len,), generator=gen).tolist(), [])])
-            feed = torch.randint(0, vocab, (warmup + steps + 1, batch), generator=gen).tolist()
+            feed = torch.randint(0, vocab, (warmup + steps + 2, batch), generator=gen).tolist()
             for i in range(warmup):
                 engine.step([StepEntry(h, [t]) for h, t in zip(handles, feed[i])])
             torch.cuda.synchronize()
@@ -471,6 +471,7 @@ def design_workload(args, peaks, design="nagolix"):
             dec_ms = a.elapsed_time(b) / steps
             launches = ops.launches - launches0
             graphs, engine.use_graphs = engine.use_graphs, False          # the profile needs the calls themselves
+            engine.step([StepEntry(h, [t]) for h, t in zip(handles, feed[-2])])     # (once without: its allocations are not the profile's)
             with ops.profile() as dec_prof:
                 engine.step([StepEntry(h, [t]) for h, t in zip(handles, feed[-1])])
             engine.use_graphs = graphs
@@ -480,8 +481,8 @@ def design_workload(args, peaks, design="nagolix"):
             out[name][model] = {
                 "prefill_tokens_per_s": round(prompt_len / pre_ms * 1e3, 1), "prefill_ms": round(pre_ms, 3),
                 "decode_tokens_per_s": round(batch / dec_ms * 1e3, 1), "decode_ms_per_step": round(dec_ms, 4),
-                "weight_bytes": llm.model.weight_bytes(), "cache_bytes": engine.cache.bytes(),
-                "decode_weight_roofline_frac": round(llm.model.weight_bytes() / (dec_ms / 1e3) / (peaks["hbm_gbs"] * 1e9), 4),
+                "weight_bytes": llm.model.weight_bytes(), "step_weight_bytes": llm.model.step_weight_bytes(), "cache_bytes": engine.cache.bytes(),
+                "decode_weight_roofline_frac": round(llm.model.step_weight_bytes() / (dec_ms / 1e3) / (peaks["hbm_gbs"] * 1e9), 4),
                 "gpu_launches_per_decode_step": launches / steps,
                 "prefill_profile_ms": {k: [v[0], round(v[1], 3)] for k, v in sorted(pre_prof.items())},
                 "decode_profile_ms": {k: [v[0], round(v[1], 4)] for k, v in sorted(dec_prof.items())},

@@ -545,10 +545,13 @@ def test_router_with_a_correction(backend):
 @pytest.mark.parametrize("backend", BACKENDS)
 def test_exact_gelu(backend):
     ops, dev = _ops(backend)
-    x = torch.linspace(-6.0, 6.0, 1001)[None].repeat(2, 1).to(_dt(backend))
+    x = torch.linspace(-6.0, 6.0, 1000)[None].repeat(2, 1).to(_dt(backend))
     got = ops.activation(x.to(dev), "gelu").cpu().double()
-    tol = 1e-6 if _dt(backend) == torch.float32 else 1e-2
-    torch.testing.assert_close(got, plain.erf_gelu(x.to(F64)), atol=tol, rtol=tol)
+    want = plain.erf_gelu(x.to(F64))
+    if _dt(backend) == torch.float32:
+        torch.testing.assert_close(got, want, atol=1e-6, rtol=1e-6)
+    else:        # one rounding to bfloat16, also far out on the negative side (apart from an absolute 1e-6)
+        torch.testing.assert_close(got, want, atol=1e-6, rtol=2.0 ** -8)
 
 
 def test_frequencies_by_band():
@@ -616,7 +619,7 @@ def test_greedy_generation_through_the_scheduler(tmp_path, backend):
         kw = dict(ops=TorchOps())
     llm = LLM(folder, max_len=128, max_bsz=3, device=backend[0], precision=backend[1], page_size=page,
               max_num_batched_tokens=24, **kw)
-    prompts = [lc.tokens_for(cfg, n, seed=20 + n) for n in (3, 30, 11, 1)]
+    prompts = [lc.clear_tokens(cfg, tensors, n, seed=20 + n, dtype=backend[1]) for n in (3, 30, 11, 1)]
     results = llm.generate(prompt_token_ids=prompts, temperature=0.0, max_new_tokens=12, disable_tqdm=True)
     compared = 0
     for prompt, r in zip(prompts, results):
@@ -625,14 +628,17 @@ def test_greedy_generation_through_the_scheduler(tmp_path, backend):
             margins: list = []
             logits = plain.forward(cfg, tensors, seq, margins_out=margins)[-1]
             top = torch.topk(logits, 2).values
-            close = min((float(m.min()) for m in margins), default=1.0) < (1e-4 if backend[1] == "float32" else 0.02)
-            if close or float(top[0] - top[1]) < (1e-3 if backend[1] == "float32" else 0.1):
-                break                         # a near tie may fall either way: stop comparing this request
-            seq.append(int(torch.argmax(logits)))
-        made = seq[len(prompt):]
-        compared += len(made)
-        assert r.error is None and r.token_ids[:len(made)] == made
-    assert compared >= (30 if backend[1] == "float32" else 1)
+            if min((float(m.min()) for m in margins), default=1.0) < (1e-4 if backend[1] == "float32" else 0.01):
+                break                         # a close call in routing may fall either way: stop comparing this request
+            token, tie = r.token_ids[len(seq) - len(prompt)], 1e-3 if backend[1] == "float32" else 0.15
+            if float(top[0] - top[1]) < tie:  # and so may a near tie of the logits
+                assert float(top[0] - logits[token]) < tie
+            else:
+                assert token == int(torch.argmax(logits))
+                compared += 1
+            seq.append(token)
+        assert r.error is None and len(r.token_ids) == 12
+    assert compared >= (30 if backend[1] == "float32" else 4)
 
 
 def test_random_weights_mode_writes_a_folder_that_loads(tmp_path):

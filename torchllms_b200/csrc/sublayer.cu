@@ -587,6 +587,19 @@ __device__ __forceinline__ float act_apply(float x, int act) {
     return r * r;
 }
 
+// The exact gelu for results that are rounded to bfloat16: 0.5 x (1 + erf(x / sqrt 2)) with erfc by formula 7.1.26 of
+// Abramowitz and Stegun, Handbook of Mathematical Functions (absolute error of erf below 1.5e-7), a third of erff's
+// instructions.  With y = |x| / sqrt 2: erfc(y) = (a1 t + ... + a5 t^5) e^(-y^2), t = 1 / (1 + 0.3275911 y).
+__device__ __forceinline__ float gelu_for_bf16(float x) {
+    const float t = __fdividef(1.f, fmaf(0.3275911f * 0.7071067811865476f, fabsf(x), 1.f));
+    float p = fmaf(1.061405429f, t, -1.453152027f);
+    p = fmaf(p, t, 1.421413741f);
+    p = fmaf(p, t, -0.284496736f);
+    p = fmaf(p, t, 0.254829592f);
+    const float erfc_y = p * t * exp2f(x * x * -0.7213475204444817f);      // (log2(e) / 2)
+    return 0.5f * x * (x > 0.f ? 2.f - erfc_y : erfc_y);
+}
+
 // One CTA per row; the row is kept in shared memory between the passes.  VEC: four columns per thread and turn.
 template <typename TD, typename TO, bool VEC>
 __global__ void norm_add_norm_kernel(float* __restrict__ h, const TD* __restrict__ delta, int splits, long long plane, const float* __restrict__ bias,
@@ -714,24 +727,29 @@ __global__ void act_kernel(const TI* __restrict__ in, int splits, long long plan
 }
 
 // bfloat16 in and out, one plane, hidden a multiple of 8: eight values (and eight ups) per thread and turn
+template <int ACT, bool GATED>
 __global__ void act_bf16x8_kernel(const __nv_bfloat16* __restrict__ in, __nv_bfloat16* __restrict__ out, long long n_chunks,
-                                  int chunks_per_row, int act, int gated) {
+                                  int chunks_per_row) {
     grid_launch_dependents();
     grid_dependency_wait();
     for (long long i = (long long)blockIdx.x * blockDim.x + threadIdx.x; i < n_chunks; i += (long long)gridDim.x * blockDim.x) {
-        const long long t = i / chunks_per_row;
-        const int c = (int)(i - t * chunks_per_row);
-        const size_t hidden = (size_t)chunks_per_row * 8;
-        const __nv_bfloat16* g = in + (size_t)t * (gated ? 2 : 1) * hidden + (size_t)c * 8;
         Vec16<__nv_bfloat16> gv, uv, ov;
-        gv.load(g);
-        if (gated) uv.load(g + hidden);
+        if (GATED) {
+            const long long t = i / chunks_per_row;
+            const int c = (int)(i - t * chunks_per_row);
+            const size_t hidden = (size_t)chunks_per_row * 8;
+            const __nv_bfloat16* g = in + (size_t)t * 2 * hidden + (size_t)c * 8;
+            gv.load(g);
+            uv.load(g + hidden);
+        } else {
+            gv.load(in + (size_t)i * 8);
+        }
 #pragma unroll
         for (int e = 0; e < 8; ++e) {
-            const float a = act_apply(gv.get(e), act);
-            ov.set(e, gated ? a * uv.get(e) : a);
+            const float a = ACT == ACT_GELU ? gelu_for_bf16(gv.get(e)) : act_apply(gv.get(e), ACT);
+            ov.set(e, GATED ? a * uv.get(e) : a);
         }
-        ov.store(out + (size_t)t * hidden + (size_t)c * 8);
+        ov.store(out + (size_t)i * 8);
     }
 }
 
@@ -841,9 +859,17 @@ extern "C" int tl_act(const void* in, int in_dtype, int splits, long long plane,
     if (in_dtype == TL_BF16 && out_dtype == TL_BF16 && splits == 1 && hidden % 8 == 0 && aligned16(in) && aligned16(out)) {
         const long long n_chunks = (long long)n_tokens * (hidden / 8);
         long long b8 = (n_chunks + 255) / 256;
-        if (b8 > 148 * 16) b8 = 148 * 16;
-        return (int)tl_launch(act_bf16x8_kernel, dim3((unsigned)b8), block, 0, s, (const __nv_bfloat16*)in, (__nv_bfloat16*)out,
-                              n_chunks, hidden / 8, act, gated);
+        if (b8 > 148 * 64) b8 = 148 * 64;
+#define TL_ACT8(A)                                                                                                              \
+    return (int)(gated ? tl_launch(act_bf16x8_kernel<A, true>, dim3((unsigned)b8), block, 0, s, (const __nv_bfloat16*)in,       \
+                                   (__nv_bfloat16*)out, n_chunks, hidden / 8)                                                   \
+                       : tl_launch(act_bf16x8_kernel<A, false>, dim3((unsigned)b8), block, 0, s, (const __nv_bfloat16*)in,      \
+                                   (__nv_bfloat16*)out, n_chunks, hidden / 8))
+        if (act == ACT_SILU) TL_ACT8(ACT_SILU);
+        if (act == ACT_GELU_TANH) TL_ACT8(ACT_GELU_TANH);
+        if (act == ACT_GELU) TL_ACT8(ACT_GELU);
+        TL_ACT8(ACT_RELU2);
+#undef TL_ACT8
     }
     if (in_dtype == TL_F32 && out_dtype == TL_F32)
         return (int)tl_launch(act_kernel<float, float>, grid, block, 0, s, (const float*)in, splits, plane, (float*)out,

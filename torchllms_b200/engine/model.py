@@ -93,6 +93,18 @@ class Model:
             + self.head.numel() * self.head.element_size() \
             + sum(t.numel() * t.element_size() for t in self.join_tensors.values())
 
+    def step_weight_bytes(self) -> int:
+        """What a step streams from memory: as :meth:`weight_bytes`, with a layer or a joining matrix counted every time
+        it runs (a span of layers that runs several times in a row is more than a cache holds)."""
+        once = sum(blk.weight_bytes() for blk in self.blocks) + sum(t.numel() * t.element_size() for t in self.join_tensors.values())
+        runs = 0
+        for run in self.spec.run_order:
+            runs += self.blocks[run.layer].weight_bytes()
+            if run.join_embedding is not None:
+                t = self.join_tensors[run.join_embedding]
+                runs += t.numel() * t.element_size()
+        return self.weight_bytes() - once + runs
+
     # ------------------------------------------------------------------- cache
     def run_needs(self) -> List[Tuple[Optional[CacheNeed], Optional[StateNeed], Optional[int]]]:
         """What each run of the run order wants from the cache manager."""
