@@ -6,6 +6,8 @@
     python -m torchllms_b200.kernels.microbench elementwise --tokens 2048
     python -m torchllms_b200.kernels.microbench peaks
     python -m torchllms_b200.kernels.microbench selective_scan --tokens 2048 --channels 4096 --state 16
+    python -m torchllms_b200.kernels.microbench attention_options --length 2048 --span 1024
+    python -m torchllms_b200.kernels.microbench rows --tokens 2048
 
 Every case is timed with CUDA events after warm-up.  Memory-bound kernels run inside a CUDA
 graph over several copies of their operands (more than the 126 MB of L2 together), so that a
@@ -196,6 +198,85 @@ def selective_scan(args) -> None:
         print(f"selective_scan {label}, {C} channels x {N}: {us:8.1f} us  {moved / us / 1e3:7.1f} GB/s of inputs, outputs and state")
 
 
+def attention_options(args) -> None:
+    """Attention with options (16 heads over 4, 128 wide): one prompt of --length tokens and a decode step of 8 requests of that
+    length, over all keys, behind a window and inside chunks of --span, with softmax and with sigmoid weights."""
+    ops = get_ops()
+    H, G, d, page, dev, bf = 16, 4, 128, 16, "cuda", torch.bfloat16
+    sinks, bias = torch.zeros(H, device=dev), torch.randn(H, device=dev) - 4.0
+    kinds = (("softmax, cap, sinks", dict(softcap=30.0, sinks=sinks)), ("softmax, cap, sinks, window", dict(softcap=30.0, sinks=sinks, window=args.span)),
+             ("softmax, sinks, chunks", dict(sinks=sinks, chunk=args.span)),
+             ("sigmoid, cap, window", dict(softcap=30.0, weights="sigmoid", score_bias=bias, window=args.span)))
+    for label, lens, past in ((f"prompt of {args.length}", [args.length], 0), (f"decode step of 8 x {args.length}", [1] * 8, args.length - 1)):
+        T, B, kv = sum(lens), len(lens), past + max(lens)
+        blocks = -(-kv // page)
+        copies = max(1, min(16, (200 << 20) // (B * blocks * G * page * d * 4)))
+        pages = [[torch.randn(B * blocks, G, page, d, device=dev).to(bf) for _ in range(copies)] for _ in "kv"]
+        table = torch.arange(B * blocks, dtype=torch.int32, device=dev).view(B, blocks)
+        q = torch.randn(T, H, d, device=dev).to(bf)
+        q_start = torch.tensor([0] + list(torch.tensor(lens).cumsum(0)), dtype=torch.int32, device=dev)
+        kv_len = torch.full((B,), kv, dtype=torch.int32, device=dev)
+        for name, kw in kinds:
+            kw = dict({"window": None}, **kw)
+            us = _time(_graphed([(lambda i=i: ops.paged_attention(
+                q, pages[0][i], pages[1][i], table, q_start, kv_len, n_seqs=B, max_q_len=max(lens), max_kv_len=kv, scale=d ** -0.5,
+                page_size=page, **kw)) for i in range(copies)]), 5) / copies
+            seen = sum(min(p + 1, kw["window"]) if kw["window"] else p % kw["chunk"] + 1 if kw.get("chunk") else p + 1
+                       for n in lens for p in range(past, past + n))
+            span = kw["window"] or kw.get("chunk") or kv
+            print(f"{label}: {name}: {us:8.1f} us  {seen * H * d * 4 / us / 1e6:7.1f} TFLOP/s  "
+                  f"{B * min(kv, span) * G * d * 4 / us / 1e3:7.1f} GB/s of keys and values")
+
+
+def rows(args) -> None:
+    """What stands between a layer's products, at width 2,048 (16 heads over 4, 128 wide, 64 rotated): norms, stores, sums
+    and activations, over --tokens rows of bfloat16 and over 8 rows of four float32 partial sums."""
+    ops = get_ops()
+    H, G, d, D, page, dev, bf = 16, 4, 128, 2048, 16, "cuda", torch.bfloat16
+
+    def line(name: str, calls, moved: float) -> None:
+        us = _time(_graphed(calls), 5) / len(calls)
+        print(f"{name}: {us:7.1f} us  {moved / us / 1e3:7.1f} GB/s")
+
+    for T, splits, copies in ((args.tokens, 1, 4), (8, 4, 64)):
+        def data(width):
+            return [torch.randn(T, width, device=dev).to(bf) if splits == 1 else torch.randn(splits, T, width, device=dev) for _ in range(copies)]
+        in_bytes = 2 if splits == 1 else 4 * splits
+        positions = torch.arange(T, dtype=torch.int32, device=dev)
+        table = torch.randn(max(T, 64), 32, 2, device=dev)
+        kp = torch.zeros(-(-T // page), G, page, d, device=dev, dtype=bf)
+        vp = torch.zeros_like(kp)
+        store = dict(n_q_heads=H, n_k_heads=G, head_dim=d, v_head_dim=d, rot_dims=64, interleaved=False, n_extra=0, k_pages=kp, v_pages=vp,
+                     slot_mapping=positions, page_size=page, out_dtype=bf)
+        width = (H + 2 * G) * d
+        bias, qn, kn = torch.randn(width, device=dev), torch.randn(H * d, device=dev), torch.randn(G * d, device=dev)
+        qkv, qk = data(width), data((H + G) * d)
+        moved = T * (width * in_bytes + width * 2)
+        line(f"rope_store, {T} rows", [(lambda x=x: ops.rope_store(x, positions, table, n_v_heads=G, bias=bias, **store)) for x in qkv], moved)
+        line(f"norm_rope_store, heads normed, {T} rows",
+             [(lambda x=x: ops.norm_rope_store(x, positions, table, bias=bias, qk_head_norm=True, v_head_norm=True, eps=1e-6, **store)) for x in qkv], moved)
+        line(f"norm_rope_store, rows normed, values are keys, {T} rows",
+             [(lambda x=x: ops.norm_rope_store(x, positions, table, values_are_keys=True, q_norm=qn, k_norm=kn, eps=1e-6, **store)) for x in qk],
+             T * ((H + G) * d * in_bytes + width * 2))
+        hs, deltas = [torch.randn(T, D, device=dev) for _ in range(copies)], data(D)
+        w, ls = torch.randn(D, device=dev), torch.randn(D, device=dev)
+        moved = T * D * (10 + in_bytes)
+        line(f"rmsnorm of a sum, {T} rows", [(lambda i=i: ops.rmsnorm(hs[i], deltas[i], w, 1e-6, bf)) for i in range(copies)], moved)
+        line(f"rmsnorm of a scaled sum, 4 groups, {T} rows",
+             [(lambda i=i: ops.rmsnorm(hs[i], deltas[i], w, 1e-6, bf, groups=4, delta_scale=ls)) for i in range(copies)], moved)
+        line(f"norm_add and norm, {T} rows",
+             [(lambda i=i: ops.norm_add(hs[i], deltas[i], w, 1e-6, bf, then_weight=w, then_eps=1e-6)) for i in range(copies)], moved)
+        line(f"stream_join, {T} rows", [(lambda i=i: ops.stream_join(hs[i], deltas[i], ls, hs[(i + 1) % copies], w, out_dtype=bf)) for i in range(copies)],
+             T * D * (16 + in_bytes))
+        line(f"stream_inject, {T} rows", [(lambda i=i: ops.stream_inject(hs[i], hs[(i + 1) % copies], w)) for i in range(copies)], T * D * 12)
+    n = 4 * args.tokens
+    us = [torch.randn(n, D, device=dev).to(bf) for _ in range(4)]
+    for act in ("gelu", "gelu_tanh", "silu", "relu2"):
+        line(f"{act}, {n} rows", [(lambda u=u: ops.activation(u, act)) for u in us], n * D * 4)
+    gu = [torch.randn(n, 2 * D, device=dev).to(bf) for _ in range(2)]
+    line(f"clamped gate, {n} rows", [(lambda u=u: ops.glu(u, limit=7.0, alpha=1.702, up_offset=1.0)) for u in gu], n * D * 6)
+
+
 def main(argv=None) -> None:
     parser = argparse.ArgumentParser(description=__doc__, formatter_class=argparse.RawDescriptionHelpFormatter)
     sub = parser.add_subparsers(dest="case", required=True)
@@ -218,6 +299,13 @@ def main(argv=None) -> None:
     p.add_argument("--channels", type=int, default=4096)
     p.add_argument("--state", type=int, default=16)
     p.set_defaults(run=selective_scan)
+    p = sub.add_parser("attention_options")
+    p.add_argument("--length", type=int, default=2048)
+    p.add_argument("--span", type=int, default=1024)
+    p.set_defaults(run=attention_options)
+    p = sub.add_parser("rows")
+    p.add_argument("--tokens", type=int, default=2048)
+    p.set_defaults(run=rows)
     p = sub.add_parser("elementwise")
     p.add_argument("--tokens", type=int, default=2048)
     p.set_defaults(run=elementwise)
