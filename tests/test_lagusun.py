@@ -316,7 +316,7 @@ def test_every_mechanism_shows(tmp_path, backend, monkeypatch):
     """A model in which leaving out any one mechanism (the sink, a head's score bias, sigmoid in place of softmax, the
     norm's groups, the norms of q, k and v, the bands of the frequencies, the layer scales, the choice's correction, the
     exact gelu) moves the plain logits: the engine holds to the real ones, from a sequence's first token on."""
-    cfg = lc.config([lc.chunked(heads=3, kv_heads=1, dim=8, rot_dims=6, size=11, scale=1.0, mlp=moe_a),
+    cfg = lc.config([lc.chunked(heads=3, kv_heads=1, dim=8, rot_dims=6, size=11, scale=1.0, mlp=lc.moe(5, 2, 16, scale=2.0, shared=12)),
                      lc.windowed(heads=2, kv_heads=1, dim=8, vdim=12, rot_dims=8, base=200.0, size=14, softcap=2.0, scale=1.0, mlp=None)],
                     width=24, vocab=61, scale=4.0, groups=3)
     dtype = lc.stored_dtype(backend)
@@ -335,9 +335,6 @@ def test_every_mechanism_shows(tmp_path, backend, monkeypatch):
     want.check(lc.feed(rp, "p", tokens, [50]), "prompt")
     want.check(lc.feed(rp, "d", tokens, []), "token by token from the first")
     want.check(lc.feed(rp, "c", tokens, [1, 2, 3, 9]), "portions")
-
-
-moe_a = lc.moe(5, 2, 16, scale=2.0, shared=12)
 
 
 # ---------------------------------------------------------------- kernels against the plain functions

@@ -372,36 +372,36 @@ __global__ void __launch_bounds__(NT, KEY_SPLIT ? 4 : 2) attention_mma_kernel(co
                     for (int e = 0; e < 4; ++e) s[nt][e] = __fdividef(1.f, 1.f + ex2(-fmaf(s[nt][e], sl, sig_bias[e >> 1])));
             } else {
 #pragma unroll
-            for (int nt = 0; nt < 2 * KG; ++nt)
+                for (int nt = 0; nt < 2 * KG; ++nt)
 #pragma unroll
-                for (int e = 0; e < 4; ++e) mx[e >> 1] = fmaxf(mx[e >> 1], s[nt][e]);
-            float alpha[2], m_safe[2];
+                    for (int e = 0; e < 4; ++e) mx[e >> 1] = fmaxf(mx[e >> 1], s[nt][e]);
+                float alpha[2], m_safe[2];
 #pragma unroll
-            for (int i = 0; i < 2; ++i) {
-                mx[i] = fmaxf(mx[i], __shfl_xor_sync(0xffffffffu, mx[i], 1));
-                mx[i] = fmaxf(mx[i], __shfl_xor_sync(0xffffffffu, mx[i], 2));
-                const float m_new = fmaxf(m[i], mx[i] * sl);       // maxima live on the base-2 scale
-                m_safe[i] = (m_new == -INFINITY) ? 0.f : m_new;                // no key seen yet: keep exponents finite
-                alpha[i] = ex2(m[i] - m_safe[i]);
-                m[i] = m_new;
-                l[i] *= alpha[i];
-            }
-#pragma unroll
-            for (int nt = 0; nt < 2 * KG; ++nt) {
-#pragma unroll
-                for (int e = 0; e < 4; ++e) {
-                    const float pv = ex2(fmaf(s[nt][e], sl, -m_safe[e >> 1]));
-                    s[nt][e] = pv;
-                    l[e >> 1] += pv;
+                for (int i = 0; i < 2; ++i) {
+                    mx[i] = fmaxf(mx[i], __shfl_xor_sync(0xffffffffu, mx[i], 1));
+                    mx[i] = fmaxf(mx[i], __shfl_xor_sync(0xffffffffu, mx[i], 2));
+                    const float m_new = fmaxf(m[i], mx[i] * sl);       // maxima live on the base-2 scale
+                    m_safe[i] = (m_new == -INFINITY) ? 0.f : m_new;                // no key seen yet: keep exponents finite
+                    alpha[i] = ex2(m[i] - m_safe[i]);
+                    m[i] = m_new;
+                    l[i] *= alpha[i];
                 }
-            }
-            if (__any_sync(0xffffffffu, alpha[0] != 1.f || alpha[1] != 1.f)) {   // the maximum moved for some row
 #pragma unroll
-                for (int i = 0; i < HD / 8; ++i) {
-                    o[i][0] *= alpha[0]; o[i][1] *= alpha[0];
-                    o[i][2] *= alpha[1]; o[i][3] *= alpha[1];
+                for (int nt = 0; nt < 2 * KG; ++nt) {
+#pragma unroll
+                    for (int e = 0; e < 4; ++e) {
+                        const float pv = ex2(fmaf(s[nt][e], sl, -m_safe[e >> 1]));
+                        s[nt][e] = pv;
+                        l[e >> 1] += pv;
+                    }
                 }
-            }
+                if (__any_sync(0xffffffffu, alpha[0] != 1.f || alpha[1] != 1.f)) {   // the maximum moved for some row
+#pragma unroll
+                    for (int i = 0; i < HD / 8; ++i) {
+                        o[i][0] *= alpha[0]; o[i][1] *= alpha[0];
+                        o[i][2] *= alpha[1]; o[i][3] *= alpha[1];
+                    }
+                }
             }
             // ---- accumulate probabilities times values.  A probability is split into two bfloat16
             // numbers (value and remainder) and multiplied twice, so the product keeps 16 bits of
