@@ -63,6 +63,21 @@ class TorchOps:
             h = h + position_table[positions.long()].float()
         return h if rows_dtype is None else (h, self.stream_rows(h, rows_dtype))
 
+    def embed_pairs(self, token_ids, table, pair_rows, last, seq_of_token, q_start, state_slot, fresh, *, mul_prev, mul_cur):
+        """table[token] + pair_rows[(previous * mul_prev + token * mul_cur) mod (rows - 1)], the last row where a request has no
+        token before; last (int32 [slots, 1]) holds every request's last token: read and left updated."""
+        buckets = pair_rows.shape[0] - 1
+        ids, rows = token_ids.tolist(), []
+        for b in range(q_start.numel() - 1):
+            slot, lo, hi = int(state_slot[b]), int(q_start[b]), int(q_start[b + 1])
+            before = None if int(fresh[b]) else int(last[slot, 0])
+            for t in range(lo, hi):
+                rows.append(buckets if before is None else (before * mul_prev + ids[t] * mul_cur) % buckets)
+                before = ids[t]
+            if hi > lo:
+                last[slot, 0] = before
+        return table[token_ids.long()].float() + pair_rows[torch.tensor(rows, device=table.device)].float()
+
     def stream_rows(self, h, dtype):
         return h if dtype == torch.float32 else h.to(dtype)
 
@@ -167,6 +182,37 @@ class TorchOps:
             k_pages[page, :, slot] = turn(k, n_k_heads).to(k_pages.dtype)
             v_pages[page, :, slot] = v.reshape(T, n_v_heads, v_head_dim).to(v_pages.dtype)
         return q.to(out_dtype).contiguous(), (torch.sigmoid(e).to(out_dtype).contiguous() if n_extra else None)
+
+    def conv_rope_store(self, proj, w_conv, state, positions, table, q_start, state_slot, fresh, *, n_seqs, max_q_len, n_q_heads,
+                        n_k_heads, head_dim, v_head_dim, rot_dims, n_extra, k_pages, v_pages, slot_mapping, page_size, out_dtype,
+                        extra_scale=1.0):
+        """A row of proj is [q heads | k heads | v heads | extra]: a short convolution over the q, k and v columns, then
+        what rope_store does in the half pairing; sigmoid(extra) * extra_scale."""
+        x = proj.float().sum(0) if proj.dim() == 3 else proj.float()
+        nc = w_conv.shape[0]
+        y = self.short_conv(x[:, :nc], w_conv, state, q_start, state_slot, fresh, n_seqs=n_seqs, max_q_len=max_q_len, activation=None,
+                            residual=False, out_dtype=torch.float32)
+        q, gate = self.rope_store(torch.cat([y, x[:, nc:]], dim=1), positions, table, n_q_heads=n_q_heads, n_k_heads=n_k_heads,
+                                  n_v_heads=n_k_heads, head_dim=head_dim, v_head_dim=v_head_dim, rot_dims=rot_dims, interleaved=False,
+                                  n_extra=n_extra, k_pages=k_pages, v_pages=v_pages, slot_mapping=slot_mapping, page_size=page_size,
+                                  out_dtype=torch.float32)
+        return q.to(out_dtype), (None if gate is None else (gate * np.float32(extra_scale)).to(out_dtype))
+
+    def delta_prep(self, proj, w_conv, state, q_start, state_slot, fresh, *, n_seqs, max_q_len, n_qk_heads, head_dim, n_v, n_small,
+                   n_low, low_pad, q_scale, unit_eps, out_dtype):
+        """A row of proj is [q | k | v | small | low | rest]: a short convolution and silu on q, k and v, q (times q_scale) and k as
+        unit vectors per head in float32, v, the small columns, and the low ones padded with zeros."""
+        x = proj.float().sum(0) if proj.dim() == 3 else proj.float()
+        nc, n = w_conv.shape[0], n_qk_heads * head_dim
+        c = self.short_conv(x[:, :nc], w_conv, state, q_start, state_slot, fresh, n_seqs=n_seqs, max_q_len=max_q_len, activation="silu",
+                            residual=False, out_dtype=torch.float32)
+        unit = dict(n_heads=n_qk_heads, head_dim=head_dim, unit_eps=unit_eps)
+        low = None
+        if n_low:
+            low = torch.zeros((x.shape[0], low_pad), dtype=out_dtype, device=x.device)
+            low[:, :n_low] = x[:, nc + n_small:nc + n_small + n_low].to(out_dtype)
+        return (self.recurrence_prep(c[:, :n], scale=q_scale, **unit), self.recurrence_prep(c[:, n:2 * n], scale=1.0, **unit),
+                c[:, 2 * n:].to(out_dtype), x[:, nc:nc + n_small].to(out_dtype), low)
 
     def norm_rope_store(self, proj, positions, table, *, n_q_heads, n_k_heads, head_dim, v_head_dim, rot_dims, interleaved, n_extra,
                         k_pages, v_pages, slot_mapping, page_size, out_dtype, bias=None, values_are_keys=False, q_norm=None,
@@ -401,7 +447,8 @@ class TorchOps:
         vh = v.float().reshape(T, H, dv)
         if decay is None:
             beta = torch.sigmoid(beta_logits.float())
-            g = torch.exp(-decay_rate * torch.nn.functional.softplus(decay_logits.float() + decay_bias))
+            soft = torch.nn.functional.softplus(decay_logits.float() + decay_bias).view(T, H, -1)      # a decay per head, or per channel
+            g = torch.exp(-decay_rate[:, None] * soft)
         out = torch.empty((T, H, dv), dtype=torch.float32, device=q.device)
         qs = q_start.tolist()
         for b in range(n_seqs):
@@ -413,21 +460,23 @@ class TorchOps:
                 if decay is not None:
                     S = decay[:, None, None] * S + kt[:, :, None] * vh[t][:, None, :]
                 else:
-                    S = g[t][:, None, None] * S
+                    S = g[t][:, :, None] * S
                     u = beta[t][:, None] * (vh[t] - torch.einsum("hkv,hk->hv", S, kt))
                     S = S + kt[:, :, None] * u[:, None, :]
                 out[t] = torch.einsum("hkv,hk->hv", S, qt)
             state[slot] = S.transpose(1, 2)
         return out.flatten(1)
 
-    def head_norm_gate(self, o, gate, weight, eps, *, head_dim, out_dtype):
-        """Every head of o (float32 [T, H * head_dim]) divided by its root mean square, times the weight (if any), times silu(gate)."""
+    def head_norm_gate(self, o, gate, weight, eps, *, head_dim, out_dtype, activation="silu", out=None):
+        """Every head of o (float32 [T, H * head_dim]) divided by its root mean square, times the weight (if any), times
+        silu(gate) or sigmoid(gate)."""
         y = o.float().unflatten(1, (-1, head_dim))
         y = y * torch.rsqrt(y.pow(2).mean(-1, keepdim=True) + eps)
         if weight is not None:
             y = y * weight
         g = gate.float()
-        return (y.flatten(1) * g * torch.sigmoid(g)).to(out_dtype)
+        y = (y.flatten(1) * (g * torch.sigmoid(g) if activation == "silu" else torch.sigmoid(g))).to(out_dtype)
+        return y if out is None else out.copy_(y)
 
     def side_gate(self, u, token_ids, table, out_dtype):
         """gelu_tanh(u) * table[token]."""
@@ -611,10 +660,11 @@ class TorchOps:
         if keep_first or distance_bias is not None or gate is not None or v_pages.shape[3] != hd \
                 or v_pages.shape[1] != KV or out_dtype not in (None, q.dtype) or softcap or sinks is not None or value_dim \
                 or chunk or weights != "softmax":
-            assert out is None and n_tokens is None and (n_v_heads or KV) == v_pages.shape[1]
-            return self._attention_general(q, k_pages, v_pages, block_table, q_start, kv_len, n_seqs, scale, window,
+            assert n_tokens is None and (n_v_heads or KV) == v_pages.shape[1]
+            o = self._attention_general(q, k_pages, v_pages, block_table, q_start, kv_len, n_seqs, scale, window,
                                            page_size, keep_first, distance_bias, distance_buckets, gate, out_dtype,
                                            softcap, sinks, value_dim, chunk, weights, score_bias)
+            return o if out is None else out.copy_(o)
         # the same contract as the kernels' front end: the step's bounds cover its requests and fit the table
         assert block_table.shape[1] * page_size >= max_kv_len, "block_table is too narrow for max_kv_len"
         assert int(kv_len[:n_seqs].max()) <= max_kv_len and n_seqs <= block_table.shape[0]

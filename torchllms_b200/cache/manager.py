@@ -137,12 +137,13 @@ class CacheManager:
     ``run_needs[i]`` is ``(cache_need, state_need, cache_of)`` of run ``i`` in
     the model's run order; a run with ``cache_of = j`` owns no pages and reads
     run ``j``'s.  ``pool_tokens`` is how many tokens all live requests may hold
-    together (each request's count rounded up to whole pages).
+    together (each request's count rounded up to whole pages).  ``model_state`` is
+    per-request state that no single run owns (:attr:`model_state`, ``[slots, ...]``).
     """
 
     def __init__(self, run_needs: Sequence[Tuple[Optional[CacheNeed], Optional[StateNeed], Optional[int]]],
                  *, page_size: int, pool_tokens: int, max_num_seqs: int, max_len: int,
-                 dtype: torch.dtype, device, max_step_tokens: Optional[int] = None):
+                 dtype: torch.dtype, device, max_step_tokens: Optional[int] = None, model_state: Optional[StateNeed] = None):
         if page_size <= 0 or pool_tokens <= 0 or max_num_seqs <= 0 or max_len <= 0:
             raise ValueError("page_size, pool_tokens, max_num_seqs and max_len must be positive")
         self.page_size = int(page_size)
@@ -200,6 +201,11 @@ class CacheManager:
                 self.state.append(torch.zeros((self.max_num_seqs, *state.shape), dtype=state.dtype,
                                               device=self.device))
 
+        # ---- state rows of the model itself (what no single run owns)
+        self.model_state: Optional[torch.Tensor] = None
+        if model_state is not None:
+            self.model_state = torch.zeros((self.max_num_seqs, *model_state.shape), dtype=model_state.dtype, device=self.device)
+
         # ---- requests
         self._free_slots: List[int] = list(range(self.max_num_seqs - 1, -1, -1))
         self._requests: Dict[int, _Request] = {}
@@ -251,7 +257,7 @@ class CacheManager:
         handle = self._next_handle
         self._next_handle += 1
         self._requests[handle] = _Request(handle, slot, 0, [[] for _ in self.groups], [0 for _ in self.groups])
-        for s in self.state:
+        for s in self.state + [self.model_state]:
             if s is not None:
                 s[slot].zero_()
         return handle

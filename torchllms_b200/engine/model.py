@@ -40,6 +40,10 @@ class Model:
         self.graph_safe = self.final_norm.graph_safe and all(b.graph_safe for b in self.blocks)
         self.embedding: Optional[torch.Tensor] = None
         self.position_table: Optional[torch.Tensor] = None
+        self.pair_rows: Optional[torch.Tensor] = None
+        if spec.pair_table is not None and (spec.position_tensor is not None or spec.keeps_history or spec.embedding_scale != 1.0
+                                            or any(getattr(b, "reads_stream", False) for b in self.blocks)):
+            raise ValueError("rows by pairs of tokens go with a plain embedding: no positions, scale, kept history or layers that read the stream itself")
         self.head: Optional[torch.Tensor] = None
         self.row_tensors: Dict[str, torch.Tensor] = {}
         self.join_tensors: Dict[str, torch.Tensor] = {}
@@ -51,6 +55,8 @@ class Model:
         out: Dict[str, ExpectedTensor] = {spec.embedding_tensor: ExpectedTensor((spec.vocab_size, spec.dim))}
         if spec.position_tensor is not None:
             out[spec.position_tensor] = ExpectedTensor((spec.max_positions, spec.dim))
+        if spec.pair_table is not None:
+            out[spec.pair_table.tensor] = ExpectedTensor((spec.pair_table.buckets + 1, spec.dim))
         for layer, blk in zip(spec.layers, self.blocks):
             for name, e in blk.expected_tensors().items():
                 out[f"{layer.name}.{name}"] = e
@@ -73,6 +79,8 @@ class Model:
         self.embedding = as_compute(tensors[spec.embedding_tensor], self.env)
         if spec.position_tensor is not None:
             self.position_table = as_compute(tensors[spec.position_tensor], self.env)
+        if spec.pair_table is not None:
+            self.pair_rows = as_compute(tensors[spec.pair_table.tensor], self.env)
         for layer, blk in zip(spec.layers, self.blocks):
             blk.load({name: tensors[f"{layer.name}.{name}"] for name in blk.expected_tensors()})
         self.final_norm.load({name: tensors[f"{spec.final_norm_prefix}.{name}"]
@@ -110,6 +118,11 @@ class Model:
         """What each run of the run order wants from the cache manager."""
         return [(self.blocks[run.layer].cache_need(), self.blocks[run.layer].state_need(), run.cache_of)
                 for run in self.spec.run_order]
+
+    def model_state_need(self) -> Optional[StateNeed]:
+        """Per-request state that belongs to the model rather than to one of its runs: the request's last token,
+        where the embedding looks at pairs."""
+        return None if self.spec.pair_table is None else StateNeed((1,), torch.int32)
 
     # ----------------------------------------------------------------- forward
     def _residual_with_history(self, ctx) -> Residual:
@@ -160,6 +173,11 @@ class Model:
         first = self.blocks[self.spec.run_order[0].layer] if self.spec.run_order else None
         if self.spec.keeps_history:
             residual = self._residual_with_history(ctx)
+        elif self.spec.pair_table is not None:
+            pairs = self.spec.pair_table
+            residual = Residual(self.ops.embed_pairs(
+                ctx.token_ids, self.embedding, self.pair_rows, ctx.model_state, ctx.seq_of_token, ctx.q_start, ctx.state_slot, ctx.fresh,
+                mul_prev=pairs.mul_prev, mul_cur=pairs.mul_cur))
         elif self.position_table is None and self.spec.embedding_scale == 1.0 and not getattr(first, "reads_stream", False):
             residual = Residual(self.ops.embed(ctx.token_ids, self.embedding))
         elif getattr(first, "reads_stream", False):

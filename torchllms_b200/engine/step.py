@@ -79,6 +79,7 @@ class StepContext:
     q_lens: List[int] = field(default_factory=list)
     kv_lens: List[int] = field(default_factory=list)
     slots: List[int] = field(default_factory=list)
+    model_state: Optional[torch.Tensor] = None   # the model's own state rows [slots, ...], where it keeps any
     decode_kv_bound: int = 0     # the context length that the one-token rows of a mixed step plan their attention for
 
 
@@ -160,7 +161,8 @@ class Engine:
         self.max_step_tokens = int(max_step_tokens)
         self.cache = CacheManager(model.run_needs(), page_size=page_size, pool_tokens=pool_tokens,
                                   max_num_seqs=max_num_seqs, max_len=self.max_len, dtype=model.dtype,
-                                  device=self.device, max_step_tokens=self.max_step_tokens)
+                                  device=self.device, max_step_tokens=self.max_step_tokens,
+                                  model_state=model.model_state_need())
         self._buf = _StepBuffers(self.cache, self.max_step_tokens, self.device)
         self._has_window = any(g.gives_back for g in self.cache.groups)
         self.vocab_size = model.spec.vocab_size
@@ -472,7 +474,7 @@ class Engine:
                     seq_of_token=buf.dev_view("seq_of_token", T), q_start=buf.dev_view("q_start", B + 1),
                     kv_len=buf.dev_view("kv_len", B), state_slot=buf.dev_view("state_slot", B),
                     fresh=buf.dev_view("fresh", B), want_rows=buf.dev_view("want_rows", n_want),
-                    q_lens=q_lens, kv_lens=kv_lens, slots=slots)
+                    q_lens=q_lens, kv_lens=kv_lens, slots=slots, model_state=cache.model_state)
                 block_tables = [buf.dev_view(f"block_table{g}", B * buf.NB).view(B, buf.NB) for g in range(len(cache.groups))]
                 slot_maps = [buf.dev_view(f"slot_mapping{g}", T) for g in range(len(cache.groups))]
                 views = [cache.run_view(i, block_tables, slot_maps) for i in range(cache.n_runs)]

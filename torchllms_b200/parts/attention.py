@@ -19,7 +19,7 @@ import torch
 
 from ..kernels.lazy import PendingProduct
 from ..weights.loader import ExpectedTensor
-from .base import (POSITION_ENCODINGS, BuildEnv, CacheNeed, Mixer, as_compute, register_mixer)
+from .base import (POSITION_ENCODINGS, BuildEnv, CacheNeed, Mixer, StateNeed, as_compute, register_mixer)
 from .rope import precise_rotary_table
 from .spec import PartSpec
 
@@ -344,7 +344,11 @@ class RotaryGatedAttention(Mixer):
       (plain weights ``q_norm.weight``, ``k_norm.weight``), ahead of the rotation;
     * rotation of the first ``rot_dims`` coordinates of every q and k head by ``p * rot_base^(-2i/rot_dims)``
       (``rot_pairing`` ``"interleaved"``: coordinate ``2i`` with ``2i + 1``; ``"half"``: ``i`` with ``i + rot_dims / 2``), the
-      frequencies optionally rescaled by band (``rot_band``, see :func:`~torchllms_b200.parts.rope.band_scaled`);
+      frequencies optionally rescaled by band (``rot_band``, see :func:`~torchllms_b200.parts.rope.band_scaled`) or along a
+      ramp (``rot_ramp``, see :func:`~torchllms_b200.parts.rope.ramp_scaled`);
+    * with ``conv_taps`` every channel of q, k and v as projected passes a causal convolution over time, ahead of the
+      rotation (tensors ``wq.conv``, ``wk.conv``, ``wv.conv`` ``[channels, conv_taps]``, the last column the current token's,
+      zeros before a request's start); the last ``conv_taps - 1`` projected rows are per-request state;
     * with ``qk_head_norm`` every rotated head of q and k, and with ``v_head_norm`` every head's value, is divided by its
       root mean square (no weight); keys and values are stored so;
     * score ``= q . k * scale``, then, with ``softcap = c > 0``, ``c * tanh(score / c)``;
@@ -355,9 +359,9 @@ class RotaryGatedAttention(Mixer):
       ``sinks="zero"``, ``exp(0)`` and no tensor; ``weights="sigmoid"``: a visible key's weight is ``sigmoid(score +
       score_bias[h])`` (tensor ``score_bias``, a number per head), not normalised over the keys;
     * an output gate ``sigmoid(wg x)``, one number per head (``gate="head"``) or per element
-      (``"element"``), ahead of ``wo``.
+      (``"element"``), ahead of ``wo``; with convolutions the gate may be multiplied by ``out_scale``, which scales the result.
 
-    One stacked product gives q, k, v and the gate's logits; one kernel adds the biases, norms, rotates,
+    One stacked product gives q, k, v and the gate's logits; one kernel adds the biases, convolves or norms, rotates,
     stores keys and values and takes the gate's sigmoid; mask, cap, sink, sigmoid and gate live in the attention
     kernel; the output bias is added where the output product is added up."""
 
@@ -368,7 +372,8 @@ class RotaryGatedAttention(Mixer):
                  rot_dims: int = 0, rot_base: float = 10000.0, rot_pairing: str = "interleaved", window: Optional[int] = None,
                  qkv_bias: bool = False, out_bias: bool = False, gate: Optional[str] = None, rot_band: Optional[Mapping[str, float]] = None,
                  chunk: Optional[int] = None, values_are_keys: bool = False, qk_row_norm: bool = False, qk_head_norm: bool = False,
-                 v_head_norm: bool = False, norm_eps: float = 1e-6, weights: str = "softmax", score_bias: bool = False):
+                 v_head_norm: bool = False, norm_eps: float = 1e-6, weights: str = "softmax", score_bias: bool = False,
+                 conv_taps: int = 0, out_scale: float = 1.0, rot_ramp: Optional[Mapping[str, float]] = None):
         if n_heads % n_kv_heads != 0:
             raise ValueError(f"n_heads ({n_heads}) must be a multiple of n_kv_heads ({n_kv_heads})")
         if rot_dims < 0 or rot_dims % 2 or rot_dims > head_dim:
@@ -387,6 +392,12 @@ class RotaryGatedAttention(Mixer):
             raise ValueError("sinks (True or 'zero') go with softmax weights, a score bias with sigmoid weights")
         if values_are_keys and v_head_dim not in (None, head_dim):
             raise ValueError(f"values that are keys have the keys' size ({head_dim}), got v_head_dim {v_head_dim}")
+        self.taps, self.out_scale = int(conv_taps), float(out_scale)
+        if self.taps < 0 or (self.taps and (qkv_bias or values_are_keys or qk_row_norm or qk_head_norm or v_head_norm
+                                            or rot_pairing != "half")):
+            raise ValueError("short convolutions go with plain q, k and v of their own, rotated in the 'half' pairing, without biases and norms")
+        if self.out_scale != 1.0 and not (self.taps and gate):
+            raise ValueError("out_scale is applied to the output gate, behind short convolutions")
         self.env = env
         self.dim, self.n_heads, self.n_kv_heads = int(dim), int(n_heads), int(n_kv_heads)
         self.head_dim = int(head_dim)
@@ -406,7 +417,10 @@ class RotaryGatedAttention(Mixer):
         self.n_v = 0 if self.values_are_keys else self.n_kv_heads * self.v_head_dim
         self.n_g = {None: 0, "head": self.n_heads, "element": self.n_heads * self.v_head_dim}[gate]
         env.ops.check_attention_sizes(self.n_heads, self.n_kv_heads, self.head_dim, env.dtype, v_head_dim=self.v_head_dim)
-        self.table = precise_rotary_table(max(self.rot_dims, 2), rot_base, 1.0, env.max_positions, env.device, band=rot_band)
+        self.table = precise_rotary_table(max(self.rot_dims, 2), rot_base, 1.0, env.max_positions, env.device, band=rot_band,
+                                          ramp=rot_ramp if self.rot_dims else None)
+        self.runs_in_halves = self.taps > 0 and not out_bias
+        self.w_conv: Optional[torch.Tensor] = None
         self.w_in = self.b_in = self.sinks = self.wo = self.bo = self.q_norm_w = self.k_norm_w = self.score_bias = None
 
     def cache_need(self) -> CacheNeed:
@@ -416,10 +430,15 @@ class RotaryGatedAttention(Mixer):
             return CacheNeed("full", self.n_kv_heads, self.head_dim, None, self.v_head_dim)
         return CacheNeed("window", self.n_kv_heads, self.head_dim, self.window, self.v_head_dim)
 
+    def state_need(self) -> Optional[StateNeed]:
+        return StateNeed((self.taps - 1, self.n_q + self.n_k + self.n_v)) if self.taps > 1 else None
+
     def expected_tensors(self) -> Dict[str, ExpectedTensor]:
         out = {"wo.weight": ExpectedTensor((self.dim, self.n_heads * self.v_head_dim))}
         for name, rows in self._projected():
             out[f"{name}.weight"] = ExpectedTensor((rows, self.dim))
+            if self.taps:
+                out[f"{name}.conv"] = ExpectedTensor((rows, self.taps))
             if self.qkv_bias:
                 out[f"{name}.bias"] = ExpectedTensor((rows,))
         if self.qk_row_norm:
@@ -456,19 +475,29 @@ class RotaryGatedAttention(Mixer):
             self.bo = tensors["wo.bias"].to(**f32).contiguous()
         if self.has_sinks:
             self.sinks = tensors["sinks"].to(**f32).contiguous()
+        if self.taps:
+            self.w_conv = torch.cat([tensors[f"{n}.conv"].to(**f32) for n, _rows in self._projected()]).contiguous()
         self.wo = as_compute(tensors["wo.weight"], self.env)
 
     def weight_bytes(self) -> int:
-        return sum(t.numel() * t.element_size() for t in (self.w_in, self.wo))
+        return sum(t.numel() * t.element_size() for t in (self.w_in, self.wo) if t is not None)
 
     def forward(self, x: torch.Tensor, ctx, cache) -> PendingProduct:
+        o = self.mix(self.env.ops.linear(x, self.w_in, partials_ok=True), ctx, cache)
+        return PendingProduct(o, self.wo, bias=self.bo)
+
+    def mix(self, proj: torch.Tensor, ctx, cache, out: Optional[torch.Tensor] = None) -> torch.Tensor:
         ops = self.env.ops
-        proj = ops.linear(x, self.w_in, partials_ok=True)
         store = dict(n_q_heads=self.n_heads, n_k_heads=self.n_kv_heads, head_dim=self.head_dim, v_head_dim=self.v_head_dim,
                      rot_dims=self.rot_dims, interleaved=self.interleaved, n_extra=self.n_g, k_pages=cache.k_pages,
                      v_pages=cache.v_pages, slot_mapping=cache.slot_mapping, page_size=cache.page_size, out_dtype=self.env.dtype,
                      bias=self.b_in)
-        if self.qk_row_norm or self.qk_head_norm or self.v_head_norm or self.values_are_keys:
+        if self.taps:
+            del store["interleaved"], store["bias"]
+            q, gate = ops.conv_rope_store(proj, self.w_conv, cache.state if self.taps > 1 else None, ctx.positions, self.table, ctx.q_start,
+                                          ctx.state_slot, ctx.fresh, n_seqs=ctx.n_seqs, max_q_len=ctx.max_q_len,
+                                          extra_scale=self.out_scale, **store)
+        elif self.qk_row_norm or self.qk_head_norm or self.v_head_norm or self.values_are_keys:
             q, gate = ops.norm_rope_store(proj, ctx.positions, self.table, values_are_keys=self.values_are_keys,
                                           q_norm=self.q_norm_w, k_norm=self.k_norm_w, qk_head_norm=self.qk_head_norm,
                                           v_head_norm=self.v_head_norm, eps=self.norm_eps, **store)
@@ -478,5 +507,6 @@ class RotaryGatedAttention(Mixer):
             q, cache.k_pages, cache.v_pages, cache.block_table, ctx.q_start, ctx.kv_len, n_seqs=ctx.n_seqs,
             max_q_len=ctx.max_q_len, max_kv_len=ctx.max_kv_len, scale=self.scale, window=self.window, chunk=self.chunk,
             page_size=cache.page_size, gate=gate, softcap=self.softcap, sinks=self.sinks, weights=self.weights,
-            score_bias=self.score_bias, impl="auto")
-        return PendingProduct(o.view(o.shape[0], self.n_heads * self.v_head_dim), self.wo, bias=self.bo)
+            score_bias=self.score_bias, impl="auto",
+            **({} if out is None else dict(out=out.unflatten(1, (self.n_heads, self.v_head_dim)))))
+        return o.view(o.shape[0], self.n_heads * self.v_head_dim) if out is None else out

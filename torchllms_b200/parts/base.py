@@ -238,6 +238,11 @@ class Mixer(Part):
     """
 
     takes_row_scaled = False
+    # A mixer that starts with one product of its input and ends with one product may be run in halves, so that a
+    # part that holds several of them can stack their products: ``w_in`` and ``wo`` are the two weights, and
+    # ``mix(proj, ctx, cache, out)`` is all that lies between: ``proj`` is ``x @ w_in.T``, a column range of wider rows or
+    # of float32 partial sums of them; the rows that ``wo`` multiplies go to ``out`` (a column range of wider rows).
+    runs_in_halves = False
 
     def cache_need(self) -> Optional[CacheNeed]:
         return None
@@ -246,6 +251,9 @@ class Mixer(Part):
         return None
 
     def forward(self, x: torch.Tensor, ctx, cache) -> torch.Tensor:
+        raise NotImplementedError
+
+    def mix(self, proj: torch.Tensor, ctx, cache, out: Optional[torch.Tensor] = None) -> torch.Tensor:
         raise NotImplementedError
 
 

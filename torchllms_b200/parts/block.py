@@ -152,8 +152,8 @@ class SandwichBlock(Block):
     ``n`` this layer's own), with the coefficients in the layer's tensor ``depth_tensor``.  Such a
     block needs a model that keeps its history (``ModelSpec.keeps_history``).
 
-    The output norm's kernel adds to the stream and, where a feed-forward follows, also takes the
-    norm in front of it, so two kernels stand between the mixer's and the feed-forward's products."""
+    The output norm's kernel adds to the stream and also takes the norm in front of whatever reads the
+    stream next (the feed-forward, or the next layer's mixer where nothing stands between)."""
 
     def __init__(self, env: BuildEnv, *, mixer: PartSpec, feed_forward: Optional[PartSpec],
                  mixer_norm: PartSpec, mixer_out_norm: PartSpec, ffn_norm: Optional[PartSpec],
@@ -213,12 +213,15 @@ class SandwichBlock(Block):
         else:
             x = self.mixer_norm.forward(residual)
         residual.normed = None
-        y = self.mixer.forward(x, ctx, cache)
-        if self.feed_forward is None:
-            self.mixer_out_norm.fold_normed(residual, y, want_rows=False)
-        else:
+        y, last = self.mixer.forward(x, ctx, cache), self.mixer_out_norm
+        if self.feed_forward is not None:
             x = self.mixer_out_norm.fold_normed(residual, y, then=self.ffn_norm)
-            self.ffn_out_norm.fold_normed(residual, self.feed_forward.forward(x, ctx), want_rows=False)
+            y, last = self.feed_forward.forward(x, ctx), self.ffn_out_norm
+        follow = residual.next_norm
+        if self.depth_inputs is None and residual.history is None and isinstance(follow, RMSNorm) and follow.groups == 1:
+            residual.normed = (follow, last.fold_normed(residual, y, then=follow))
+        else:
+            last.fold_normed(residual, y, want_rows=False)
         if self.depth_inputs is not None:
             history, level = residual.history, residual.level
             if history is None or self.depth_inputs != level + 2:

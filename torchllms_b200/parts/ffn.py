@@ -148,3 +148,31 @@ class PolyNormFeedForward(FeedForward):
         ops = self.env.ops
         y = ops.polynorm(ops.linear(x, self.w_up, partials_ok=True), self.coef, self.eps, out_dtype=self.env.dtype)
         return PendingProduct(y, self.w_down)
+
+
+@register_feed_forward("activated")
+class ActivatedFeedForward(FeedForward):
+    """Dense feed-forward without a gate: ``down(act(up x))``, ``act`` being ``gelu_tanh`` (``0.5 z (1 + tanh(sqrt(2 / pi)
+    (z + 0.044715 z^3)))``), ``silu``, ``relu2`` or ``gelu`` (with erf), in float32 arithmetic."""
+
+    graph_safe = True
+
+    def __init__(self, env: BuildEnv, *, dim: int, hidden: int, activation: str):
+        if activation not in ("gelu_tanh", "silu", "relu2", "gelu"):
+            raise ValueError(f"unknown activation {activation!r}; known: gelu_tanh, silu, relu2, gelu")
+        self.env = env
+        self.dim, self.hidden, self.activation = int(dim), int(hidden), activation
+        self.w_up: Optional[torch.Tensor] = None
+        self.w_down: Optional[torch.Tensor] = None
+
+    def expected_tensors(self) -> Dict[str, ExpectedTensor]:
+        return {"up.weight": ExpectedTensor((self.hidden, self.dim)), "down.weight": ExpectedTensor((self.dim, self.hidden))}
+
+    def load(self, tensors: Mapping[str, torch.Tensor]) -> None:
+        self.w_up = as_compute(tensors["up.weight"], self.env)
+        self.w_down = as_compute(tensors["down.weight"], self.env)
+
+    def forward(self, x: torch.Tensor, ctx) -> PendingProduct:
+        ops = self.env.ops
+        u = ops.activation(ops.linear(x, self.w_up, partials_ok=True), self.activation, out_dtype=self.env.dtype)
+        return PendingProduct(u, self.w_down)

@@ -33,11 +33,14 @@ class RMSNorm(Norm):
     graph_safe = True
     can_defer = True
 
-    def __init__(self, env: BuildEnv, *, dim: int, eps: float, offset: float = 0.0, scalar: bool = False, groups: int = 1):
+    def __init__(self, env: BuildEnv, *, dim: int, eps: float, offset: float = 0.0, scalar: bool = False, groups: int = 1,
+                 weight_scale: float = 1.0):
         """``offset``: what is added to the stored weight (1 for a weight that is kept around zero).
         ``scalar``: the stored weight is one number for all coordinates (a tensor without axes).
         ``groups``: the row is cut into so many equal runs of neighbouring coordinates, each divided by a root
-        mean square of its own (one scale per row is not enough then, so nothing is deferred)."""
+        mean square of its own (one scale per row is not enough then, so nothing is deferred).
+        ``weight_scale``: what the weight is multiplied by, in 32-bit (a norm on a sublayer's output whose result enters
+        the stream multiplied by a constant)."""
         if groups < 1 or dim % groups:
             raise ValueError(f"a norm over {dim} coordinates cannot have {groups} equal groups")
         self.groups = int(groups)
@@ -46,7 +49,7 @@ class RMSNorm(Norm):
         self.scalar = bool(scalar)
         self.dim = int(dim)
         self.eps = float(eps)
-        self.offset = float(offset)
+        self.offset, self.weight_scale = float(offset), float(weight_scale)
         self.weight: Optional[torch.Tensor] = None
 
     def expected_tensors(self) -> Dict[str, ExpectedTensor]:
@@ -55,6 +58,8 @@ class RMSNorm(Norm):
     def load(self, tensors: Mapping[str, torch.Tensor]) -> None:
         # Kept in 32-bit whatever the activation dtype: the kernel multiplies in 32-bit.
         w = tensors["weight"].to(device=self.env.device, dtype=torch.float32) + self.offset
+        if self.weight_scale != 1.0:
+            w = w * self.weight_scale
         self.weight = (w.reshape(1).expand(self.dim) if self.scalar else w).contiguous()
 
     def forward(self, residual: Residual, rows: Optional[torch.Tensor] = None, deferred_ok: bool = False):

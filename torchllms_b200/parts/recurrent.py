@@ -140,78 +140,117 @@ class GatedDelta(Mixer):
 
         ``S <- g_t S``;  ``u = beta_t (v_t - S^T k_t)``;  ``S <- S + k_t u^T``;  ``o_t = S^T q_t``
 
-    with ``beta = sigmoid(wb x)`` and ``g = exp(-exp(A_log) softplus(wa x + dt_bias))`` per head.  q
+    with ``beta = sigmoid(wb x)`` per head.  The decay ``g`` is one number per head
+    (``decay="head"``: ``g = exp(-exp(A_log) softplus(wa x + dt_bias))``) or one per head and key coordinate
+    (``decay="channel"``: ``g = exp(-exp(A_log_h) softplus(wa2 (wa1 x) + dt_bias))``, ``head_dim`` numbers a head, each acting on
+    its own row of ``S``; the inner size is the stored tensors').  q
     and k (``n_qk_heads`` heads, shared by ``n_heads / n_qk_heads`` value heads each) and v pass a
     short causal convolution over time (``conv_taps`` taps per channel, the last one the current
     token's) and ``silu``; q and k become unit vectors (``x / sqrt(sum(x^2) + unit_eps)``) and q is
     multiplied by ``q_scale``.  Each head's ``o`` is RMS-normed over its values with the weight
-    ``norm.weight`` (shared by heads), multiplied by ``silu(wg x)`` and projected by ``wo``.
+    ``norm.weight`` (shared by heads), multiplied by an output gate (``gate_activation``: ``silu`` or ``sigmoid``) of ``wg x``
+    or, with ``low_rank_gate``, of ``wg2 (wg1 x)``, and projected by ``wo``.  ``out_scale`` scales the result.
 
     State per request: the convolutions' last ``conv_taps - 1`` inputs and the heads' matrices (kept
-    as ``S^T``, ``[heads, v_head_dim, head_dim]``), all float32.  One stacked product gives ``[q | k | v | b | a | g]``."""
+    as ``S^T``, ``[heads, v_head_dim, head_dim]``), all float32.  One stacked product gives
+    ``[q | k | v | b | a | g]``, ``a`` and ``g`` being the inner numbers where they are of low rank; one kernel convolves,
+    activates and norms; the outer products of the low-rank terms are one product over their inner numbers side by side."""
 
     graph_safe = True
 
     def __init__(self, env: BuildEnv, *, dim: int, n_heads: int, n_qk_heads: int, head_dim: int, v_head_dim: int,
-                 conv_taps: int, q_scale: float, norm_eps: float, unit_eps: float = 1e-6):
+                 conv_taps: int, q_scale: float, norm_eps: float, unit_eps: float = 1e-6, decay: str = "head",
+                 low_rank_gate: bool = False, gate_activation: str = "silu", out_scale: float = 1.0):
         if n_heads % n_qk_heads != 0:
             raise ValueError(f"n_heads ({n_heads}) must be a multiple of n_qk_heads ({n_qk_heads})")
         if conv_taps < 1:
             raise ValueError(f"a convolution has at least one tap, got {conv_taps}")
+        if decay not in ("head", "channel"):
+            raise ValueError(f"a decay is one number per 'head' or per 'channel', got {decay!r}")
+        if gate_activation not in ("silu", "sigmoid"):
+            raise ValueError(f"an output gate is 'silu' or 'sigmoid', got {gate_activation!r}")
         self.env = env
         self.dim, self.n_heads, self.n_qk_heads = int(dim), int(n_heads), int(n_qk_heads)
         self.head_dim, self.v_head_dim, self.taps = int(head_dim), int(v_head_dim), int(conv_taps)
         self.q_scale, self.norm_eps, self.unit_eps = float(q_scale), float(norm_eps), float(unit_eps)
+        self.per_channel, self.low_rank_gate = decay == "channel", bool(low_rank_gate)
+        self.gate_activation, self.out_scale = gate_activation, float(out_scale)
+        # with every term behind the convolutions of low rank, nothing but the preparing kernel reads the product
+        self.runs_in_halves = self.per_channel and self.low_rank_gate
         self.n_qk, self.n_v = self.n_qk_heads * self.head_dim, self.n_heads * self.v_head_dim
         self.n_conv = 2 * self.n_qk + self.n_v
+        self.n_small = self.n_heads * (1 if self.per_channel else 2)           # beta's logits, and a decay's per head
+        self.n_decay = self.n_heads * self.head_dim if self.per_channel else self.n_heads
         self._need = join_states([("conv", StateNeed((self.taps - 1, self.n_conv)) if self.taps > 1 else None),
                                   ("matrix", StateNeed((self.n_heads, self.v_head_dim, self.head_dim)))])      # S^T per head
-        self.w_in = self.w_conv = self.decay_rate = self.decay_bias = self.norm_w = self.wo = None
+        self.n_low = 0                                                         # inner numbers of the low-rank terms, and padded
+        self.low_pad = 0
+        self.w_in = self.w_conv = self.w_low = self.decay_rate = self.decay_bias = self.norm_w = self.wo = None
 
     def state_need(self) -> StateNeed:
         return self._need
 
     def expected_tensors(self) -> Dict[str, ExpectedTensor]:
         d, H = self.dim, self.n_heads
-        return {"wq.weight": ExpectedTensor((self.n_qk, d)), "wk.weight": ExpectedTensor((self.n_qk, d)),
-                "wv.weight": ExpectedTensor((self.n_v, d)), "wq.conv": ExpectedTensor((self.n_qk, self.taps)),
-                "wk.conv": ExpectedTensor((self.n_qk, self.taps)), "wv.conv": ExpectedTensor((self.n_v, self.taps)),
-                "wb.weight": ExpectedTensor((H, d)), "wa.weight": ExpectedTensor((H, d)), "A_log": ExpectedTensor((H,)),
-                "dt_bias": ExpectedTensor((H,)), "norm.weight": ExpectedTensor((self.v_head_dim,)),
-                "wg.weight": ExpectedTensor((self.n_v, d)), "wo.weight": ExpectedTensor((d, self.n_v))}
+        out = {"wq.weight": ExpectedTensor((self.n_qk, d)), "wk.weight": ExpectedTensor((self.n_qk, d)),
+               "wv.weight": ExpectedTensor((self.n_v, d)), "wq.conv": ExpectedTensor((self.n_qk, self.taps)),
+               "wk.conv": ExpectedTensor((self.n_qk, self.taps)), "wv.conv": ExpectedTensor((self.n_v, self.taps)),
+               "wb.weight": ExpectedTensor((H, d)), "A_log": ExpectedTensor((H,)), "dt_bias": ExpectedTensor((self.n_decay,)),
+               "norm.weight": ExpectedTensor((self.v_head_dim,)), "wo.weight": ExpectedTensor((d, self.n_v))}
+        for name, rows, low in (("wa", self.n_decay, self.per_channel), ("wg", self.n_v, self.low_rank_gate)):
+            if low:
+                out.update({f"{name}1.weight": ExpectedTensor((-1, d)), f"{name}2.weight": ExpectedTensor((rows, -1))})
+            else:
+                out[f"{name}.weight"] = ExpectedTensor((rows, d))
+        return out
 
     def load(self, tensors: Mapping[str, torch.Tensor]) -> None:
         f32 = dict(device=self.env.device, dtype=torch.float32)
-        names = ("wq.weight", "wk.weight", "wv.weight", "wb.weight", "wa.weight", "wg.weight")
+        names = ["wq.weight", "wk.weight", "wv.weight", "wb.weight"] + ["wa1.weight" if self.per_channel else "wa.weight"] \
+            + ["wg1.weight" if self.low_rank_gate else "wg.weight"]
         self.w_in = torch.cat([as_compute(tensors[n], self.env) for n in names])
         self.w_conv = torch.cat([tensors[n].to(**f32) for n in ("wq.conv", "wk.conv", "wv.conv")]).contiguous()
+        outer = [tensors[f"{n}2.weight"] for n, low in (("wa", self.per_channel), ("wg", self.low_rank_gate)) if low]
+        inner = [tensors[f"{n}1.weight"].shape[0] for n, low in (("wa", self.per_channel), ("wg", self.low_rank_gate)) if low]
+        if outer:
+            if [w.shape[1] for w in outer] != inner:
+                raise ValueError(f"low-rank terms: inner sizes {[w.shape[1] for w in outer]} of the second matrices, {inner} of the first")
+            # the second matrices on the diagonal, zero columns up to a multiple of eight: [decays | gate] = w_low [inner numbers]
+            self.n_low, self.low_pad = sum(inner), -(-sum(inner) // 8) * 8
+            w = torch.zeros((sum(m.shape[0] for m in outer), self.low_pad), dtype=outer[0].dtype, device=outer[0].device)
+            r = c = 0
+            for m in outer:
+                w[r:r + m.shape[0], c:c + m.shape[1]] = m
+                r, c = r + m.shape[0], c + m.shape[1]
+            self.w_low = as_compute(w, self.env)
         self.decay_rate = torch.exp(tensors["A_log"].to(**f32)).contiguous()       # exp(A_log), taken once
         self.decay_bias = tensors["dt_bias"].to(**f32).contiguous()
-        self.norm_w = tensors["norm.weight"].to(**f32).contiguous()
+        self.norm_w = (tensors["norm.weight"].to(**f32) * self.out_scale).contiguous()
         self.wo = as_compute(tensors["wo.weight"], self.env)
 
     def weight_bytes(self) -> int:
-        return sum(t.numel() * t.element_size() for t in (self.w_in, self.wo))
+        return sum(t.numel() * t.element_size() for t in (self.w_in, self.w_low, self.wo) if t is not None)
 
     def forward(self, x: torch.Tensor, ctx, cache) -> PendingProduct:
+        # (a gate of full rank is read from the product's rows by the last kernel, which takes no partial sums)
+        proj = self.env.ops.linear(x, self.w_in, partials_ok=self.low_rank_gate)
+        return PendingProduct(self.mix(proj, ctx, cache), self.wo)
+
+    def mix(self, proj: torch.Tensor, ctx, cache, out: Optional[torch.Tensor] = None) -> torch.Tensor:
         ops = self.env.ops
-        H, n, nv, nc = self.n_heads, self.n_qk, self.n_v, self.n_conv
-        proj = ops.linear(x, self.w_in)
-        if self.taps > 1:
-            c = ops.short_conv(proj[:, :nc], self.w_conv, state_field(cache.state, self._need, "conv"), ctx.q_start,
-                               ctx.state_slot, ctx.fresh, n_seqs=ctx.n_seqs, max_q_len=ctx.max_q_len, activation="silu",
-                               residual=False, out_dtype=self.env.dtype)
-        else:
-            c = ops.short_conv(proj[:, :nc], self.w_conv, None, ctx.q_start, ctx.state_slot, ctx.fresh, n_seqs=ctx.n_seqs,
-                               max_q_len=ctx.max_q_len, activation="silu", residual=False, out_dtype=self.env.dtype)
-        unit = dict(n_heads=self.n_qk_heads, head_dim=self.head_dim, unit_eps=self.unit_eps)
-        q = ops.recurrence_prep(c[:, :n], scale=self.q_scale, **unit)
-        k = ops.recurrence_prep(c[:, n:2 * n], scale=1.0, **unit)
-        o = _matrix_state_scan(ops, q, k, c[:, 2 * n:], state_field(cache.state, self._need, "matrix"), ctx,
-                               beta_logits=proj[:, nc:nc + H], decay_logits=proj[:, nc + H:nc + 2 * H],
-                               decay_rate=self.decay_rate, decay_bias=self.decay_bias)
-        y = ops.head_norm_gate(o, proj[:, nc + 2 * H:], self.norm_w, self.norm_eps, head_dim=self.v_head_dim, out_dtype=self.env.dtype)
-        return PendingProduct(y, self.wo)
+        H, nv, nc = self.n_heads, self.n_v, self.n_conv
+        conv_state = state_field(cache.state, self._need, "conv") if self.taps > 1 else None
+        q, k, v, small, low = ops.delta_prep(
+            proj, self.w_conv, conv_state, ctx.q_start, ctx.state_slot, ctx.fresh, n_seqs=ctx.n_seqs, max_q_len=ctx.max_q_len,
+            n_qk_heads=self.n_qk_heads, head_dim=self.head_dim, n_v=nv, n_small=self.n_small, n_low=self.n_low, low_pad=self.low_pad,
+            q_scale=self.q_scale, unit_eps=self.unit_eps, out_dtype=self.env.dtype)
+        outer = None if low is None else ops.linear(low, self.w_low)
+        decay = outer[:, :self.n_decay] if self.per_channel else small[:, H:]
+        gate = outer[:, outer.shape[1] - nv:] if self.low_rank_gate else proj[:, nc + self.n_small + self.n_low:]
+        o = _matrix_state_scan(ops, q, k, v, state_field(cache.state, self._need, "matrix"), ctx, beta_logits=small[:, :H],
+                               decay_logits=decay, decay_rate=self.decay_rate, decay_bias=self.decay_bias)
+        return ops.head_norm_gate(o, gate, self.norm_w, self.norm_eps, head_dim=self.v_head_dim, out_dtype=self.env.dtype,
+                                  activation=self.gate_activation, out=out)
 
 
 @register_mixer("selective_scan")

@@ -67,22 +67,41 @@ def band_scaled(freq: torch.Tensor, factor: float, low: float, high: float, orig
     return torch.where(wavelen < original / high, freq, torch.where(wavelen > original / low, freq / factor, blended))
 
 
+def ramp_scaled(freq: torch.Tensor, theta: float, factor: float, original: float, fast: float, slow: float):
+    """Frequencies rescaled along a ramp (YaRN) in ``freq``'s own precision, and what cos and sin are multiplied by.
+    ``freq[i] = theta^(-2i/dims)``.  The coordinate that turns ``n`` times within ``original`` positions is
+    ``c(n) = dims ln(original / (2 pi n)) / (2 ln theta)``; pairs up to ``floor(c(fast))`` keep their frequency, pairs from
+    ``ceil(c(slow))`` on are divided by ``factor``, and in between the two are blended linearly in the pair's number.  Cos
+    and sin grow by ``0.1 ln(factor) + 1``."""
+    dims = 2 * freq.numel()
+    at = lambda turns: dims * math.log(original / (2.0 * math.pi * turns)) / (2.0 * math.log(theta))
+    lo, hi = max(math.floor(at(fast)), 0), min(math.ceil(at(slow)), dims - 1)
+    i = torch.arange(freq.numel(), dtype=freq.dtype)
+    ramp = ((i - lo) / max(hi - lo, 0.001)).clamp(0.0, 1.0)
+    return freq / factor * ramp + freq * (1.0 - ramp), 0.1 * math.log(factor) + 1.0
+
+
 def precise_rotary_table(dims: int, theta: float, factor: float, max_positions: int, device="cpu",
-                         band: Optional[Mapping[str, float]] = None) -> torch.Tensor:
+                         band: Optional[Mapping[str, float]] = None, ramp: Optional[Mapping[str, float]] = None) -> torch.Tensor:
     """``[max_positions, dims / 2, 2]`` float32 (cos, sin) of the angles ``p * theta^(-2i/dims) / factor``,
     the angles taken in 64-bit so that the table is exact to float32 rounding at any position.
-    ``band`` (``factor``, ``low``, ``high``, ``original``) rescales the frequencies by :func:`band_scaled`.
+    ``band`` (``factor``, ``low``, ``high``, ``original``) rescales the frequencies by :func:`band_scaled`; ``ramp``
+    (``factor``, ``original``, ``fast``, ``slow``) rescales frequencies and entries by :func:`ramp_scaled`.
     Layers with the same numbers on the same device share one table."""
     bands = None if band is None else tuple(float(band[k]) for k in ("factor", "low", "high", "original"))
-    key = (int(dims), float(theta), float(factor), int(max_positions), str(device), bands)
+    ramps = None if ramp is None else tuple(float(ramp[k]) for k in ("factor", "original", "fast", "slow"))
+    key = (int(dims), float(theta), float(factor), int(max_positions), str(device), bands, ramps)
     table = _precise_tables.get(key)
     if table is None:
         i = torch.arange(dims // 2, dtype=torch.float64)
         freq = float(theta) ** (-2.0 * i / dims) / float(factor)
         if bands is not None:
             freq = band_scaled(freq, *bands)
+        grow = 1.0
+        if ramps is not None:
+            freq, grow = ramp_scaled(freq, float(theta), *ramps)
         angles = torch.arange(max_positions, dtype=torch.float64)[:, None] * freq[None, :]
-        table = torch.stack([torch.cos(angles), torch.sin(angles)], dim=-1).to(torch.float32).contiguous().to(device)
+        table = (grow * torch.stack([torch.cos(angles), torch.sin(angles)], dim=-1)).to(torch.float32).contiguous().to(device)
         if len(_precise_tables) >= 8:
             _precise_tables.clear()
         _precise_tables[key] = table

@@ -71,6 +71,18 @@ class RunEntry:
 
 
 @dataclass(frozen=True)
+class PairTable:
+    """A table of rows by pairs of neighbouring tokens, added to the embedding: with ``p`` the request's token before
+    ``t``, row ``(p * mul_prev + t * mul_cur) mod buckets`` of the model-level ``[buckets + 1, dim]`` tensor; a request's
+    first token, which has none before it, takes the last row.  The last token of every request is model-level state."""
+
+    tensor: str
+    buckets: int
+    mul_prev: int
+    mul_cur: int
+
+
+@dataclass(frozen=True)
 class ModelSpec:
     dim: int
     vocab_size: int
@@ -89,6 +101,7 @@ class ModelSpec:
     embedding_norm_prefix: str = "embedding_norm"    # prefix of that norm's tensors
     logit_scale: float = 1.0         # the head's products leave multiplied by this
     row_tensors: Tuple[Tuple[str, int], ...] = ()    # model-level (name, rows) tensors [rows, dim] whose rows runs add to the stream (RunEntry.add_row)
+    pair_table: Optional[PairTable] = None           # rows by pairs of neighbouring tokens, added to the embedding
     join_tensors: Tuple[str, ...] = ()               # model-level [dim, 2 dim] matrices that join the stream and the embedding output (RunEntry.join_embedding)
 
     def __post_init__(self):
