@@ -116,15 +116,14 @@ def channel_delta(q, k, v, beta, decay):
     decay each at its own rate, then is corrected under the current key and read by the current query."""
     n, H, dv = v.shape
     G, d = k.shape[1:]
+    of = [a // (H // G) for a in range(H)]           # the head of q and k that goes with head a
+    S = torch.zeros(H, d, dv, dtype=F64)
     out = torch.zeros(n, H, dv, dtype=F64)
-    for a in range(H):
-        g = a // (H // G)
-        S = torch.zeros(d, dv, dtype=F64)
-        for t in range(n):
-            S = decay[t, a][:, None] * S
-            u = beta[t, a] * (v[t, a] - S.T @ k[t, g])
-            S = S + torch.outer(k[t, g], u)
-            out[t, a] = S.T @ q[t, g]
+    for t in range(n):
+        S = decay[t][:, :, None] * S
+        u = beta[t][:, None] * (v[t] - torch.einsum("hdv,hd->hv", S, k[t, of]))
+        S = S + k[t, of][:, :, None] * u[:, None, :]
+        out[t] = torch.einsum("hdv,hd->hv", S, q[t, of])
     return out
 
 

@@ -62,6 +62,7 @@ struct AttnParams {
     const void* gate;    // [T, n_heads] (gate_mode 1) or [T, n_heads * v_head_dim] (gate_mode 2), in q's dtype
     int gate_mode, n_bucket, keep_first;
     int n_v_heads, out_f32;
+    long long out_pitch;       // elements between two tokens' results
     int v_stride;        // elements between stored values (v_head_dim unless values are parts of wider vectors)
     float softcap;       // 0: none
     const float* sinks;  // [n_heads] or null
@@ -256,8 +257,9 @@ __global__ void __launch_bounds__(NT) paged_attention_kernel(const AttnParams p)
     const int head = kvh * p.group + g0 + rr % ng;
     const size_t row = (size_t)tok * p.n_heads + head;
     if (p.n_splits == 1) {
-        T* o = reinterpret_cast<T*>(p.out) + row * dv;
-        float* o32 = reinterpret_cast<float*>(p.out) + row * dv;
+        const size_t out_at = (size_t)tok * p.out_pitch + (size_t)head * dv;
+        T* o = reinterpret_cast<T*>(p.out) + out_at;
+        float* o32 = reinterpret_cast<float*>(p.out) + out_at;
         if (p.sinks != nullptr) {
             // one more term of the denominator: exp(sink - M) with M = max(m, sink), everything else rescaled to M
             const float sink = p.sinks[head];
@@ -295,8 +297,9 @@ template <typename T>
 __global__ void attention_merge_kernel(const float* __restrict__ part_o, const float* __restrict__ part_ml,
                                        T* __restrict__ out, int n_splits, int head_dim,
                                        const T* __restrict__ gate, int gate_mode, int out_f32,
-                                       const float* __restrict__ sinks, int n_heads, int sigmoid) {
+                                       const float* __restrict__ sinks, int n_heads, int sigmoid, long long out_pitch) {
     const size_t row = blockIdx.x;
+    const size_t out_at = row / n_heads * out_pitch + row % n_heads * head_dim;
     const float* ml = part_ml + row * n_splits * 2;
     float M = -INFINITY;
     for (int i = 0; i < n_splits; ++i) M = fmaxf(M, ml[2 * i]);
@@ -315,8 +318,8 @@ __global__ void attention_merge_kernel(const float* __restrict__ part_o, const f
         float o = sigmoid ? num : den > 0.f ? num / den : 0.f;       // (without a sum to divide by the partial results just add up)
         if (gate_mode == 1) o *= to_float(gate[row]);
         else if (gate_mode == 2) o *= to_float(gate[row * head_dim + d]);
-        if (out_f32) reinterpret_cast<float*>(out)[row * head_dim + d] = o;
-        else out[row * head_dim + d] = from_float<T>(o);
+        if (out_f32) reinterpret_cast<float*>(out)[out_at + d] = o;
+        else out[out_at + d] = from_float<T>(o);
     }
 }
 
@@ -391,6 +394,7 @@ struct TlAttentionOptions {
     int chunk;              // 0: none; not together with a window
     int sigmoid;            // 1: sigmoid weights without a sum over the keys; not together with sinks
     const float* score_bias;   // [n_heads] or null; sigmoid only
+    long long out_pitch;       // elements between two tokens' results; 0: n_heads * v_head_dim
 };
 
 // How many key splits the general kernel would use for this batch, and how many float32 words of
@@ -464,6 +468,7 @@ extern "C" int tl_paged_attention_ex(const void* q, const void* k_pages, const v
     p.n_v_heads = o.n_v_heads; p.out_f32 = o.out_f32;
     p.v_stride = o.v_stride; p.softcap = o.softcap; p.sinks = o.sinks;
     p.chunk = o.chunk; p.sigmoid = o.sigmoid; p.score_bias = o.score_bias;
+    p.out_pitch = o.out_pitch > 0 ? o.out_pitch : (long long)n_heads * o.v_head_dim;
     p.n_splits = pl.n_splits;
     p.scale = scale;
     p.part_o = workspace;
@@ -481,11 +486,12 @@ extern "C" int tl_paged_attention_ex(const void* q, const void* k_pages, const v
         const unsigned rows = (unsigned)n_tokens * n_heads;
         if (dtype == TL_F32)
             attention_merge_kernel<float><<<rows, threads, 0, s>>>(p.part_o, p.part_ml, (float*)out, pl.n_splits, o.v_head_dim,
-                                                                    (const float*)o.gate, o.gate_mode, o.out_f32, o.sinks, n_heads, o.sigmoid);
+                                                                    (const float*)o.gate, o.gate_mode, o.out_f32, o.sinks, n_heads, o.sigmoid,
+                                                                    p.out_pitch);
         else
             attention_merge_kernel<__nv_bfloat16><<<rows, threads, 0, s>>>(p.part_o, p.part_ml, (__nv_bfloat16*)out, pl.n_splits,
                                                                             o.v_head_dim, (const __nv_bfloat16*)o.gate, o.gate_mode, o.out_f32,
-                                                                            o.sinks, n_heads, o.sigmoid);
+                                                                            o.sinks, n_heads, o.sigmoid, p.out_pitch);
         TL_LAUNCH_CHECK();
     }
     return TL_OK;

@@ -69,6 +69,7 @@ struct MmaParams {
     int bias_cols;              // row split: the bias of so many distances (from 0) is tabulated in shared memory per head of the tile
     int n_v_heads;              // value heads of v_pages; key head j goes with value head j % n_v_heads
     int out_f32;                // 1: out holds float32
+    long long out_pitch;        // elements between two tokens' results
     float cap_log2;             // softcap * log2(e); 0: scores are not capped
     float scale_over_cap;       // scale / softcap
     const float* sinks;         // [n_heads] or null (natural-log scale, as stored)
@@ -463,7 +464,8 @@ __global__ void __launch_bounds__(NT, KEY_SPLIT ? 4 : 2) attention_mma_kernel(co
             const int tok = qs + tok0 + warp * p.tpw + rr / ng;
             const int head = kvh * p.group + g0 + rr % ng;
             const size_t row = (size_t)tok * p.n_heads + head;
-            __nv_bfloat16* dst = p.out + row * dv;
+            const size_t out_at = EXT ? (size_t)tok * p.out_pitch + (size_t)head * dv : row * dv;
+            __nv_bfloat16* dst = p.out + out_at;
             if (EXT && !SIG && p.sinks != nullptr) {
                 // one more term of the denominator, without a value: everything is rescaled to max(m, sink)
                 const float sink2 = p.sinks[head] * LOG2E;
@@ -484,7 +486,7 @@ __global__ void __launch_bounds__(NT, KEY_SPLIT ? 4 : 2) attention_mma_kernel(co
                     a *= gv.x;
                     c *= gv.y;
                 }
-                if (EXT && p.out_f32) *reinterpret_cast<float2*>(reinterpret_cast<float*>(p.out) + row * dv + nt * 8 + 2 * t) = make_float2(a, c);
+                if (EXT && p.out_f32) *reinterpret_cast<float2*>(reinterpret_cast<float*>(p.out) + out_at + nt * 8 + 2 * t) = make_float2(a, c);
                 else *reinterpret_cast<unsigned*>(dst + nt * 8 + 2 * t) = pack_bf16(a, c);
             }
         }
@@ -540,8 +542,9 @@ __global__ void __launch_bounds__(NT, KEY_SPLIT ? 4 : 2) attention_mma_kernel(co
             float v = SIG ? num : den > 0.f ? num / den : 0.f;
             if (EXT && p.gate_mode == 1) v *= __bfloat162float(p.gate[row]);
             else if (EXT && p.gate_mode == 2) v *= __bfloat162float(p.gate[row * dv + d]);
-            if (EXT && p.out_f32) reinterpret_cast<float*>(p.out)[row * dv + d] = v;
-            else p.out[row * dv + d] = __float2bfloat16_rn(v);
+            const size_t out_at = EXT ? (size_t)tok * p.out_pitch + (size_t)head * dv : row * dv;
+            if (EXT && p.out_f32) reinterpret_cast<float*>(p.out)[out_at + d] = v;
+            else p.out[out_at + d] = __float2bfloat16_rn(v);
         } else {
             p.part_o[(row * p.n_splits + split) * dv + d] = num;
             if (d == 0) {
@@ -559,7 +562,8 @@ constexpr int MERGE_MAX_SPLITS = 256;
 __global__ void merge_partials_kernel(const float* __restrict__ part_o, const float* __restrict__ part_ml,
                                       __nv_bfloat16* __restrict__ out, int n_splits, int head_dim,
                                       const __nv_bfloat16* __restrict__ gate = nullptr, int gate_mode = 0, int out_f32 = 0,
-                                      const float* __restrict__ sinks = nullptr, int n_heads = 1, int sigmoid = 0) {
+                                      const float* __restrict__ sinks = nullptr, int n_heads = 1, int sigmoid = 0,
+                                      long long out_pitch = 0) {
     __shared__ float wgt[MERGE_MAX_SPLITS];
     __shared__ float red[2];
     const size_t row = blockIdx.x;
@@ -589,8 +593,9 @@ __global__ void merge_partials_kernel(const float* __restrict__ part_o, const fl
         float v = num * inv;
         if (gate_mode == 1) v *= __bfloat162float(gate[row]);
         else if (gate_mode == 2) v *= __bfloat162float(gate[row * head_dim + d]);
-        if (out_f32) reinterpret_cast<float*>(out)[row * head_dim + d] = v;
-        else out[row * head_dim + d] = __float2bfloat16_rn(v);
+        const size_t out_at = (out_pitch > 0 ? row / n_heads * out_pitch + row % n_heads * head_dim : row * head_dim) + d;
+        if (out_f32) reinterpret_cast<float*>(out)[out_at] = v;
+        else out[out_at] = __float2bfloat16_rn(v);
     }
 }
 
@@ -716,7 +721,7 @@ extern "C" int tl_paged_attention_mma(const void* q, const void* k_pages, const 
     p.scale_log2 = scale * LOG2E;
     p.part_o = workspace;
     p.part_ml = workspace ? workspace + (size_t)n_tokens * n_heads * pl.n_splits * head_dim : nullptr;
-    p.hd = p.dv = head_dim; p.shared_kv = 0; p.keep_first = 0; p.rel = nullptr; p.bucket = nullptr; p.n_bucket = 0; p.n_v_heads = n_kv_heads; p.out_f32 = 0;
+    p.hd = p.dv = head_dim; p.shared_kv = 0; p.keep_first = 0; p.rel = nullptr; p.bucket = nullptr; p.n_bucket = 0; p.n_v_heads = n_kv_heads; p.out_f32 = 0; p.out_pitch = 0;
     p.gate = nullptr; p.gate_mode = 0; p.bias_cols = 0; p.cap_log2 = 0.f; p.scale_over_cap = 0.f; p.sinks = nullptr;
     p.chunk = 0; p.score_bias = nullptr;
 
@@ -756,6 +761,7 @@ struct TlAttentionOptions {
     int chunk;              // 0: none; a query sees keys of its own run of so many positions; not together with a window
     int sigmoid;            // 1: weights are sigmoid(score + score_bias[head]), not normalised; not together with sinks or rel
     const float* score_bias;   // [n_heads] or null; sigmoid only
+    long long out_pitch;       // elements between two tokens' results; 0: n_heads * v_head_dim
 };
 
 // 1 if the extended form takes keys of head_dim and values of v_head_dim elements, else 0.
@@ -793,6 +799,7 @@ extern "C" int tl_paged_attention_mma_ex(const void* q, const void* k_pages, con
     if (v_pages == k_pages && dv > head_dim) return TL_BAD_SIZE;
     if (o.v_stride != 0 && !(v_pages == k_pages && o.v_stride == head_dim)) return TL_BAD_SIZE;
     if (o.softcap < 0.f || (o.softcap > 0.f && o.rel != nullptr)) return TL_BAD_SIZE;
+    if (o.out_pitch < 0 || o.out_pitch % 2 != 0) return TL_BAD_ALIGN;                 // (results leave in pairs)
     if (o.chunk < 0 || (o.chunk > 0 && (window > 0 || o.rel != nullptr)) || (o.sigmoid && (o.sinks != nullptr || o.rel != nullptr)) ||
         (o.score_bias != nullptr && !o.sigmoid))
         return TL_BAD_SIZE;
@@ -825,6 +832,7 @@ extern "C" int tl_paged_attention_mma_ex(const void* q, const void* k_pages, con
     p.cap_log2 = o.softcap > 0.f ? o.softcap * LOG2E : 0.f;
     p.scale_over_cap = o.softcap > 0.f ? scale / o.softcap : 0.f;
     p.sinks = o.sinks;
+    p.out_pitch = o.out_pitch > 0 ? o.out_pitch : (long long)n_heads * dv;
     p.chunk = o.chunk; p.score_bias = o.score_bias;
     // distances a row-split CTA meets inside its window (all of them when there is no window), as far as
     // 20 KB of shared memory hold them for the heads of a tile
@@ -848,7 +856,8 @@ extern "C" int tl_paged_attention_mma_ex(const void* q, const void* k_pages, con
     if (rc != TL_OK) return rc;
     if (pl.n_splits > 1) {
         merge_partials_kernel<<<dim3((unsigned)n_tokens * (unsigned)n_heads), dim3(dv >= 128 ? 128u : 64u), 0, s>>>(
-            p.part_o, p.part_ml, p.out, pl.n_splits, dv, p.gate, p.gate_mode, p.out_f32, p.sinks, n_heads, o.sigmoid);
+            p.part_o, p.part_ml, p.out, pl.n_splits, dv, p.gate, p.gate_mode, p.out_f32, p.sinks, n_heads, o.sigmoid,
+            p.out_pitch);
         TL_LAUNCH_CHECK();
     }
     return TL_OK;

@@ -7,11 +7,12 @@
 //                    i + rot/2) or made a unit vector per head, then scaled.
 // linear_recurrence: per head a dk x dv matrix S in float32 that every token updates and reads:
 //                      fixed decay:  S <- d_h S + k v^T
-//                      delta rule:   S <- g S;  u = beta (v - S^T k);  S <- S + k u^T
+//                      delta rule:   S <- g S;  u = beta (v - S^T k);  S <- S + k u^T   (g: a number per head, or one per
+//                                    head and key coordinate, each acting on its own row of S)
 //                    and o = S^T q.  Tokens are walked in order, so a result does not depend on how
 //                    a request was cut into portions.
 // head_norm_gate:    every head of o divided by its root mean square, times a weight shared by the
-//                    heads (or none), times silu(gate).
+//                    heads (or none), times silu(gate) or sigmoid(gate).
 //
 // All arithmetic is float32; inputs that come from a product may be bfloat16 and may be column
 // ranges of a wider row (a row pitch goes with every such pointer).  State rows may be fields of a
@@ -168,8 +169,9 @@ struct HeadNormParams {
     const void* gate;        // [T] rows of pitch ldg, H * hd columns
     long long ldg;
     const float* weight;     // [hd] or null
-    void* out;               // [T][H * hd]
-    int n_heads, head_dim;
+    void* out;               // [T] rows of pitch ldo, H * hd columns
+    long long ldo;           // pitch of out's rows
+    int n_heads, head_dim, sigmoid;
     float eps;
     long long n_rows;
 };
@@ -185,14 +187,15 @@ __global__ void __launch_bounds__(NT) head_norm_gate_kernel(const HeadNormParams
     const int h = (int)(row - t * p.n_heads);
     const float* o = p.o + (size_t)row * p.head_dim;
     const TI* g = reinterpret_cast<const TI*>(p.gate) + (size_t)t * p.ldg + (size_t)h * p.head_dim;
-    TO* out = reinterpret_cast<TO*>(p.out) + (size_t)row * p.head_dim;
+    TO* out = reinterpret_cast<TO*>(p.out) + (size_t)t * p.ldo + (size_t)h * p.head_dim;
     float ssq = 0.f;
     for (int d = lane; d < p.head_dim; d += 32) ssq = fmaf(o[d], o[d], ssq);
     const float r = rsqrtf(warp_sum(ssq) / (float)p.head_dim + p.eps);
     for (int d = lane; d < p.head_dim; d += 32) {
         float v = o[d] * r;
         if (p.weight != nullptr) v *= p.weight[d];
-        out[d] = from_float<TO>(v * silu_f(to_float(g[d])));
+        const float z = to_float(g[d]);
+        out[d] = from_float<TO>(v * (p.sigmoid ? 1.f / (1.f + expf(-z)) : silu_f(z)));
     }
 }
 
@@ -205,10 +208,11 @@ struct RecurrenceParams {
     const void* v;           // [T] rows of pitch ldv, H * dv columns
     long long ldv;
     const void* beta;        // [T] rows of pitch ldg, H columns (delta rule) or null
-    const void* gate;        // [T] rows of pitch ldg, H columns (delta rule)
-    long long ldg;
+    const void* gate;        // [T] rows of pitch ldz, H columns (delta rule) or H * dk (a decay per channel)
+    long long ldg, ldz;
+    const float* g;          // [T][H * dk]: the decays per channel themselves (DECAYS)
     const float* decay;      // [H]: the fixed decay, or (delta rule) exp(A_log)
-    const float* decay_bias; // [H] (delta rule)
+    const float* decay_bias; // [H] (delta rule), or [H * dk]
     float* state;            // [slots] rows of pitch state_pitch, each [H][dv][dk]: a column's keys lie side by side
     long long state_pitch;
     const int* q_start;
@@ -232,12 +236,16 @@ struct RecurrenceParams {
 //     delta:  S^T k and S^T q of the decayed state are g (S^T k) and g (S^T q);  u = beta (v - g S^T k);
 //             o = g (S^T q) + u (k . q)
 // with S the state before the token and k . q taken once per token when its rows arrive.  That leaves one
-// dependent chain per token (the update of S) instead of two reductions one after the other.
-template <int R, int KS, bool DELTA, typename TV>
+// dependent chain per token (the update of S) instead of two reductions one after the other.  A decay per channel is
+// applied to S first (its numbers lie in shared memory beside k and q), and both sums are taken from the decayed state.
+enum Decay : int { FIXED = 0, HEAD = 1, CHANNEL_LOGITS = 2, CHANNEL_DECAYS = 3 };
+
+template <int R, int KS, int MODE, typename TV>
 __global__ void __launch_bounds__(NT) linear_recurrence_kernel(const RecurrenceParams p) {
     extern __shared__ __align__(16) float smem[];
     grid_launch_dependents();
     grid_dependency_wait();
+    constexpr bool DELTA = MODE != FIXED, CHANNEL = MODE == CHANNEL_LOGITS || MODE == CHANNEL_DECAYS;
     constexpr int SLOT = R + 4;                          // a slice in shared memory
     constexpr int PITCH = KS * SLOT;
     constexpr int COLS = 4 * (32 / KS);                  // columns of a CTA
@@ -258,6 +266,7 @@ __global__ void __launch_bounds__(NT) linear_recurrence_kernel(const RecurrenceP
     float* sg = sv + RC_TOKENS * COLS;                  // [RC_TOKENS]: the token's decay
     float* sb = sg + RC_TOKENS;                         // [RC_TOKENS]: the token's beta
     float* skq = sb + RC_TOKENS;                        // [RC_TOKENS]: k . q
+    float* sd = skq + RC_TOKENS;                        // [RC_TOKENS][PITCH]: a decay per channel (CHANNEL only)
     float* st = p.state + (size_t)p.state_slot[b] * p.state_pitch + ((size_t)h * p.dv + (live ? j : 0)) * p.dk;
     float S[R];
     const bool fresh = p.fresh[b] != 0;
@@ -267,7 +276,7 @@ __global__ void __launch_bounds__(NT) linear_recurrence_kernel(const RecurrenceP
         S[r] = (!fresh && live && i < p.dk) ? st[i] : 0.f;
     }
     const float fixed = DELTA ? 0.f : p.decay[h];
-    const float rate = DELTA ? p.decay[h] : 0.f, dbias = DELTA ? p.decay_bias[h] : 0.f;
+    const float rate = DELTA && MODE != CHANNEL_DECAYS ? p.decay[h] : 0.f, dbias = MODE == HEAD ? p.decay_bias[h] : 0.f;
     const TV* v = reinterpret_cast<const TV*>(p.v);
     const int qk_row = p.G * p.dk;
     // a warp brings whole rows (tokens warp, warp + 4, ...), a lane the places lane, lane + 32, ... of each: which
@@ -279,7 +288,7 @@ __global__ void __launch_bounds__(NT) linear_recurrence_kernel(const RecurrenceP
         const int x = lane + 32 * it, sl = x / SLOT, r = x - sl * SLOT, d = sl * R + r;
         coord[it] = (x < PITCH && r < R && d < p.dk) ? d : -1;
     }
-    float fq[TPW * XN], fk[TPW * XN], fv[V_EACH], fa = 0.f, fb = 0.f;
+    float fq[TPW * XN], fk[TPW * XN], fd[CHANNEL ? TPW * XN : 1], fv[V_EACH], fa = 0.f, fb = 0.f;
     // the rows of the 16 tokens from t0 on, into registers (zeros past the portion's end)
     auto fetch = [&](int t0) {
         const int n = min(len - t0, RC_TOKENS);
@@ -292,6 +301,11 @@ __global__ void __launch_bounds__(NT) linear_recurrence_kernel(const RecurrenceP
                 const bool in = tt < n && coord[it] >= 0;
                 fq[w * XN + it] = in ? p.q[row + coord[it]] : 0.f;
                 fk[w * XN + it] = in ? p.k[row + coord[it]] : 0.f;
+                if (MODE == CHANNEL_DECAYS)
+                    fd[w * XN + it] = in ? p.g[((size_t)(start + t0 + tt) * p.H + h) * p.dk + coord[it]] : 0.f;
+                if (MODE == CHANNEL_LOGITS)
+                    fd[w * XN + it] = in ? to_float(reinterpret_cast<const TV*>(p.gate)[(size_t)(start + t0 + tt) * p.ldz + (size_t)h * p.dk + coord[it]])
+                                               + p.decay_bias[(size_t)h * p.dk + coord[it]] : 0.f;
             }
         }
 #pragma unroll
@@ -300,9 +314,9 @@ __global__ void __launch_bounds__(NT) linear_recurrence_kernel(const RecurrenceP
             fv[i] = (tt < n && col < p.dv) ? to_float(v[(size_t)(start + t0 + tt) * p.ldv + (size_t)h * p.dv + col]) : 0.f;
         }
         if (DELTA && threadIdx.x < n) {
-            const size_t at = (size_t)(start + t0 + threadIdx.x) * p.ldg + h;
-            fa = to_float(reinterpret_cast<const TV*>(p.gate)[at]);
-            fb = to_float(reinterpret_cast<const TV*>(p.beta)[at]);
+            const size_t t = (size_t)(start + t0 + threadIdx.x);
+            if (MODE == HEAD) fa = to_float(reinterpret_cast<const TV*>(p.gate)[t * p.ldz + h]);
+            fb = to_float(reinterpret_cast<const TV*>(p.beta)[t * p.ldg + h]);
         }
     };
     fetch(0);
@@ -319,6 +333,11 @@ __global__ void __launch_bounds__(NT) linear_recurrence_kernel(const RecurrenceP
                 if (x < PITCH) {
                     sq[tt * PITCH + x] = fq[w * XN + it];
                     sk[tt * PITCH + x] = fk[w * XN + it];
+                    if (MODE == CHANNEL_DECAYS) sd[tt * PITCH + x] = fd[w * XN + it];
+                    if (MODE == CHANNEL_LOGITS && coord[it] >= 0) {
+                        const float a = fd[w * XN + it];
+                        sd[tt * PITCH + x] = tt < n ? expf(-rate * (a > 20.f ? a : log1pf(expf(a)))) : 0.f;
+                    }
                 }
                 acc = fmaf(fq[w * XN + it], fk[w * XN + it], acc);
             }
@@ -329,9 +348,11 @@ __global__ void __launch_bounds__(NT) linear_recurrence_kernel(const RecurrenceP
         for (int i = 0; i < V_EACH; ++i)
             if (threadIdx.x + i * NT < RC_TOKENS * COLS) sv[threadIdx.x + i * NT] = fv[i];
         if (DELTA && threadIdx.x < n) {
-            const float a = fa + dbias;
-            const float soft = a > 20.f ? a : log1pf(expf(a));
-            sg[threadIdx.x] = expf(-rate * soft);
+            if (MODE == HEAD) {
+                const float a = fa + dbias;
+                const float soft = a > 20.f ? a : log1pf(expf(a));
+                sg[threadIdx.x] = expf(-rate * soft);
+            }
             sb[threadIdx.x] = 1.f / (1.f + expf(-fb));
         }
         __syncthreads();
@@ -340,6 +361,17 @@ __global__ void __launch_bounds__(NT) linear_recurrence_kernel(const RecurrenceP
             const float4* kt = reinterpret_cast<const float4*>(sk + tt * PITCH + s * SLOT);
             const float4* qt = reinterpret_cast<const float4*>(sq + tt * PITCH + s * SLOT);
             const float vt = sv[tt * COLS + jl], kq = skq[tt];
+            if (CHANNEL) {
+                const float4* gt = reinterpret_cast<const float4*>(sd + tt * PITCH + s * SLOT);
+#pragma unroll
+                for (int r = 0; r < R / 4; ++r) {
+                    const float4 gv = gt[r];
+                    S[4 * r] *= gv.x;
+                    S[4 * r + 1] *= gv.y;
+                    S[4 * r + 2] *= gv.z;
+                    S[4 * r + 3] *= gv.w;
+                }
+            }
             float4 kv[R / 4];
             float d0 = 0.f, d1 = 0.f, d2 = 0.f, d3 = 0.f, o0 = 0.f, o1 = 0.f, o2 = 0.f, o3 = 0.f;
 #pragma unroll
@@ -364,7 +396,17 @@ __global__ void __launch_bounds__(NT) linear_recurrence_kernel(const RecurrenceP
                 if (DELTA) dot += __shfl_xor_sync(0xffffffffu, dot, off);
             }
             float o;
-            if (DELTA) {
+            if (CHANNEL) {
+                const float u = sb[tt] * (vt - dot);
+                o = fmaf(u, kq, oq);
+#pragma unroll
+                for (int r = 0; r < R / 4; ++r) {
+                    S[4 * r] = fmaf(kv[r].x, u, S[4 * r]);
+                    S[4 * r + 1] = fmaf(kv[r].y, u, S[4 * r + 1]);
+                    S[4 * r + 2] = fmaf(kv[r].z, u, S[4 * r + 2]);
+                    S[4 * r + 3] = fmaf(kv[r].w, u, S[4 * r + 3]);
+                }
+            } else if (DELTA) {
                 const float gt = sg[tt];
                 const float u = sb[tt] * (vt - gt * dot);
                 o = fmaf(u, kq, gt * oq);
@@ -393,6 +435,14 @@ __global__ void __launch_bounds__(NT) linear_recurrence_kernel(const RecurrenceP
         const int i = s * R + r;
         if (live && i < p.dk) st[i] = S[r];
     }
+}
+
+cudaError_t launch_recurrence(void (*kernel)(const RecurrenceParams), dim3 grid, dim3 block, size_t smem, cudaStream_t s, const RecurrenceParams& p) {
+    if (smem > 48 * 1024) {        // (keys of more than 128 with a decay per channel)
+        const cudaError_t e = cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+        if (e != cudaSuccess) return e;
+    }
+    return tl_launch(kernel, grid, block, smem, s, p);
 }
 
 }  // namespace
@@ -452,20 +502,24 @@ extern "C" int tl_recurrence_prep(const void* x, int in_dtype, long long ldx, fl
 }
 
 // q, k: float32 [n_tokens][qk_heads * dk]; v: rows of pitch ldv, heads * dv columns; state: float32, per slot a row of
-// pitch state_pitch holding [heads][dv][dk] (the matrix of a head with a column's keys side by side); out: float32 [n_tokens][heads * dv].  delta == 0: decay is [heads], the
-// fixed decay.  delta != 0: beta and gate are rows of pitch ldg with `heads` columns (of v's dtype), decay is
-// exp(A_log) per head and decay_bias the bias inside the softplus.
+// pitch state_pitch holding [heads][dv][dk] (the matrix of a head with a column's keys side by side); out: float32 [n_tokens][heads * dv].
+// mode 0: decay is [heads], the fixed decay.  Otherwise the delta rule: beta are rows of pitch ldg with `heads` columns (of v's
+// dtype).  mode 1: gate are rows of pitch ldz with `heads` columns, decay is exp(A_log) per head and decay_bias [heads] the bias
+// inside the softplus.  mode 2: gate has heads * dk columns and decay_bias heads * dk numbers.  mode 3: gate is float32
+// [n_tokens][heads * dk], the decays themselves.
 extern "C" int tl_linear_recurrence(const float* q, const float* k, const void* v, int v_dtype, long long ldv, const void* beta,
-                                    const void* gate, long long ldg, const float* decay, const float* decay_bias, float* state,
+                                    long long ldg, const void* gate, long long ldz, const float* decay, const float* decay_bias, float* state,
                                     long long state_pitch, const int* q_start, const int* state_slot, const int* fresh,
-                                    float* out, int n_tokens, int n_seqs, int heads, int qk_heads, int dk, int dv, int delta,
+                                    float* out, int n_tokens, int n_seqs, int heads, int qk_heads, int dk, int dv, int mode,
                                     void* stream) {
     if (n_tokens <= 0 || n_seqs <= 0) return TL_OK;
     if (heads <= 0 || qk_heads <= 0 || heads % qk_heads != 0 || dk <= 0 || dk > 256 || dv <= 0 || n_seqs > 65535 || heads > 65535)
         return TL_BAD_SIZE;
-    if (decay == nullptr || (delta && (beta == nullptr || gate == nullptr || decay_bias == nullptr))) return TL_BAD_SIZE;
+    if (mode < FIXED || mode > CHANNEL_DECAYS || (mode != CHANNEL_DECAYS && decay == nullptr)) return TL_BAD_SIZE;
+    if (mode != FIXED && (beta == nullptr || gate == nullptr || (mode != CHANNEL_DECAYS && decay_bias == nullptr))) return TL_BAD_SIZE;
     RecurrenceParams p;
-    p.q = q; p.k = k; p.v = v; p.ldv = ldv; p.beta = beta; p.gate = gate; p.ldg = ldg; p.decay = decay; p.decay_bias = decay_bias;
+    p.q = q; p.k = k; p.v = v; p.ldv = ldv; p.beta = beta; p.gate = gate; p.ldg = ldg; p.ldz = ldz;
+    p.g = mode == CHANNEL_DECAYS ? (const float*)gate : nullptr; p.decay = decay; p.decay_bias = decay_bias;
     p.state = state; p.state_pitch = state_pitch; p.q_start = q_start; p.state_slot = state_slot; p.fresh = fresh; p.out = out;
     p.H = heads; p.G = qk_heads; p.dk = dk; p.dv = dv;
     // slices of the key size per column (TORCHLLMS_B200_REC_SLICES=4|8|16 overrides the choice, for comparisons), and a
@@ -480,12 +534,13 @@ extern "C" int tl_linear_recurrence(const float* q, const float* k, const void* 
     const int share = (dk + ks - 1) / ks;
     const int rows = share <= 8 ? 8 : share <= 12 ? 12 : share <= 16 ? 16 : share <= 24 ? 24 : 32;
     const int cols = 4 * (32 / ks);
-    const size_t smem = ((size_t)2 * RC_TOKENS * ks * (rows + 4) + RC_TOKENS * cols + 3 * RC_TOKENS) * sizeof(float);
+    const size_t smem = ((size_t)(mode >= CHANNEL_LOGITS ? 3 : 2) * RC_TOKENS * ks * (rows + 4) + RC_TOKENS * cols + 3 * RC_TOKENS) * sizeof(float);
     const dim3 grid((dv + cols - 1) / cols, heads, n_seqs), block(NT);
     cudaStream_t s = (cudaStream_t)stream;
+#define TL_REC_MODE(R, KS, MODE, TV) launch_recurrence(linear_recurrence_kernel<R, KS, MODE, TV>, grid, block, smem, s, p)
 #define TL_REC(R, KS, TV)                                                                                           \
-    (delta ? tl_launch(linear_recurrence_kernel<R, KS, true, TV>, grid, block, smem, s, p)                          \
-           : tl_launch(linear_recurrence_kernel<R, KS, false, TV>, grid, block, smem, s, p))
+    (mode == FIXED ? TL_REC_MODE(R, KS, FIXED, TV) : mode == HEAD ? TL_REC_MODE(R, KS, HEAD, TV)                     \
+     : mode == CHANNEL_LOGITS ? TL_REC_MODE(R, KS, CHANNEL_LOGITS, TV) : TL_REC_MODE(R, KS, CHANNEL_DECAYS, TV))
 #define TL_REC_SIZES(TV)                                                                                            \
     (ks == 4 ? (rows == 8 ? TL_REC(8, 4, TV) : rows <= 16 ? TL_REC(16, 4, TV) : rows == 24 ? TL_REC(24, 4, TV) : TL_REC(32, 4, TV)) \
      : ks == 8 ? (rows == 8 ? TL_REC(8, 8, TV) : rows == 12 ? TL_REC(12, 8, TV) : TL_REC(16, 8, TV))                \
@@ -494,17 +549,19 @@ extern "C" int tl_linear_recurrence(const float* q, const float* k, const void* 
     if (v_dtype == TL_BF16) return (int)TL_REC_SIZES(__nv_bfloat16);
 #undef TL_REC_SIZES
 #undef TL_REC
+#undef TL_REC_MODE
     return TL_BAD_DTYPE;
 }
 
 // o: float32 [n_tokens][n_heads * head_dim]; gate: rows of pitch ldg, n_heads * head_dim columns; weight: float32
-// [head_dim] or null; out: [n_tokens][n_heads * head_dim] of out_dtype.
+// [head_dim] or null; out: [n_tokens] rows of pitch ldo of out_dtype; sigmoid: the gate's function (0: silu).
 extern "C" int tl_head_norm_gate(const float* o, const void* gate, int gate_dtype, long long ldg, const float* weight, void* out,
-                                 int out_dtype, int n_tokens, int n_heads, int head_dim, float eps, void* stream) {
+                                 int out_dtype, long long ldo, int n_tokens, int n_heads, int head_dim, float eps, int sigmoid, void* stream) {
     if (n_tokens <= 0) return TL_OK;
     if (n_heads <= 0 || head_dim <= 0) return TL_BAD_SIZE;
     HeadNormParams p;
     p.o = o; p.gate = gate; p.ldg = ldg; p.weight = weight; p.out = out; p.n_heads = n_heads; p.head_dim = head_dim; p.eps = eps;
+    p.ldo = ldo; p.sigmoid = sigmoid;
     p.n_rows = (long long)n_tokens * n_heads;
     const dim3 grid((unsigned)((p.n_rows + NT / 32 - 1) / (NT / 32))), block(NT);
     cudaStream_t s = (cudaStream_t)stream;

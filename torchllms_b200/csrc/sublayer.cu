@@ -2,6 +2,7 @@
 //
 // embed_positions:  h[t] = table[id[t]] * scale + positions[p[t]]       (float32 stream; optionally
 //                   the same rows in bfloat16 for the first product)
+// embed_pairs:      h[t] = table[id[t]] + a row chosen by the token and the one before it
 // stream_rows:      the float32 stream in bfloat16
 // norm_add:         d = sum of delta's planes;  h[t] += d / sqrt(mean(d^2) + eps) * w   (float32),
 //                   and the new h[t] in bfloat16 for the sublayer that reads the stream next
@@ -56,6 +57,37 @@ __global__ void embed_positions_kernel(const int* __restrict__ ids, const int* _
         if (pos != nullptr) v += to_float(pos[d]);
         out[(size_t)t * dim + d] = v;
         if (rows_out != nullptr) rows_out[(size_t)t * dim + d] = __float2bfloat16_rn(v);
+    }
+}
+
+// h[t] = table[id[t]] + pair_rows[(id[t - 1] * mul_prev + id[t] * mul_cur) mod buckets]; a portion's first token finds the
+// token before it in last[slot], and takes row `buckets` at a request's start.  The CTA of that token also leaves the
+// portion's last token there: it is the only one that reads or writes the slot.
+template <typename T>
+__global__ void embed_pairs_kernel(const int* __restrict__ ids, const T* __restrict__ table, const T* __restrict__ pair_rows,
+                                   int* __restrict__ last, const int* __restrict__ seq_of_token, const int* __restrict__ q_start,
+                                   const int* __restrict__ state_slot, const int* __restrict__ fresh, long long mul_prev,
+                                   long long mul_cur, int buckets, float* __restrict__ out, int dim, int vocab) {
+    grid_launch_dependents();
+    grid_dependency_wait();
+    const int t = blockIdx.x, b = seq_of_token[t];
+    int id = ids[t];
+    (void)TL_CHECK(id >= 0 && id < vocab, TL_DBG_TOKEN_ID);
+    id = id < 0 ? 0 : (id >= vocab ? vocab - 1 : id);   // the host rejects such ids; stay in bounds anyway
+    const bool first = t == q_start[b];
+    int row = buckets;
+    if (!first || fresh[b] == 0) {
+        const long long before = first ? last[state_slot[b]] : ids[t - 1];
+        long long r = (before * mul_prev + (long long)id * mul_cur) % buckets;
+        if (r < 0) r += buckets;
+        row = (int)r;
+    }
+    const T* a = table + (size_t)id * dim;
+    const T* p = pair_rows + (size_t)row * dim;
+    for (int d = threadIdx.x; d < dim; d += blockDim.x) out[(size_t)t * dim + d] = to_float(a[d]) + to_float(p[d]);
+    if (first) {
+        __syncthreads();                                 // every thread has read the slot
+        if (threadIdx.x == 0) last[state_slot[b]] = ids[q_start[b + 1] - 1];
     }
 }
 
@@ -412,6 +444,23 @@ extern "C" int tl_embed_positions(const int* ids, const int* positions, const vo
     else
         return TL_BAD_DTYPE;
     return (int)e;
+}
+
+// table: [vocab][dim], pair_rows: [buckets + 1][dim], both of table_dtype; last: int32 [slots]; out: float32 [n_tokens][dim].
+extern "C" int tl_embed_pairs(const int* ids, const void* table, const void* pair_rows, int table_dtype, int* last,
+                              const int* seq_of_token, const int* q_start, const int* state_slot, const int* fresh, long long mul_prev,
+                              long long mul_cur, int buckets, float* out, int n_tokens, int dim, int vocab, void* stream) {
+    if (n_tokens <= 0) return TL_OK;
+    if (dim <= 0 || vocab <= 0 || buckets <= 0 || last == nullptr) return TL_BAD_SIZE;
+    cudaStream_t s = (cudaStream_t)stream;
+    if (table_dtype == TL_F32)
+        return (int)tl_launch(embed_pairs_kernel<float>, dim3(n_tokens), dim3(row_threads(dim)), 0, s, ids, (const float*)table,
+                              (const float*)pair_rows, last, seq_of_token, q_start, state_slot, fresh, mul_prev, mul_cur, buckets, out, dim, vocab);
+    if (table_dtype == TL_BF16)
+        return (int)tl_launch(embed_pairs_kernel<__nv_bfloat16>, dim3(n_tokens), dim3(row_threads(dim)), 0, s, ids,
+                              (const __nv_bfloat16*)table, (const __nv_bfloat16*)pair_rows, last, seq_of_token, q_start, state_slot, fresh,
+                              mul_prev, mul_cur, buckets, out, dim, vocab);
+    return TL_BAD_DTYPE;
 }
 
 extern "C" int tl_stream_rows(const float* h, void* out, long long n, void* stream) {

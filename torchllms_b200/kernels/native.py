@@ -151,7 +151,7 @@ class NativeOps:
     # ------------------------------------------------------------ libraries
     def prepare(self, dtype: torch.dtype, sampling: bool = True) -> None:
         """Compile, side by side, what a model of this dtype will call."""
-        names = ["elementwise", "sublayer", "rope", "attention", "gemm_simt", "recurrent", "moe", "matrix_state", "stream_sum"]
+        names = ["elementwise", "sublayer", "rope", "attention", "gemm_simt", "recurrent", "moe", "matrix_state", "stream_sum", "conv_mixers"]
         if dtype == torch.bfloat16:
             names += ["attention_mma", "attention_decode", "gemm_tcgen05"]
         if sampling:
@@ -227,6 +227,31 @@ class NativeOps:
         rc = self._lib("elementwise").tl_embed(_ptr(token_ids), _ptr(table), _DT[table.dtype], _ptr(out),
                                               n, dim, vocab, _stream())
         _check(rc, "embed")
+        self.launches += 1
+        return out
+
+    @_timed
+    def embed_pairs(self, token_ids: torch.Tensor, table: torch.Tensor, pair_rows: torch.Tensor, last: torch.Tensor,
+                    seq_of_token: torch.Tensor, q_start: torch.Tensor, state_slot: torch.Tensor, fresh: torch.Tensor, *,
+                    mul_prev: int, mul_cur: int) -> torch.Tensor:
+        """The float32 stream ``table[id] + pair_rows[(previous id * mul_prev + id * mul_cur) mod buckets]``, where ``pair_rows``
+        has ``buckets + 1`` rows and a request's first token takes the last one.  ``last`` (int32 ``[slots, 1]``) holds every
+        request's last token at ``state_slot[b]``: read for the first token of a portion and left as the portion leaves it."""
+        for t, name in ((token_ids, "token_ids"), (seq_of_token, "seq_of_token"), (q_start, "q_start"), (state_slot, "state_slot"),
+                        (fresh, "fresh"), (last, "last tokens")):
+            _cuda_contig(t, name, torch.int32)
+        _cuda_contig(table, "embedding table")
+        _cuda_contig(pair_rows, "pair rows", table.dtype)
+        _need(table.dtype in _DT and table.dim() == 2 and pair_rows.dim() == 2 and pair_rows.shape[0] > 1
+              and pair_rows.shape[1] == table.shape[1], "embed_pairs: table [vocab, dim] and pair rows [buckets + 1, dim] of one dtype")
+        n, (vocab, dim) = token_ids.numel(), table.shape
+        _need(seq_of_token.numel() == n and q_start.numel() > state_slot.numel() >= 1 and fresh.numel() == state_slot.numel(),
+              "embed_pairs: one request per token; q_start, state_slot and fresh must cover every request")
+        out = torch.empty((n, dim), dtype=torch.float32, device=table.device)
+        rc = self._lib("sublayer").tl_embed_pairs(
+            _ptr(token_ids), _ptr(table), _ptr(pair_rows), _DT[table.dtype], _ptr(last), _ptr(seq_of_token), _ptr(q_start), _ptr(state_slot),
+            _ptr(fresh), ctypes.c_longlong(mul_prev), ctypes.c_longlong(mul_cur), pair_rows.shape[0] - 1, _ptr(out), n, dim, vocab, _stream())
+        _check(rc, "embed_pairs")
         self.launches += 1
         return out
 
@@ -935,6 +960,96 @@ class NativeOps:
         self.launches += 2 if (max_q_len > 8 and taps > 1) else 1
         return out
 
+    @staticmethod
+    def _planes_view(t: torch.Tensor, width: int, name: str):
+        """Rows ``[T, width]`` or float32 partial sums ``[splits, T, width]`` that may be a column range of wider rows:
+        ``(splits, the planes' distance, the rows' pitch)`` in elements."""
+        _need(t.is_cuda and t.dim() in (2, 3) and t.dtype in _DT and t.shape[-1] == width and t.stride(-1) == 1,
+              f"{name} must be [tokens, {width}] or partial sums of it on the GPU, columns side by side")
+        splits = t.shape[0] if t.dim() == 3 else 1
+        _need(splits == 1 or t.dtype == torch.float32, "partial sums must be float32")
+        return splits, ctypes.c_longlong(t.stride(0) if splits > 1 else 0), ctypes.c_longlong(t.stride(-2))
+
+    def _conv_args(self, w_conv: torch.Tensor, state: Optional[torch.Tensor], columns: int):
+        """``(taps pointer, number of taps, state pointer, the slots' pitch)`` of a convolution over so many channels."""
+        _cuda_contig(w_conv, "convolution taps", torch.float32)
+        _need(w_conv.dim() == 2 and w_conv.shape[0] == columns and 1 <= w_conv.shape[1] <= 8, f"convolution taps must be [{columns}, taps], at most 8 taps")
+        taps, pitch = w_conv.shape[1], ctypes.c_longlong(0)
+        if taps > 1:
+            _need(state is not None, "a convolution of several taps keeps state")
+            pitch = self._state_view(state, (taps - 1) * columns, "convolution state")
+        return _ptr(w_conv), taps, _ptr(state if taps > 1 else None), pitch
+
+    @_timed
+    def conv_rope_store(self, proj: torch.Tensor, w_conv: torch.Tensor, state: Optional[torch.Tensor], positions: torch.Tensor,
+                        table: torch.Tensor, q_start: torch.Tensor, state_slot: torch.Tensor, fresh: torch.Tensor, *, n_seqs: int,
+                        max_q_len: int, n_q_heads: int, n_k_heads: int, head_dim: int, v_head_dim: int, rot_dims: int, n_extra: int,
+                        k_pages: torch.Tensor, v_pages: torch.Tensor, slot_mapping: torch.Tensor, page_size: int, out_dtype: torch.dtype,
+                        extra_scale: float = 1.0):
+        """What follows a stacked projection ``[q heads | k heads | v heads | extra]`` (``[T, width]`` or float32 partial sums,
+        a column range of wider rows will do) where every channel of q, k and v passes a causal convolution over time
+        first (``w_conv`` float32 ``[channels, taps]``; ``state`` as in :meth:`short_conv`): then, as :meth:`rope_store` does in
+        the half pairing, rotation, the page writes, ``q [T, n_q_heads, head_dim]`` and ``extra_scale * sigmoid(extra)``."""
+        cols = (n_q_heads + n_k_heads) * head_dim + n_k_heads * v_head_dim
+        splits, plane, ld = self._planes_view(proj, cols + n_extra, "projection")
+        conv = self._conv_args(w_conv, state, cols)
+        self._seq_index(q_start, state_slot, fresh, n_seqs)
+        _cuda_contig(positions, "positions", torch.int32)
+        _cuda_contig(table, "rotary table", torch.float32)
+        _cuda_contig(slot_mapping, "slot_mapping", torch.int32)
+        _cuda_contig(k_pages, "k_pages", out_dtype)
+        _cuda_contig(v_pages, "v_pages", out_dtype)
+        _need(out_dtype in _DT and (out_dtype == proj.dtype or proj.dtype == torch.float32), "conv_rope_store cannot widen bfloat16 input")
+        _need(0 <= rot_dims <= head_dim and rot_dims % 2 == 0, "rot_dims must be even and at most head_dim")
+        _need(table.dim() == 3 and table.shape[2] == 2 and (rot_dims == 0 or table.shape[1] == rot_dims // 2),
+              "rotary table must be [positions, rot_dims / 2, 2]")
+        T = proj.shape[-2]
+        _need(positions.numel() == T and slot_mapping.numel() == T, "one position and one cache slot per token")
+        _need(k_pages.shape[1:] == (n_k_heads, page_size, head_dim) and v_pages.shape[1:] == (n_k_heads, page_size, v_head_dim)
+              and v_pages.shape[0] == k_pages.shape[0], "pages must be [pages, heads, page_size, size] for keys and for values")
+        self._debug_limit("conv_mixers", 0, k_pages.shape[0])
+        q = torch.empty((T, n_q_heads, head_dim), dtype=out_dtype, device=proj.device)
+        extra = torch.empty((T, n_extra), dtype=out_dtype, device=proj.device) if n_extra else None
+        rc = self._lib("conv_mixers").tl_conv_rope_store(
+            _ptr(proj), _DT[proj.dtype], splits, plane, ld, *conv, _ptr(q_start), _ptr(state_slot), _ptr(fresh), _ptr(positions), _ptr(table),
+            _ptr(slot_mapping), _ptr(q), _ptr(extra), _ptr(k_pages), _ptr(v_pages), _DT[out_dtype], T, n_seqs, max_q_len, n_q_heads,
+            n_k_heads, head_dim, v_head_dim, rot_dims, n_extra, ctypes.c_float(extra_scale), page_size, table.shape[0], _stream())
+        _check(rc, "conv_rope_store")
+        self.launches += 2 if (max_q_len > 16 and w_conv.shape[1] > 1) else 1
+        return q, extra
+
+    @_timed
+    def delta_prep(self, proj: torch.Tensor, w_conv: torch.Tensor, state: Optional[torch.Tensor], q_start: torch.Tensor,
+                   state_slot: torch.Tensor, fresh: torch.Tensor, *, n_seqs: int, max_q_len: int, n_qk_heads: int, head_dim: int,
+                   n_v: int, n_small: int, n_low: int, low_pad: int, q_scale: float, unit_eps: float, out_dtype: torch.dtype):
+        """What a delta rule needs of a stacked projection ``[q heads | k heads | v | small | low | ...]`` (``[T, width]`` or
+        float32 partial sums, a column range of wider rows will do): q, k and v pass a causal convolution over time and
+        ``silu`` (``w_conv`` and ``state`` as in :meth:`short_conv`), every head of q and k becomes a unit vector (``x / sqrt(sum(x^2) +
+        unit_eps)``, q times ``q_scale``).  Returns ``(q, k, v, small, low)``: q and k float32 ``[T, n_qk_heads * head_dim]``, the rest
+        in ``out_dtype``, ``low`` as ``[T, low_pad]`` with zeros behind its ``n_low`` columns (``None`` without any)."""
+        n_qk = n_qk_heads * head_dim
+        _need(proj.dim() in (2, 3) and proj.shape[-1] >= 2 * n_qk + n_v + n_small + n_low, "projection rows must hold [q | k | v | small | low]")
+        splits, plane, ld = self._planes_view(proj, proj.shape[-1], "projection")
+        conv = self._conv_args(w_conv, state, 2 * n_qk + n_v)
+        self._seq_index(q_start, state_slot, fresh, n_seqs)
+        _need(out_dtype in _DT and (out_dtype == proj.dtype or proj.dtype == torch.float32), "delta_prep cannot widen bfloat16 input")
+        _need(head_dim <= 256, f"delta_prep takes heads of at most 256, got {head_dim}")
+        T, dev = proj.shape[-2], proj.device
+        q = torch.empty((T, n_qk), dtype=torch.float32, device=dev)
+        k = torch.empty_like(q)
+        v = torch.empty((T, n_v), dtype=out_dtype, device=dev)
+        small = torch.empty((T, n_small), dtype=out_dtype, device=dev)
+        low = torch.empty((T, low_pad), dtype=out_dtype, device=dev) if n_low else None
+        rc = self._lib("conv_mixers").tl_delta_prep(
+            _ptr(proj), _DT[proj.dtype], splits, plane, ld, *conv, _ptr(q_start), _ptr(state_slot), _ptr(fresh), _ptr(q), _ptr(k), _ptr(v),
+            _ptr(small), _ptr(low), _DT[out_dtype], T, n_seqs, max_q_len, n_qk_heads, head_dim, n_v, n_small, n_low, low_pad,
+            ctypes.c_float(q_scale), ctypes.c_float(unit_eps), _stream())
+        _check(rc, "delta_prep")
+        self.launches += 2 if (max_q_len > 16 and w_conv.shape[1] > 1) else 1
+        return q, k, v, small, low
+
+    DECAYS_MIN_Q = 9      # portions from which decays per channel are worked out by a kernel of their own, once per token
+
     @_timed
     def recurrence_prep(self, x: torch.Tensor, *, scale: float, n_heads: int, head_dim: int,
                         positions: Optional[torch.Tensor] = None, table: Optional[torch.Tensor] = None, rot_dims: int = 0,
@@ -973,7 +1088,8 @@ class NativeOps:
         """A matrix ``S`` (``dk x dv``, float32) per head and request that every token updates and then reads,
         ``o = S^T q``.  With ``decay`` (float32 ``[H]``): ``S <- decay_h S + k v^T``.  Otherwise the gated delta rule:
         ``S <- g S; u = beta (v - S^T k); S <- S + k u^T`` with ``beta = sigmoid(beta_logits)`` and
-        ``g = exp(-decay_rate softplus(decay_logits + decay_bias))`` (logits ``[T, H]``, the rest float32 ``[H]``).
+        ``g = exp(-decay_rate softplus(decay_logits + decay_bias))`` (logits ``[T, H]``, the rest float32 ``[H]``), or with a decay
+        per head and key coordinate: ``decay_logits`` ``[T, H * dk]`` and ``decay_bias`` ``[H * dk]``, each acting on its row of ``S``.
         ``q``, ``k``: float32 ``[T, G * dk]``, ``G`` heads each shared by ``H / G`` value heads; ``v``: ``[T, H * dv]``;
         ``state``: ``[slots, H, dv, dk]`` (a head's matrix with a column's keys side by side), read (zeros where
         ``fresh``) and left updated.  Returns float32 ``[T, H * dv]``."""
@@ -990,32 +1106,43 @@ class NativeOps:
         _need(dk <= 256, f"linear_recurrence keeps a head's state in registers: key size {dk} exceeds 256")
         self._seq_index(q_start, state_slot, fresh, n_seqs)
         delta = decay is None
-        ldg = ctypes.c_longlong(0)
+        ldg = ldz = ctypes.c_longlong(0)
+        mode = 0
         if delta:
-            for t, name in ((decay_rate, "decay_rate"), (decay_bias, "decay_bias")):
-                _cuda_contig(t, name, torch.float32)
-                _need(t.numel() == H, f"{name}: one number per head")
-            ldg = self._rows_view(beta_logits, "beta_logits")
-            _need(self._rows_view(decay_logits, "decay_logits").value == ldg.value and beta_logits.shape == (T, H)
-                  and decay_logits.shape == (T, H) and beta_logits.dtype == v.dtype and decay_logits.dtype == v.dtype,
-                  "beta_logits and decay_logits must be [T, H] of v's dtype with one row pitch")
+            per_channel = decay_logits.shape == (T, H * dk) and decay_bias.numel() == H * dk
+            mode = 2 if per_channel else 1
+            _cuda_contig(decay_rate, "decay_rate", torch.float32)
+            _cuda_contig(decay_bias, "decay_bias", torch.float32)
+            _need(decay_rate.numel() == H and (per_channel or decay_bias.numel() == H), "decay_rate: one number per head; decay_bias: one per logit")
+            ldg, ldz = self._rows_view(beta_logits, "beta_logits"), self._rows_view(decay_logits, "decay_logits")
+            _need(beta_logits.shape == (T, H) and (per_channel or decay_logits.shape == (T, H)) and beta_logits.dtype == v.dtype
+                  and decay_logits.dtype == v.dtype, "beta_logits must be [T, H] and decay_logits [T, H] or [T, H * dk], of v's dtype")
+            if per_channel and max_q_len >= self.DECAYS_MIN_Q:
+                # long portions: the decays once per token (few tokens: by every CTA of the recurrence for itself)
+                decays = torch.empty((T, H * dk), dtype=torch.float32, device=q.device)
+                _check(self._lib("conv_mixers").tl_channel_decay(_ptr(decay_logits), _DT[decay_logits.dtype], ldz, _ptr(decay_rate), _ptr(decay_bias),
+                                                                 _ptr(decays), T, H * dk, dk, _stream()), "channel_decay")
+                self.launches += 1
+                mode, decay_logits = 3, decays
         else:
             _cuda_contig(decay, "decay", torch.float32)
             _need(decay.numel() == H, "decay: one number per head")
         out = torch.empty((T, H * dv), dtype=torch.float32, device=q.device)
         rc = self._lib("matrix_state").tl_linear_recurrence(
-            _ptr(q), _ptr(k), _ptr(v), _DT[v.dtype], ldv, _ptr(beta_logits), _ptr(decay_logits), ldg,
+            _ptr(q), _ptr(k), _ptr(v), _DT[v.dtype], ldv, _ptr(beta_logits), ldg, _ptr(decay_logits), ldz,
             _ptr(decay_rate if delta else decay), _ptr(decay_bias), _ptr(state), pitch, _ptr(q_start), _ptr(state_slot), _ptr(fresh),
-            _ptr(out), T, n_seqs, H, G, dk, dv, 1 if delta else 0, _stream())
+            _ptr(out), T, n_seqs, H, G, dk, dv, mode, _stream())
         _check(rc, "linear_recurrence")
         self.launches += 1
         return out
 
     @_timed
     def head_norm_gate(self, o: torch.Tensor, gate: torch.Tensor, weight: Optional[torch.Tensor], eps: float, *, head_dim: int,
-                       out_dtype: torch.dtype) -> torch.Tensor:
+                       out_dtype: torch.dtype, activation: str = "silu", out: Optional[torch.Tensor] = None) -> torch.Tensor:
         """Every head (``head_dim`` numbers) of ``o`` (float32 ``[T, H * head_dim]``) divided by its root mean square,
-        times ``weight`` (float32 ``[head_dim]``, shared by the heads; ``None``: no weight), times ``silu(gate)``."""
+        times ``weight`` (float32 ``[head_dim]``, shared by the heads; ``None``: no weight), times ``silu(gate)`` or, with
+        ``activation="sigmoid"``, ``sigmoid(gate)``.  ``out`` may be given: a column range of wider rows will do."""
+        _need(activation in ("silu", "sigmoid"), f"head_norm_gate: an output gate is 'silu' or 'sigmoid', got {activation!r}")
         _cuda_contig(o, "recurrence output", torch.float32)
         ldg = self._rows_view(gate, "gate")
         _need(o.dim() == 2 and o.shape[1] % head_dim == 0 and gate.shape == o.shape, "head_norm_gate: o and gate [T, H * head_dim]")
@@ -1023,9 +1150,13 @@ class NativeOps:
         if weight is not None:
             _cuda_contig(weight, "head norm weight", torch.float32)
             _need(weight.numel() == head_dim, "the head norm's weight has head_dim numbers")
-        out = torch.empty(o.shape, dtype=out_dtype, device=o.device)
-        rc = self._lib("matrix_state").tl_head_norm_gate(_ptr(o), _ptr(gate), _DT[gate.dtype], ldg, _ptr(weight), _ptr(out), _DT[out_dtype],
-                                                        o.shape[0], o.shape[1] // head_dim, head_dim, ctypes.c_float(eps), _stream())
+        if out is None:
+            out = torch.empty(o.shape, dtype=out_dtype, device=o.device)
+        ldo = self._rows_view(out, "head_norm_gate output")
+        _need(out.shape == o.shape and out.dtype == out_dtype, "head_norm_gate: out has o's shape and the output dtype")
+        rc = self._lib("matrix_state").tl_head_norm_gate(_ptr(o), _ptr(gate), _DT[gate.dtype], ldg, _ptr(weight), _ptr(out), _DT[out_dtype], ldo,
+                                                        o.shape[0], o.shape[1] // head_dim, head_dim, ctypes.c_float(eps),
+                                                        1 if activation == "sigmoid" else 0, _stream())
         _check(rc, "head_norm_gate")
         self.launches += 1
         return out
@@ -1588,6 +1719,8 @@ class NativeOps:
         calls fill one tensor.  ``allow_split``: False keeps every request's keys in one CTA, True lets
         the kernel split them as it sees fit; the decode kernel also takes a number of splits (above 1).
 
+        ``out`` may be a column range of wider rows for the general and the extended mma.sync kernel.
+
         The general kernel alone also takes: values of another size than keys (``v_pages``
         ``[pages, kv_heads, page_size, v_dim]``, possibly the very tensor ``k_pages``; the result is
         ``[T, H, v_dim]``), ``keep_first`` (with a window: the first so many keys of a request stay
@@ -1604,7 +1737,8 @@ class NativeOps:
         ``sigmoid(score + score_bias[h])``, ``score_bias`` float32 ``[H]`` or ``None``, not divided by the weights' sum)."""
         if keep_first or distance_bias is not None or gate is not None or v_pages.shape[-1] != q.shape[-1] \
                 or q.shape[-1] % 16 != 0 or v_pages.shape[1] != k_pages.shape[1] or out_dtype not in (None, q.dtype) \
-                or softcap or sinks is not None or value_dim or chunk or weights != "softmax":
+                or softcap or sinks is not None or value_dim or chunk or weights != "softmax" \
+                or (out is not None and not out.is_contiguous()):
             _need(impl in ("auto", "general", "mma"), "only the general and the mma.sync attention kernels take these options")
             return self._paged_attention_general(q, k_pages, v_pages, block_table, q_start, kv_len, n_seqs, max_q_len,
                                                  max_kv_len, scale, window, page_size, allow_split, n_tokens, out,
@@ -1702,7 +1836,7 @@ class NativeOps:
                     ("bucket", ctypes.c_void_p), ("n_bucket", ctypes.c_int), ("gate", ctypes.c_void_p),
                     ("gate_mode", ctypes.c_int), ("n_v_heads", ctypes.c_int), ("out_f32", ctypes.c_int),
                     ("softcap", ctypes.c_float), ("sinks", ctypes.c_void_p), ("v_stride", ctypes.c_int), ("chunk", ctypes.c_int),
-                    ("sigmoid", ctypes.c_int), ("score_bias", ctypes.c_void_p)]
+                    ("sigmoid", ctypes.c_int), ("score_bias", ctypes.c_void_p), ("out_pitch", ctypes.c_longlong)]
 
     def _paged_attention_general(self, q, k_pages, v_pages, block_table, q_start, kv_len, n_seqs, max_q_len, max_kv_len,
                                  scale, window, page_size, allow_split, n_tokens, out, keep_first, distance_bias,
@@ -1744,11 +1878,13 @@ class NativeOps:
         if out is None:
             out = torch.empty((T_all, n_heads, v_dim), dtype=out_dtype, device=q.device)
         else:
-            _cuda_contig(out, "out", out_dtype)
-            _need(out.shape == (T_all, n_heads, v_dim), "out must be [tokens, heads, v_dim]")
+            # (a column range of wider rows will do)
+            _need(out.is_cuda and out.dtype == out_dtype and out.shape == (T_all, n_heads, v_dim) and (v_dim == 1 or out.stride(2) == 1)
+                  and (n_heads == 1 or out.stride(1) == v_dim), "out must be [tokens, heads, v_dim], a token's heads side by side")
+        out_pitch = out.stride(0)
         opt = self._AttentionOptions(v_dim, int(keep_first), None, None, 0, None, 0, v_heads,
                                      1 if (out_dtype == torch.float32 and q.dtype != torch.float32) else 0,
-                                     float(softcap or 0.0), None, v_stride, int(chunk or 0), 1 if weights == "sigmoid" else 0, None)
+                                     float(softcap or 0.0), None, v_stride, int(chunk or 0), 1 if weights == "sigmoid" else 0, None, out_pitch)
         _need(not (chunk and window) and (chunk is None or chunk > 0), "attention looks back through a window or inside chunks of at least one position")
         _need(weights in ("softmax", "sigmoid") and not (weights == "sigmoid" and (sinks is not None or distance_bias is not None)),
               "attention weights are 'softmax' or 'sigmoid'; sinks and a distance bias go with softmax")
@@ -1777,7 +1913,7 @@ class NativeOps:
         n_splits, floats = ctypes.c_int(0), ctypes.c_longlong(0)
         mma_ok = (q.dtype == torch.bfloat16 and impl in ("auto", "mma") and self.use_mma_options
                   and self._lib("attention_mma").tl_attention_mma_ex_supports(head_dim, v_dim) == 1
-                  and not ((softcap or chunk) and distance_bias is not None))
+                  and not ((softcap or chunk) and distance_bias is not None) and out_pitch % 2 == 0)
         _need(impl != "mma" or mma_ok, "the mma.sync kernel takes bfloat16 and keys and values that are multiples of 8 up to 128")
         if mma_ok:
             lib = self._lib("attention_mma")
