@@ -390,11 +390,28 @@ def _looped_zusitar_config(z, vocab, max_len):
                          loop_start=z["loop"][0], loop_stop=z["loop"][1], loop_times=z["loop"][2], max_seq_len=max_len)
 
 
+# Bomotar at the same widths: every layer an attention behind short convolutions beside a delta rule with a decay per
+# channel (low-rank projections of a head's size), with a dense feed-forward and with grouped experts by turns
+BOMOTAR_SIZES = {name: dict(z, groups=4, keep_groups=2) for name, z in NUNOSUN_SIZES.items()}
+
+
+def _bomotar_config(z, vocab, max_len):
+    from torchllms_b200.models.bomotar import AttentionConfig, BomotarConfig, DeltaConfig, LayerConfig, MlpConfig, ParallelConfig, RampScaling
+    hd = z["head_dim"]
+    left = AttentionConfig(heads=z["heads"], kv_heads=z["kv_heads"], dim=hd, vdim=hd, scale=hd ** -0.5, conv=z["conv"], rot_dims=z["rot_dims"],
+                           rot_base=1000000.0, scaling=RampScaling(4.0, 8192.0, 32.0, 1.0))
+    right = DeltaConfig(heads=z["state_heads"], kv_heads=z["kv_heads"], dim=hd, vdim=hd, conv=z["conv"])
+    mlps = [MlpConfig("dense", z["ff"]), MlpConfig("moe", z["expert_ff"], experts=z["experts"], top=z["top"], groups=z["groups"], keep_groups=z["keep_groups"])]
+    layers = tuple(LayerConfig(ParallelConfig(left, right, 0.7, 0.7), mlps[i % 2]) for i in range(z["layers"]))
+    return BomotarConfig("Bomotar", vocab, z["dim"], 1e-6, 0.7, buckets=65536, mul_prev=31, mul_cur=7, layers=layers, max_seq_len=max_len)
+
+
 # design -> (its name, the table of sizes, how its configuration is made, the model it stands beside)
 DESIGNS = {"nagolix": ("Nagolix", DESIGN_SIZES, _nagolix_config, "llama"), "rakuvik": ("Rakuvik", RAKUVIK_SIZES, _rakuvik_config, "llama"),
            "nunosun": ("Nunosun", NUNOSUN_SIZES, _nunosun_config, "rakuvik"),
            "zusitar": ("Zusitar", ZUSITAR_SIZES, _zusitar_config, "rakuvik"),
-           "lagusun": ("Lagusun", LAGUSUN_SIZES, _lagusun_config, "zusitar")}
+           "lagusun": ("Lagusun", LAGUSUN_SIZES, _lagusun_config, "zusitar"),
+           "bomotar": ("Bomotar", BOMOTAR_SIZES, _bomotar_config, "nunosun")}
 
 
 def design_workload(args, peaks, design="nagolix"):
@@ -406,7 +423,8 @@ def design_workload(args, peaks, design="nagolix"):
     alternate minGRU with a dense feed-forward, differential attention with experts, minGRU with experts,
     differential attention reading the first one's keys and values with experts.  Nunosun and Zusitar stand beside
     Rakuvik, the closest model (recurrent layers, attention, experts), at the same sizes; Lagusun beside a Zusitar
-    whose layers are all attention with experts, with the same loop."""
+    whose layers are all attention with experts, with the same loop; Bomotar beside Nunosun, whose layers are an attention
+    beside a retention and a delta rule by turns."""
     import torch
     from torchllms_b200.engine.step import StepEntry
     from torchllms_b200.inference import LLM
@@ -422,7 +440,7 @@ def design_workload(args, peaks, design="nagolix"):
         hd = z["head_dim"]
         configs = {
             design: make_config(z, vocab, max_len),
-            beside: {"rakuvik": _rakuvik_config, "zusitar": _looped_zusitar_config}[beside](z, vocab, max_len),
+            beside: {"rakuvik": _rakuvik_config, "zusitar": _looped_zusitar_config, "nunosun": _nunosun_config}[beside](z, vocab, max_len),
         } if beside != "llama" else {
             design: make_config(z, vocab, max_len),
             "llama": LlamaConfig(architecture="LlamaForCausalLM", n_layers=z["layers"], dim=z["dim"], n_heads=z["heads"],
@@ -504,11 +522,12 @@ def main():
     ap.add_argument("--layers", type=int, default=SHAPE_8B["n_layers"], help="fewer layers than the shape has (named in config)")
     ap.add_argument("--batch", type=int, default=8)
     ap.add_argument("--skip-points", action="store_true", help="only the headline batch and the prefill")
-    ap.add_argument("--workload", default="decode_8b", choices=["decode_8b", "design_nagolix", "design_rakuvik", "design_nunosun", "design_zusitar", "design_lagusun"] + sorted(SERVE),
+    ap.add_argument("--workload", default="decode_8b", choices=["decode_8b", "design_nagolix", "design_rakuvik", "design_nunosun", "design_zusitar", "design_lagusun", "design_bomotar"] + sorted(SERVE),
                     help="decode_8b: the headline (default); serve_1b, long_3b: whole serving runs through LLM.generate; "
                          "design_nagolix, design_rakuvik: that design beside the Llama decoder at equal sizes; "
                          "design_nunosun, design_zusitar: that design beside Rakuvik at equal sizes; "
-                         "design_lagusun: Lagusun beside a Zusitar of attention layers")
+                         "design_lagusun: Lagusun beside a Zusitar of attention layers; "
+                         "design_bomotar: Bomotar beside Nunosun")
     ap.add_argument("--context-len", type=int, default=PROMPT_LEN,
                     help="prompt length of the decode measurements (the headline is 2,048; the prefill figure stays at 2,048)")
     ap.add_argument("--long-contexts", type=lambda t: [int(x) for x in t.split(",") if x], default=[8192, 32768],

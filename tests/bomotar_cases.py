@@ -201,9 +201,10 @@ def clear_tokens(cfg: dict, tensors, n: int, seed: int = 0, dtype: str = "bfloat
 class Expected:
     """The plain logits of a sequence and how far an engine may be from them.  In float32: 2e-4 of
     the largest logit on every logit (8e-4 at least: a wrong key, expert or state moves them by tenths).  In bfloat16
-    the yardstick is what rounding itself does to this model: the plain implementation is run a second time with
-    bfloat16 rounding of every projection and activation, and a row of the engine's logits may differ from the exact
-    ones (root mean square over the vocabulary) by three times what that emulation differs, the
+    the yardstick is what rounding itself does to this model: the plain implementation is run again with
+    bfloat16 rounding of every projection and activation, to nearest and twice up or down at random, and a row of the
+    engine's logits may differ from the exact ones (root mean square over the vocabulary) by three times what the worst
+    of these differs, the
     typical row's figure standing in where a row's own is smaller; one row in twenty may pass
     that, by half at most."""
 
@@ -211,8 +212,10 @@ class Expected:
         self.dtype = dtype
         self.logits = plain.forward(cfg, tensors, tokens).to(torch.float32).numpy()
         if dtype == "bfloat16":
-            rounded = plain.forward(cfg, tensors, tokens, rounding=torch.bfloat16).to(torch.float32).numpy()
-            noise = np.sqrt(((rounded - self.logits) ** 2).mean(-1))
+            noise = 0.0
+            for rounding in (torch.bfloat16, plain.either_way(1), plain.either_way(2)):
+                rounded = plain.forward(cfg, tensors, tokens, rounding=rounding).to(torch.float32).numpy()
+                noise = np.maximum(noise, np.sqrt(((rounded - self.logits) ** 2).mean(-1)))
             self.allowed = 3.0 * np.maximum(noise, np.median(noise))
 
     def check(self, got: np.ndarray, what: str = "") -> None:

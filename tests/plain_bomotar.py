@@ -7,7 +7,7 @@ and this file can only agree by computing the same design.
 
 ``rounding=torch.bfloat16`` rounds the results of the matrix products, of the short convolutions and
 of the activations, which the design allows in 16 bits: it shows how far 16-bit storage alone moves
-the logits.
+the logits.  A function in its place rounds as it likes (:func:`either_way`).
 """
 
 from __future__ import annotations
@@ -22,7 +22,20 @@ UNIT_EPS = 1e-6
 
 
 def _r(x: torch.Tensor, rounding) -> torch.Tensor:
-    return x if rounding is None else x.to(rounding).to(F64)
+    if rounding is None:
+        return x
+    return rounding(x) if callable(rounding) else x.to(rounding).to(F64)
+
+
+def either_way(seed: int):
+    """A rounding to bfloat16's grid that goes up or down with the probabilities of the distances: another sample of what
+    16-bit storage may do than rounding to nearest is."""
+    g = torch.Generator().manual_seed(seed)
+
+    def rounded(x: torch.Tensor) -> torch.Tensor:
+        step = torch.exp2(torch.floor(torch.log2(x.abs().clamp(min=1e-30))) - 7)
+        return torch.floor(x / step + torch.rand(x.shape, generator=g, dtype=F64)) * step
+    return rounded
 
 
 def rms(x: torch.Tensor, eps: float) -> torch.Tensor:

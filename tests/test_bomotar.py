@@ -660,7 +660,7 @@ def test_greedy_generation_through_the_scheduler(tmp_path, backend):
         kw = dict(ops=TorchOps())
     llm = LLM(folder, max_len=128, max_bsz=3, device=backend[0], precision=backend[1], page_size=page,
               max_num_batched_tokens=24, **kw)
-    prompts = [bc.tokens_for(cfg, n, seed=20 + n) for n in (3, 30, 11, 1)]
+    prompts = [bc.clear_tokens(cfg, tensors, n, seed=20 + n, dtype=backend[1]) for n in (3, 30, 11, 1)]
     results = llm.generate(prompt_token_ids=prompts, temperature=0.0, max_new_tokens=12, disable_tqdm=True)
     margin = 1e-3 if backend[1] == "float32" else 0.1
     router_margin = 1e-4 if backend[1] == "float32" else 0.03

@@ -334,9 +334,9 @@ __global__ void __launch_bounds__(NT) linear_recurrence_kernel(const RecurrenceP
                     sq[tt * PITCH + x] = fq[w * XN + it];
                     sk[tt * PITCH + x] = fk[w * XN + it];
                     if (MODE == CHANNEL_DECAYS) sd[tt * PITCH + x] = fd[w * XN + it];
-                    if (MODE == CHANNEL_LOGITS && coord[it] >= 0) {
+                    if (MODE == CHANNEL_LOGITS) {             // (zeros past dk: they multiply the state's unused places)
                         const float a = fd[w * XN + it];
-                        sd[tt * PITCH + x] = tt < n ? expf(-rate * (a > 20.f ? a : log1pf(expf(a)))) : 0.f;
+                        sd[tt * PITCH + x] = tt < n && coord[it] >= 0 ? expf(-rate * (a > 20.f ? a : log1pf(expf(a)))) : 0.f;
                     }
                 }
                 acc = fmaf(fq[w * XN + it], fk[w * XN + it], acc);
