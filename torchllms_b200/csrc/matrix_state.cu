@@ -210,7 +210,6 @@ struct RecurrenceParams {
     const void* beta;        // [T] rows of pitch ldg, H columns (delta rule) or null
     const void* gate;        // [T] rows of pitch ldz, H columns (delta rule) or H * dk (a decay per channel)
     long long ldg, ldz;
-    const float* g;          // [T][H * dk]: the decays per channel themselves (DECAYS)
     const float* decay;      // [H]: the fixed decay, or (delta rule) exp(A_log)
     const float* decay_bias; // [H] (delta rule), or [H * dk]
     float* state;            // [slots] rows of pitch state_pitch, each [H][dv][dk]: a column's keys lie side by side
@@ -238,14 +237,15 @@ struct RecurrenceParams {
 // with S the state before the token and k . q taken once per token when its rows arrive.  That leaves one
 // dependent chain per token (the update of S) instead of two reductions one after the other.  A decay per channel is
 // applied to S first (its numbers lie in shared memory beside k and q), and both sums are taken from the decayed state.
-enum Decay : int { FIXED = 0, HEAD = 1, CHANNEL_LOGITS = 2, CHANNEL_DECAYS = 3 };
+// (Steps with long portions go through recurrence_blocks.cu, four tokens at a time.)
+enum Decay : int { FIXED = 0, HEAD = 1, CHANNEL = 2 };
 
 template <int R, int KS, int MODE, typename TV>
 __global__ void __launch_bounds__(NT) linear_recurrence_kernel(const RecurrenceParams p) {
     extern __shared__ __align__(16) float smem[];
     grid_launch_dependents();
     grid_dependency_wait();
-    constexpr bool DELTA = MODE != FIXED, CHANNEL = MODE == CHANNEL_LOGITS || MODE == CHANNEL_DECAYS;
+    constexpr bool DELTA = MODE != FIXED;
     constexpr int SLOT = R + 4;                          // a slice in shared memory
     constexpr int PITCH = KS * SLOT;
     constexpr int COLS = 4 * (32 / KS);                  // columns of a CTA
@@ -276,7 +276,7 @@ __global__ void __launch_bounds__(NT) linear_recurrence_kernel(const RecurrenceP
         S[r] = (!fresh && live && i < p.dk) ? st[i] : 0.f;
     }
     const float fixed = DELTA ? 0.f : p.decay[h];
-    const float rate = DELTA && MODE != CHANNEL_DECAYS ? p.decay[h] : 0.f, dbias = MODE == HEAD ? p.decay_bias[h] : 0.f;
+    const float rate = DELTA ? p.decay[h] : 0.f, dbias = MODE == HEAD ? p.decay_bias[h] : 0.f;
     const TV* v = reinterpret_cast<const TV*>(p.v);
     const int qk_row = p.G * p.dk;
     // a warp brings whole rows (tokens warp, warp + 4, ...), a lane the places lane, lane + 32, ... of each: which
@@ -288,7 +288,7 @@ __global__ void __launch_bounds__(NT) linear_recurrence_kernel(const RecurrenceP
         const int x = lane + 32 * it, sl = x / SLOT, r = x - sl * SLOT, d = sl * R + r;
         coord[it] = (x < PITCH && r < R && d < p.dk) ? d : -1;
     }
-    float fq[TPW * XN], fk[TPW * XN], fd[CHANNEL ? TPW * XN : 1], fv[V_EACH], fa = 0.f, fb = 0.f;
+    float fq[TPW * XN], fk[TPW * XN], fd[MODE == CHANNEL ? TPW * XN : 1], fv[V_EACH], fa = 0.f, fb = 0.f;
     // the rows of the 16 tokens from t0 on, into registers (zeros past the portion's end)
     auto fetch = [&](int t0) {
         const int n = min(len - t0, RC_TOKENS);
@@ -301,9 +301,7 @@ __global__ void __launch_bounds__(NT) linear_recurrence_kernel(const RecurrenceP
                 const bool in = tt < n && coord[it] >= 0;
                 fq[w * XN + it] = in ? p.q[row + coord[it]] : 0.f;
                 fk[w * XN + it] = in ? p.k[row + coord[it]] : 0.f;
-                if (MODE == CHANNEL_DECAYS)
-                    fd[w * XN + it] = in ? p.g[((size_t)(start + t0 + tt) * p.H + h) * p.dk + coord[it]] : 0.f;
-                if (MODE == CHANNEL_LOGITS)
+                if (MODE == CHANNEL)
                     fd[w * XN + it] = in ? to_float(reinterpret_cast<const TV*>(p.gate)[(size_t)(start + t0 + tt) * p.ldz + (size_t)h * p.dk + coord[it]])
                                                + p.decay_bias[(size_t)h * p.dk + coord[it]] : 0.f;
             }
@@ -333,8 +331,7 @@ __global__ void __launch_bounds__(NT) linear_recurrence_kernel(const RecurrenceP
                 if (x < PITCH) {
                     sq[tt * PITCH + x] = fq[w * XN + it];
                     sk[tt * PITCH + x] = fk[w * XN + it];
-                    if (MODE == CHANNEL_DECAYS) sd[tt * PITCH + x] = fd[w * XN + it];
-                    if (MODE == CHANNEL_LOGITS) {             // (zeros past dk: they multiply the state's unused places)
+                    if (MODE == CHANNEL) {             // (zeros past dk: they multiply the state's unused places)
                         const float a = fd[w * XN + it];
                         sd[tt * PITCH + x] = tt < n && coord[it] >= 0 ? expf(-rate * (a > 20.f ? a : log1pf(expf(a)))) : 0.f;
                     }
@@ -361,7 +358,7 @@ __global__ void __launch_bounds__(NT) linear_recurrence_kernel(const RecurrenceP
             const float4* kt = reinterpret_cast<const float4*>(sk + tt * PITCH + s * SLOT);
             const float4* qt = reinterpret_cast<const float4*>(sq + tt * PITCH + s * SLOT);
             const float vt = sv[tt * COLS + jl], kq = skq[tt];
-            if (CHANNEL) {
+            if (MODE == CHANNEL) {
                 const float4* gt = reinterpret_cast<const float4*>(sd + tt * PITCH + s * SLOT);
 #pragma unroll
                 for (int r = 0; r < R / 4; ++r) {
@@ -396,7 +393,7 @@ __global__ void __launch_bounds__(NT) linear_recurrence_kernel(const RecurrenceP
                 if (DELTA) dot += __shfl_xor_sync(0xffffffffu, dot, off);
             }
             float o;
-            if (CHANNEL) {
+            if (MODE == CHANNEL) {
                 const float u = sb[tt] * (vt - dot);
                 o = fmaf(u, kq, oq);
 #pragma unroll
@@ -505,8 +502,7 @@ extern "C" int tl_recurrence_prep(const void* x, int in_dtype, long long ldx, fl
 // pitch state_pitch holding [heads][dv][dk] (the matrix of a head with a column's keys side by side); out: float32 [n_tokens][heads * dv].
 // mode 0: decay is [heads], the fixed decay.  Otherwise the delta rule: beta are rows of pitch ldg with `heads` columns (of v's
 // dtype).  mode 1: gate are rows of pitch ldz with `heads` columns, decay is exp(A_log) per head and decay_bias [heads] the bias
-// inside the softplus.  mode 2: gate has heads * dk columns and decay_bias heads * dk numbers.  mode 3: gate is float32
-// [n_tokens][heads * dk], the decays themselves.
+// inside the softplus.  mode 2: gate has heads * dk columns and decay_bias heads * dk numbers.
 extern "C" int tl_linear_recurrence(const float* q, const float* k, const void* v, int v_dtype, long long ldv, const void* beta,
                                     long long ldg, const void* gate, long long ldz, const float* decay, const float* decay_bias, float* state,
                                     long long state_pitch, const int* q_start, const int* state_slot, const int* fresh,
@@ -515,11 +511,10 @@ extern "C" int tl_linear_recurrence(const float* q, const float* k, const void* 
     if (n_tokens <= 0 || n_seqs <= 0) return TL_OK;
     if (heads <= 0 || qk_heads <= 0 || heads % qk_heads != 0 || dk <= 0 || dk > 256 || dv <= 0 || n_seqs > 65535 || heads > 65535)
         return TL_BAD_SIZE;
-    if (mode < FIXED || mode > CHANNEL_DECAYS || (mode != CHANNEL_DECAYS && decay == nullptr)) return TL_BAD_SIZE;
-    if (mode != FIXED && (beta == nullptr || gate == nullptr || (mode != CHANNEL_DECAYS && decay_bias == nullptr))) return TL_BAD_SIZE;
+    if (mode < FIXED || mode > CHANNEL || decay == nullptr) return TL_BAD_SIZE;
+    if (mode != FIXED && (beta == nullptr || gate == nullptr || decay_bias == nullptr)) return TL_BAD_SIZE;
     RecurrenceParams p;
-    p.q = q; p.k = k; p.v = v; p.ldv = ldv; p.beta = beta; p.gate = gate; p.ldg = ldg; p.ldz = ldz;
-    p.g = mode == CHANNEL_DECAYS ? (const float*)gate : nullptr; p.decay = decay; p.decay_bias = decay_bias;
+    p.q = q; p.k = k; p.v = v; p.ldv = ldv; p.beta = beta; p.gate = gate; p.ldg = ldg; p.ldz = ldz; p.decay = decay; p.decay_bias = decay_bias;
     p.state = state; p.state_pitch = state_pitch; p.q_start = q_start; p.state_slot = state_slot; p.fresh = fresh; p.out = out;
     p.H = heads; p.G = qk_heads; p.dk = dk; p.dv = dv;
     // slices of the key size per column (TORCHLLMS_B200_REC_SLICES=4|8|16 overrides the choice, for comparisons), and a
@@ -534,13 +529,12 @@ extern "C" int tl_linear_recurrence(const float* q, const float* k, const void* 
     const int share = (dk + ks - 1) / ks;
     const int rows = share <= 8 ? 8 : share <= 12 ? 12 : share <= 16 ? 16 : share <= 24 ? 24 : 32;
     const int cols = 4 * (32 / ks);
-    const size_t smem = ((size_t)(mode >= CHANNEL_LOGITS ? 3 : 2) * RC_TOKENS * ks * (rows + 4) + RC_TOKENS * cols + 3 * RC_TOKENS) * sizeof(float);
+    const size_t smem = ((size_t)(mode == CHANNEL ? 3 : 2) * RC_TOKENS * ks * (rows + 4) + RC_TOKENS * cols + 3 * RC_TOKENS) * sizeof(float);
     const dim3 grid((dv + cols - 1) / cols, heads, n_seqs), block(NT);
     cudaStream_t s = (cudaStream_t)stream;
 #define TL_REC_MODE(R, KS, MODE, TV) launch_recurrence(linear_recurrence_kernel<R, KS, MODE, TV>, grid, block, smem, s, p)
 #define TL_REC(R, KS, TV)                                                                                           \
-    (mode == FIXED ? TL_REC_MODE(R, KS, FIXED, TV) : mode == HEAD ? TL_REC_MODE(R, KS, HEAD, TV)                     \
-     : mode == CHANNEL_LOGITS ? TL_REC_MODE(R, KS, CHANNEL_LOGITS, TV) : TL_REC_MODE(R, KS, CHANNEL_DECAYS, TV))
+    (mode == FIXED ? TL_REC_MODE(R, KS, FIXED, TV) : mode == HEAD ? TL_REC_MODE(R, KS, HEAD, TV) : TL_REC_MODE(R, KS, CHANNEL, TV))
 #define TL_REC_SIZES(TV)                                                                                            \
     (ks == 4 ? (rows == 8 ? TL_REC(8, 4, TV) : rows <= 16 ? TL_REC(16, 4, TV) : rows == 24 ? TL_REC(24, 4, TV) : TL_REC(32, 4, TV)) \
      : ks == 8 ? (rows == 8 ? TL_REC(8, 8, TV) : rows == 12 ? TL_REC(12, 8, TV) : TL_REC(16, 8, TV))                \

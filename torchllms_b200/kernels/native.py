@@ -151,7 +151,7 @@ class NativeOps:
     # ------------------------------------------------------------ libraries
     def prepare(self, dtype: torch.dtype, sampling: bool = True) -> None:
         """Compile, side by side, what a model of this dtype will call."""
-        names = ["elementwise", "sublayer", "rope", "attention", "gemm_simt", "recurrent", "moe", "matrix_state", "stream_sum", "conv_mixers"]
+        names = ["elementwise", "sublayer", "rope", "attention", "gemm_simt", "recurrent", "moe", "matrix_state", "stream_sum", "conv_mixers", "recurrence_blocks"]
         if dtype == torch.bfloat16:
             names += ["attention_mma", "attention_decode", "gemm_tcgen05"]
         if sampling:
@@ -1048,7 +1048,7 @@ class NativeOps:
         self.launches += 2 if (max_q_len > 16 and w_conv.shape[1] > 1) else 1
         return q, k, v, small, low
 
-    DECAYS_MIN_Q = 9      # portions from which decays per channel are worked out by a kernel of their own, once per token
+    BLOCKS_MIN_Q = 9      # steps with portions at least this long run a matrix recurrence four tokens at a time
 
     @_timed
     def recurrence_prep(self, x: torch.Tensor, *, scale: float, n_heads: int, head_dim: int,
@@ -1092,7 +1092,8 @@ class NativeOps:
         per head and key coordinate: ``decay_logits`` ``[T, H * dk]`` and ``decay_bias`` ``[H * dk]``, each acting on its row of ``S``.
         ``q``, ``k``: float32 ``[T, G * dk]``, ``G`` heads each shared by ``H / G`` value heads; ``v``: ``[T, H * dv]``;
         ``state``: ``[slots, H, dv, dk]`` (a head's matrix with a column's keys side by side), read (zeros where
-        ``fresh``) and left updated.  Returns float32 ``[T, H * dv]``."""
+        ``fresh``) and left updated.  Returns float32 ``[T, H * dv]``.  Steps with long portions take four tokens at a time
+        (the same rule written out), others one."""
         _cuda_contig(q, "q", torch.float32)
         _cuda_contig(k, "k", torch.float32)
         ldv = self._rows_view(v, "v")
@@ -1105,7 +1106,7 @@ class NativeOps:
         _need(G > 0 and H % G == 0, f"{H} value heads cannot share {G} heads of q and k")
         _need(dk <= 256, f"linear_recurrence keeps a head's state in registers: key size {dk} exceeds 256")
         self._seq_index(q_start, state_slot, fresh, n_seqs)
-        delta = decay is None
+        delta, blocks = decay is None, max_q_len >= self.BLOCKS_MIN_Q
         ldg = ldz = ctypes.c_longlong(0)
         mode = 0
         if delta:
@@ -1117,8 +1118,8 @@ class NativeOps:
             ldg, ldz = self._rows_view(beta_logits, "beta_logits"), self._rows_view(decay_logits, "decay_logits")
             _need(beta_logits.shape == (T, H) and (per_channel or decay_logits.shape == (T, H)) and beta_logits.dtype == v.dtype
                   and decay_logits.dtype == v.dtype, "beta_logits must be [T, H] and decay_logits [T, H] or [T, H * dk], of v's dtype")
-            if per_channel and max_q_len >= self.DECAYS_MIN_Q:
-                # long portions: the decays once per token (few tokens: by every CTA of the recurrence for itself)
+            if per_channel and blocks:
+                # the decays once per token (in steps of short portions: by every CTA of the recurrence for itself)
                 decays = torch.empty((T, H * dk), dtype=torch.float32, device=q.device)
                 _check(self._lib("conv_mixers").tl_channel_decay(_ptr(decay_logits), _DT[decay_logits.dtype], ldz, _ptr(decay_rate), _ptr(decay_bias),
                                                                  _ptr(decays), T, H * dk, dk, _stream()), "channel_decay")
@@ -1128,7 +1129,8 @@ class NativeOps:
             _cuda_contig(decay, "decay", torch.float32)
             _need(decay.numel() == H, "decay: one number per head")
         out = torch.empty((T, H * dv), dtype=torch.float32, device=q.device)
-        rc = self._lib("matrix_state").tl_linear_recurrence(
+        run = self._lib("recurrence_blocks").tl_recurrence_blocks if blocks else self._lib("matrix_state").tl_linear_recurrence
+        rc = run(
             _ptr(q), _ptr(k), _ptr(v), _DT[v.dtype], ldv, _ptr(beta_logits), ldg, _ptr(decay_logits), ldz,
             _ptr(decay_rate if delta else decay), _ptr(decay_bias), _ptr(state), pitch, _ptr(q_start), _ptr(state_slot), _ptr(fresh),
             _ptr(out), T, n_seqs, H, G, dk, dv, mode, _stream())
