@@ -412,7 +412,7 @@ def test_convolution_rotation_and_store(backend):
                 (q_start, slot_t, fresh_t), how = _steps(lens, slots, fresh, dev)
                 held = state_all.to(dev)
                 view = wide.to(dev)[..., off:off + W]
-                got_q, gate = ops.conv_rope_store(view if splits > 1 else view[0], w.to(dev), field(held), pos.to(torch.int32).to(dev), table, q_start,
+                got_q, gate = ops.conv_rope_store(view if splits > 1 else view[0], w.t().contiguous().to(dev), field(held), pos.to(torch.int32).to(dev), table, q_start,
                                                   slot_t, fresh_t, n_q_heads=H, n_k_heads=G, head_dim=d, v_head_dim=dv, rot_dims=rot,
                                                   n_extra=extra, k_pages=kp, v_pages=vp, slot_mapping=sm.to(torch.int32).to(dev),
                                                   page_size=page, out_dtype=dt, extra_scale=1.7, **how)
@@ -459,7 +459,7 @@ def test_preparing_a_delta_rule(backend):
                 held = state.to(dev) if taps > 1 else None
                 view = wide.to(dev)[..., off:]
                 pad = -(-n_low // 8) * 8
-                got = ops.delta_prep(view if splits > 1 else view[0], w.to(dev), held, q_start, slot_t, fresh_t, n_qk_heads=heads, head_dim=d, n_v=n_v,
+                got = ops.delta_prep(view if splits > 1 else view[0], w.t().contiguous().to(dev), held, q_start, slot_t, fresh_t, n_qk_heads=heads, head_dim=d, n_v=n_v,
                                      n_small=n_small, n_low=n_low, low_pad=pad, q_scale=0.3, unit_eps=1e-6, out_dtype=dt, **how)
                 tol = dict(atol=2e-5, rtol=2e-5) if dt == torch.float32 else dict(atol=2e-2, rtol=2e-2)
                 torch.testing.assert_close(got[0].cpu().double(), q, atol=2e-5, rtol=1e-4)

@@ -189,8 +189,8 @@ class TorchOps:
         """A row of proj is [q heads | k heads | v heads | extra]: a short convolution over the q, k and v columns, then
         what rope_store does in the half pairing; sigmoid(extra) * extra_scale."""
         x = proj.float().sum(0) if proj.dim() == 3 else proj.float()
-        nc = w_conv.shape[0]
-        y = self.short_conv(x[:, :nc], w_conv, state, q_start, state_slot, fresh, n_seqs=n_seqs, max_q_len=max_q_len, activation=None,
+        nc = w_conv.shape[1]
+        y = self.short_conv(x[:, :nc], w_conv.t(), state, q_start, state_slot, fresh, n_seqs=n_seqs, max_q_len=max_q_len, activation=None,
                             residual=False, out_dtype=torch.float32)
         q, gate = self.rope_store(torch.cat([y, x[:, nc:]], dim=1), positions, table, n_q_heads=n_q_heads, n_k_heads=n_k_heads,
                                   n_v_heads=n_k_heads, head_dim=head_dim, v_head_dim=v_head_dim, rot_dims=rot_dims, interleaved=False,
@@ -203,8 +203,8 @@ class TorchOps:
         """A row of proj is [q | k | v | small | low | rest]: a short convolution and silu on q, k and v, q (times q_scale) and k as
         unit vectors per head in float32, v, the small columns, and the low ones padded with zeros."""
         x = proj.float().sum(0) if proj.dim() == 3 else proj.float()
-        nc, n = w_conv.shape[0], n_qk_heads * head_dim
-        c = self.short_conv(x[:, :nc], w_conv, state, q_start, state_slot, fresh, n_seqs=n_seqs, max_q_len=max_q_len, activation="silu",
+        nc, n = w_conv.shape[1], n_qk_heads * head_dim
+        c = self.short_conv(x[:, :nc], w_conv.t(), state, q_start, state_slot, fresh, n_seqs=n_seqs, max_q_len=max_q_len, activation="silu",
                             residual=False, out_dtype=torch.float32)
         unit = dict(n_heads=n_qk_heads, head_dim=head_dim, unit_eps=unit_eps)
         low = None

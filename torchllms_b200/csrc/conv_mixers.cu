@@ -1,5 +1,5 @@
 // What stands between a mixer's stacked input projection and its attention or recurrence where every channel of
-// q, k and v passes a short causal convolution over time first:  y_t = sum_j w[c][j] u_(t - taps + 1 + j), the last
+// q, k and v passes a short causal convolution over time first:  y_t = sum_j w[j][c] u_(t - taps + 1 + j), the last
 // taps - 1 inputs of every request being its state (zeros for a fresh one).
 //
 // conv_rope_store: row [q heads | k heads | v heads | extra]: convolution of the q, k and v columns, rotation of the
@@ -28,7 +28,7 @@ struct ConvInput {
     const void* proj;        // [splits][T] rows of pitch ld
     int splits;
     long long plane, ld;
-    const float* w;          // [C][taps], the last column the current token's
+    const float* w;          // [taps][C], the last row the current token's
     float* state;            // [slots] rows of pitch state_pitch, each [taps - 1][C]; null with one tap
     long long state_pitch;
     const int* q_start;      // [B + 1]
@@ -102,14 +102,12 @@ __device__ __forceinline__ Cols<VEC> conv_cols(const ConvInput& p, int start, in
 template <int VEC, int TM>
 struct Window {
     Cols<VEC> in[TM];
-    float w[VEC][TM];
+    Cols<VEC> w[TM];
     template <typename TI>
     __device__ __forceinline__ void open(const ConvInput& p, int start, int r0, int c, const float* st, bool fresh) {
         const int off = TM - p.taps;
 #pragma unroll
-        for (int e = 0; e < VEC; ++e)
-#pragma unroll
-            for (int j = 0; j < TM; ++j) w[e][j] = j >= off ? p.w[(size_t)(c + e) * p.taps + (j - off)] : 0.f;
+        for (int j = 0; j < TM; ++j) w[j] = j >= off ? load_cols<VEC>(p.w + (size_t)(j - off) * p.C + c) : zero_cols<VEC>();
         // before the first push: the inputs r0 - (TM - 1) .. r0 - 1 lie in places 1 .. TM - 1
         in[0] = zero_cols<VEC>();
 #pragma unroll
@@ -125,7 +123,7 @@ struct Window {
         for (int e = 0; e < VEC; ++e) {
             float acc = 0.f;
 #pragma unroll
-            for (int j = 0; j < TM; ++j) acc = fmaf(w[e][j], in[j].v[e], acc);
+            for (int j = 0; j < TM; ++j) acc = fmaf(w[j].v[e], in[j].v[e], acc);
             y.v[e] = acc;
         }
         return y;
@@ -408,13 +406,13 @@ bool good_input(const ConvInput& x, int n_seqs, int max_q_len) {
 // whether rows and state may be read four columns at a time (column offsets are the caller's to check)
 bool vector_input(const ConvInput& x, int in_dtype) {
     const uintptr_t a = reinterpret_cast<uintptr_t>(x.proj);
-    return x.C % 4 == 0 && x.ld % 4 == 0 && x.plane % 4 == 0 && a % (in_dtype == TL_F32 ? 16 : 8) == 0 && x.state_pitch % 4 == 0 && aligned16(x.state);
+    return x.C % 4 == 0 && aligned16(x.w) && x.ld % 4 == 0 && x.plane % 4 == 0 && a % (in_dtype == TL_F32 ? 16 : 8) == 0 && x.state_pitch % 4 == 0 && aligned16(x.state);
 }
 
 }  // namespace
 
 // proj: [splits][n_tokens] rows of pitch ld (elements of in_dtype), planes `plane` apart, columns [q heads | k heads | v heads |
-// extra]; w: float32 [q, k and v columns][taps]; state: float32 rows of pitch state_pitch per slot, [taps - 1][columns] each (null
+// extra]; w: float32 [taps][q, k and v columns]; state: float32 rows of pitch state_pitch per slot, [taps - 1][columns] each (null
 // with one tap); table: float32 [table_rows, rot / 2, 2]; q_out [n_tokens, n_q, hd], extra_out [n_tokens, n_extra] and pages
 // ([pages, n_k, page_size, hd] and [.., dv]) of dtype.
 extern "C" int tl_conv_rope_store(const void* proj, int in_dtype, int splits, long long plane, long long ld, const float* w, int taps,
@@ -457,7 +455,7 @@ extern "C" int tl_conv_rope_store(const void* proj, int in_dtype, int splits, lo
     return p.x.n_chunks > 1 && p.x.state != nullptr ? launch_state(p.x, in_dtype, n_seqs, s) : TL_OK;
 }
 
-// proj as above with columns [q heads | k heads | v | small | low | ...]; w: float32 [2 * heads * hd + n_v][taps]; q, k: float32
+// proj as above with columns [q heads | k heads | v | small | low | ...]; w: float32 [taps][2 * heads * hd + n_v]; q, k: float32
 // [n_tokens][heads * hd]; v [n_tokens][n_v], small [n_tokens][n_small], low [n_tokens][low_pad] of dtype (low null with n_low 0).
 extern "C" int tl_delta_prep(const void* proj, int in_dtype, int splits, long long plane, long long ld, const float* w, int taps,
                              float* state, long long state_pitch, const int* q_start, const int* state_slot, const int* fresh, float* q,

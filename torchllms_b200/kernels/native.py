@@ -151,7 +151,7 @@ class NativeOps:
     # ------------------------------------------------------------ libraries
     def prepare(self, dtype: torch.dtype, sampling: bool = True) -> None:
         """Compile, side by side, what a model of this dtype will call."""
-        names = ["elementwise", "sublayer", "rope", "attention", "gemm_simt", "recurrent", "moe", "matrix_state", "stream_sum", "conv_mixers", "recurrence_blocks"]
+        names = ["elementwise", "sublayer", "rope", "attention", "gemm_simt", "recurrent", "moe", "matrix_state", "stream_sum", "conv_mixers", "matrix_recurrence"]
         if dtype == torch.bfloat16:
             names += ["attention_mma", "attention_decode", "gemm_tcgen05"]
         if sampling:
@@ -973,8 +973,8 @@ class NativeOps:
     def _conv_args(self, w_conv: torch.Tensor, state: Optional[torch.Tensor], columns: int):
         """``(taps pointer, number of taps, state pointer, the slots' pitch)`` of a convolution over so many channels."""
         _cuda_contig(w_conv, "convolution taps", torch.float32)
-        _need(w_conv.dim() == 2 and w_conv.shape[0] == columns and 1 <= w_conv.shape[1] <= 8, f"convolution taps must be [{columns}, taps], at most 8 taps")
-        taps, pitch = w_conv.shape[1], ctypes.c_longlong(0)
+        _need(w_conv.dim() == 2 and w_conv.shape[1] == columns and 1 <= w_conv.shape[0] <= 8, f"convolution taps must be [taps, {columns}], at most 8 taps")
+        taps, pitch = w_conv.shape[0], ctypes.c_longlong(0)
         if taps > 1:
             _need(state is not None, "a convolution of several taps keeps state")
             pitch = self._state_view(state, (taps - 1) * columns, "convolution state")
@@ -988,7 +988,7 @@ class NativeOps:
                         extra_scale: float = 1.0):
         """What follows a stacked projection ``[q heads | k heads | v heads | extra]`` (``[T, width]`` or float32 partial sums,
         a column range of wider rows will do) where every channel of q, k and v passes a causal convolution over time
-        first (``w_conv`` float32 ``[channels, taps]``; ``state`` as in :meth:`short_conv`): then, as :meth:`rope_store` does in
+        first (``w_conv`` float32 ``[taps, channels]``; ``state`` as in :meth:`short_conv`): then, as :meth:`rope_store` does in
         the half pairing, rotation, the page writes, ``q [T, n_q_heads, head_dim]`` and ``extra_scale * sigmoid(extra)``."""
         cols = (n_q_heads + n_k_heads) * head_dim + n_k_heads * v_head_dim
         splits, plane, ld = self._planes_view(proj, cols + n_extra, "projection")
@@ -1015,7 +1015,7 @@ class NativeOps:
             _ptr(slot_mapping), _ptr(q), _ptr(extra), _ptr(k_pages), _ptr(v_pages), _DT[out_dtype], T, n_seqs, max_q_len, n_q_heads,
             n_k_heads, head_dim, v_head_dim, rot_dims, n_extra, ctypes.c_float(extra_scale), page_size, table.shape[0], _stream())
         _check(rc, "conv_rope_store")
-        self.launches += 2 if (max_q_len > 16 and w_conv.shape[1] > 1) else 1
+        self.launches += 2 if (max_q_len > 16 and w_conv.shape[0] > 1) else 1
         return q, extra
 
     @_timed
@@ -1024,7 +1024,7 @@ class NativeOps:
                    n_v: int, n_small: int, n_low: int, low_pad: int, q_scale: float, unit_eps: float, out_dtype: torch.dtype):
         """What a delta rule needs of a stacked projection ``[q heads | k heads | v | small | low | ...]`` (``[T, width]`` or
         float32 partial sums, a column range of wider rows will do): q, k and v pass a causal convolution over time and
-        ``silu`` (``w_conv`` and ``state`` as in :meth:`short_conv`), every head of q and k becomes a unit vector (``x / sqrt(sum(x^2) +
+        ``silu`` (``w_conv`` and ``state`` as in :meth:`conv_rope_store`), every head of q and k becomes a unit vector (``x / sqrt(sum(x^2) +
         unit_eps)``, q times ``q_scale``).  Returns ``(q, k, v, small, low)``: q and k float32 ``[T, n_qk_heads * head_dim]``, the rest
         in ``out_dtype``, ``low`` as ``[T, low_pad]`` with zeros behind its ``n_low`` columns (``None`` without any)."""
         n_qk = n_qk_heads * head_dim
@@ -1045,7 +1045,7 @@ class NativeOps:
             _ptr(small), _ptr(low), _DT[out_dtype], T, n_seqs, max_q_len, n_qk_heads, head_dim, n_v, n_small, n_low, low_pad,
             ctypes.c_float(q_scale), ctypes.c_float(unit_eps), _stream())
         _check(rc, "delta_prep")
-        self.launches += 2 if (max_q_len > 16 and w_conv.shape[1] > 1) else 1
+        self.launches += 2 if (max_q_len > 16 and w_conv.shape[0] > 1) else 1
         return q, k, v, small, low
 
     BLOCKS_MIN_Q = 9      # steps with portions at least this long run a matrix recurrence four tokens at a time
@@ -1124,16 +1124,15 @@ class NativeOps:
                 _check(self._lib("conv_mixers").tl_channel_decay(_ptr(decay_logits), _DT[decay_logits.dtype], ldz, _ptr(decay_rate), _ptr(decay_bias),
                                                                  _ptr(decays), T, H * dk, dk, _stream()), "channel_decay")
                 self.launches += 1
-                mode, decay_logits = 3, decays
+                decay_logits = decays
         else:
             _cuda_contig(decay, "decay", torch.float32)
             _need(decay.numel() == H, "decay: one number per head")
         out = torch.empty((T, H * dv), dtype=torch.float32, device=q.device)
-        run = self._lib("recurrence_blocks").tl_recurrence_blocks if blocks else self._lib("matrix_state").tl_linear_recurrence
-        rc = run(
+        rc = self._lib("matrix_recurrence").tl_linear_recurrence(
             _ptr(q), _ptr(k), _ptr(v), _DT[v.dtype], ldv, _ptr(beta_logits), ldg, _ptr(decay_logits), ldz,
             _ptr(decay_rate if delta else decay), _ptr(decay_bias), _ptr(state), pitch, _ptr(q_start), _ptr(state_slot), _ptr(fresh),
-            _ptr(out), T, n_seqs, H, G, dk, dv, mode, _stream())
+            _ptr(out), T, n_seqs, H, G, dk, dv, mode, 1 if blocks else 0, _stream())
         _check(rc, "linear_recurrence")
         self.launches += 1
         return out

@@ -476,7 +476,7 @@ class RotaryGatedAttention(Mixer):
         if self.has_sinks:
             self.sinks = tensors["sinks"].to(**f32).contiguous()
         if self.taps:
-            self.w_conv = torch.cat([tensors[f"{n}.conv"].to(**f32) for n, _rows in self._projected()]).contiguous()
+            self.w_conv = torch.cat([tensors[f"{n}.conv"].to(**f32) for n, _rows in self._projected()]).t().contiguous()       # [taps, channels]
         self.wo = as_compute(tensors["wo.weight"], self.env)
 
     def weight_bytes(self) -> int:

@@ -209,7 +209,7 @@ class GatedDelta(Mixer):
         names = ["wq.weight", "wk.weight", "wv.weight", "wb.weight"] + ["wa1.weight" if self.per_channel else "wa.weight"] \
             + ["wg1.weight" if self.low_rank_gate else "wg.weight"]
         self.w_in = torch.cat([as_compute(tensors[n], self.env) for n in names])
-        self.w_conv = torch.cat([tensors[n].to(**f32) for n in ("wq.conv", "wk.conv", "wv.conv")]).contiguous()
+        self.w_conv = torch.cat([tensors[n].to(**f32) for n in ("wq.conv", "wk.conv", "wv.conv")]).t().contiguous()      # [taps, channels]
         outer = [tensors[f"{n}2.weight"] for n, low in (("wa", self.per_channel), ("wg", self.low_rank_gate)) if low]
         inner = [tensors[f"{n}1.weight"].shape[0] for n, low in (("wa", self.per_channel), ("wg", self.low_rank_gate)) if low]
         if outer:
