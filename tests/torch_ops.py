@@ -8,6 +8,7 @@ Nothing in the package imports this file.
 
 from __future__ import annotations
 
+import contextlib
 import math
 from typing import Optional
 
@@ -52,6 +53,13 @@ class TorchOps:
     name = "torch-twin"
 
     def prepare(self, dtype, sampling=True):
+        pass
+
+    @contextlib.contextmanager
+    def aside(self, max_q_len):
+        yield
+
+    def rejoin(self):
         pass
 
     def check_attention_sizes(self, n_heads, n_kv_heads, head_dim, dtype, v_head_dim=None):

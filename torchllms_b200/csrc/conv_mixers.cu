@@ -11,8 +11,8 @@
 // channel_decay:   g = exp(-rate_h softplus(z + bias)) per head and key coordinate, float32.
 //
 // Rows are column ranges of wider rows (a row pitch) and may be float32 partial sums of a split-K product (planes),
-// added up on the way in.  A thread (conv_rope_store) or a warp (delta_prep) owns columns and walks up to TOK tokens of a
-// portion with a window of the last inputs in registers.  In a step of short portions it also leaves the new
+// added up on the way in.  A thread (conv_rope_store) or a warp (delta_prep) owns columns of TOK tokens of a
+// portion, with a window of the inputs before them in registers.  In a step of short portions it also leaves the new
 // state; with longer portions a kernel of its own does that afterwards, since several owners read the old one.
 // All arithmetic is float32.
 #include "common.cuh"
@@ -20,8 +20,7 @@
 namespace {
 
 constexpr int MAX_TAPS = 8;
-constexpr int TOK = 16;            // tokens of a portion that one owner of columns walks
-constexpr int GROUP = 4;           // of which so many are in flight
+constexpr int TOK = 4;             // tokens of a portion that one owner of columns takes: all its loads are in flight at once
 constexpr int NT = 128;
 
 struct ConvInput {
@@ -167,18 +166,16 @@ __global__ void __launch_bounds__(NT) conv_rope_store_kernel(const StoreParams p
     if (item >= n_qk + n_v) {                                   // the gate's columns take no part in the convolution
         const int c = (item - n_qk - n_v) * VEC;
         T* out = reinterpret_cast<T*>(p.extra_out);
-        for (int i0 = 0; i0 < n; i0 += GROUP) {
-            Cols<VEC> x[GROUP];
+        Cols<VEC> x[TOK];
 #pragma unroll
-            for (int i = 0; i < GROUP; ++i)
-                x[i] = i0 + i < n ? row_cols<VEC, TI>(p.x, (long long)start + r0 + i0 + i, p.x.C + c) : zero_cols<VEC>();
+        for (int i = 0; i < TOK; ++i)
+            x[i] = i < n ? row_cols<VEC, TI>(p.x, (long long)start + r0 + i, p.x.C + c) : zero_cols<VEC>();
 #pragma unroll
-            for (int i = 0; i < GROUP; ++i) {
-                if (i0 + i >= n) break;
+        for (int i = 0; i < TOK; ++i) {
+            if (i >= n) break;
 #pragma unroll
-                for (int e = 0; e < VEC; ++e) x[i].v[e] = p.extra_scale / (1.f + expf(-x[i].v[e]));
-                store_cols<VEC>(out + ((size_t)start + r0 + i0 + i) * p.n_extra + c, x[i]);
-            }
+            for (int e = 0; e < VEC; ++e) x[i].v[e] = p.extra_scale / (1.f + expf(-x[i].v[e]));
+            store_cols<VEC>(out + ((size_t)start + r0 + i) * p.n_extra + c, x[i]);
         }
         return;
     }
@@ -204,18 +201,18 @@ __global__ void __launch_bounds__(NT) conv_rope_store_kernel(const StoreParams p
     Window<VEC, TM> wa, wb;
     wa.template open<TI>(p.x, start, r0, c0, st, fresh);
     if (c1 >= 0) wb.template open<TI>(p.x, start, r0, c1, st, fresh);
-    for (int i0 = 0; i0 < n; i0 += GROUP) {
-        Cols<VEC> xa[GROUP], xb[GROUP];
+    {
+        Cols<VEC> xa[TOK], xb[TOK];
 #pragma unroll
-        for (int i = 0; i < GROUP; ++i) {
-            const bool in = i0 + i < n;
-            xa[i] = in ? row_cols<VEC, TI>(p.x, (long long)start + r0 + i0 + i, c0) : zero_cols<VEC>();
-            xb[i] = in && c1 >= 0 ? row_cols<VEC, TI>(p.x, (long long)start + r0 + i0 + i, c1) : zero_cols<VEC>();
+        for (int i = 0; i < TOK; ++i) {
+            const bool in = i < n;
+            xa[i] = in ? row_cols<VEC, TI>(p.x, (long long)start + r0 + i, c0) : zero_cols<VEC>();
+            xb[i] = in && c1 >= 0 ? row_cols<VEC, TI>(p.x, (long long)start + r0 + i, c1) : zero_cols<VEC>();
         }
 #pragma unroll
-        for (int i = 0; i < GROUP; ++i) {
-            if (i0 + i >= n) break;
-            const int t = start + r0 + i0 + i;
+        for (int i = 0; i < TOK; ++i) {
+            if (i >= n) break;
+            const int t = start + r0 + i;
             Cols<VEC> ya = wa.push(xa[i]), yb;
             if (c1 >= 0) {
                 yb = wb.push(xb[i]);
@@ -301,11 +298,16 @@ __global__ void __launch_bounds__(NT) delta_prep_kernel(const DeltaParams p) {
         for (int e = lane; e < UNIT; e += 32) {
             const int c = base + e;
             if (c >= p.n_small + p.low_pad) break;
-            for (int i = 0; i < n; ++i) {
-                const long long t = (long long)start + r0 + i;
-                const float x = c < p.n_small + p.n_low ? row_cols<1, TI>(p.x, t, p.x.C + c).v[0] : 0.f;
-                if (c < p.n_small) reinterpret_cast<T*>(p.small)[t * p.n_small + c] = from_float<T>(x);
-                else reinterpret_cast<T*>(p.low)[t * p.low_pad + (c - p.n_small)] = from_float<T>(x);
+            float x[TOK];
+#pragma unroll
+            for (int i = 0; i < TOK; ++i)
+                x[i] = i < n && c < p.n_small + p.n_low ? row_cols<1, TI>(p.x, (long long)start + r0 + i, p.x.C + c).v[0] : 0.f;
+#pragma unroll
+            for (int i = 0; i < TOK; ++i) {
+                if (i >= n) break;
+                const size_t t = (size_t)start + r0 + i;
+                if (c < p.n_small) reinterpret_cast<T*>(p.small)[t * p.n_small + c] = from_float<T>(x[i]);
+                else reinterpret_cast<T*>(p.low)[t * p.low_pad + (c - p.n_small)] = from_float<T>(x[i]);
             }
         }
         return;
@@ -326,19 +328,19 @@ __global__ void __launch_bounds__(NT) delta_prep_kernel(const DeltaParams p) {
     const bool is_q = unit < p.heads;
     const float scale = is_q ? p.q_scale : 1.f;
     float* qk_out = is_q ? p.q + (size_t)unit * p.hd : p.k + (size_t)(unit - p.heads) * p.hd;
-    for (int i0 = 0; i0 < n; i0 += GROUP) {
-        Cols<VEC> y[GROUP][IT];
+    {
+        Cols<VEC> y[TOK][IT];
 #pragma unroll
-        for (int i = 0; i < GROUP; ++i)
+        for (int i = 0; i < TOK; ++i)
 #pragma unroll
             for (int it = 0; it < IT; ++it)
-                y[i][it] = i0 + i < n && mine[it] ? row_cols<VEC, TI>(p.x, (long long)start + r0 + i0 + i, c_lo + (it * 32 + lane) * VEC)
+                y[i][it] = i < n && mine[it] ? row_cols<VEC, TI>(p.x, (long long)start + r0 + i, c_lo + (it * 32 + lane) * VEC)
                                                   : zero_cols<VEC>();
-        float ssq[GROUP];
+        float ssq[TOK];
 #pragma unroll
-        for (int i = 0; i < GROUP; ++i) {
+        for (int i = 0; i < TOK; ++i) {
             ssq[i] = 0.f;
-            if (i0 + i < n) {
+            if (i < n) {
 #pragma unroll
                 for (int it = 0; it < IT; ++it) {
                     if (!mine[it]) continue;
@@ -354,12 +356,12 @@ __global__ void __launch_bounds__(NT) delta_prep_kernel(const DeltaParams p) {
         }
         if (!is_v) {
 #pragma unroll
-            for (int i = 0; i < GROUP; ++i) ssq[i] = rsqrtf(warp_sum(ssq[i]) + p.unit_eps) * scale;
+            for (int i = 0; i < TOK; ++i) ssq[i] = rsqrtf(warp_sum(ssq[i]) + p.unit_eps) * scale;
         }
 #pragma unroll
-        for (int i = 0; i < GROUP; ++i) {
-            if (i0 + i >= n) break;
-            const size_t t = (size_t)start + r0 + i0 + i;
+        for (int i = 0; i < TOK; ++i) {
+            if (i >= n) break;
+            const size_t t = (size_t)start + r0 + i;
 #pragma unroll
             for (int it = 0; it < IT; ++it) {
                 if (!mine[it]) continue;

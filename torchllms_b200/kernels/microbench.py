@@ -8,6 +8,7 @@
     python -m torchllms_b200.kernels.microbench selective_scan --tokens 2048 --channels 4096 --state 16
     python -m torchllms_b200.kernels.microbench attention_options --length 2048 --span 1024
     python -m torchllms_b200.kernels.microbench rows --tokens 2048
+    python -m torchllms_b200.kernels.microbench delta --tokens 2048 --heads 16
 
 Every case is timed with CUDA events after warm-up.  Memory-bound kernels run inside a CUDA
 graph over several copies of their operands (more than the 126 MB of L2 together), so that a
@@ -277,6 +278,64 @@ def rows(args) -> None:
     line(f"clamped gate, {n} rows", [(lambda u=u: ops.glu(u, limit=7.0, alpha=1.702, up_offset=1.0)) for u in gu], n * D * 6)
 
 
+def delta(args) -> None:
+    """Mixers behind short convolutions (4 taps, heads of 128, a quarter as many shared heads): what follows the input
+    projection, the matrix recurrences and the head norm, for one prompt of --tokens and for 8 decoded tokens (whose
+    projections arrive as two float32 partial sums).  GB/s of the algorithmic bytes."""
+    from ..parts.rope import precise_rotary_table
+    ops = get_ops()
+    H, d, page, taps, low, dev, bf = args.heads, 128, 16, 4, 256, "cuda", torch.bfloat16
+    G, f32 = max(H // 4, 1), torch.float32
+    i32 = lambda xs: torch.tensor(xs, dtype=torch.int32, device=dev)
+
+    def line(name: str, calls, moved: float) -> None:
+        us = _time(_graphed(calls), 5) / len(calls)
+        print(f"{name}: {us:7.1f} us  {moved / us / 1e3:7.1f} GB/s")
+
+    left, right = (2 * H + 2 * G) * d, 2 * G * d + H * d + H + low
+    for T, B, splits, copies in ((args.tokens, 1, 1, 4), (8, 8, 2, 16)):
+        rows = [torch.randn(splits, T, left + right, device=dev).to(bf if splits == 1 else f32) for _ in range(copies)]
+        rows = [r if splits > 1 else r[0] for r in rows]
+        each = 2 if splits == 1 else 4 * splits
+        at = (i32([b * T // B for b in range(B + 1)]), i32(list(range(B))), i32([int(B == 1)] * B))
+        how = dict(n_seqs=B, max_q_len=T // B)
+        positions = torch.arange(T, dtype=torch.int32, device=dev)
+        kp = torch.zeros(-(-T // page), G, page, d, device=dev, dtype=bf)
+        vp, table = torch.zeros_like(kp), precise_rotary_table(d, 1e6, 1.0, max(T, 64), dev)
+        n_left, n_right = (H + 2 * G) * d, (H + 2 * G) * d
+        wl, wr = torch.randn(taps, n_left, device=dev), torch.randn(taps, n_right, device=dev)
+        sl, sr = torch.zeros(B, taps - 1, n_left, device=dev), torch.zeros(B, taps - 1, n_right, device=dev)
+        store = dict(n_q_heads=H, n_k_heads=G, head_dim=d, v_head_dim=d, rot_dims=d, n_extra=H * d, k_pages=kp, v_pages=vp,
+                     slot_mapping=positions, page_size=page, out_dtype=bf)
+        line(f"conv_rope_store, {T} rows", [(lambda r=r: ops.conv_rope_store(r[..., :left], wl, sl, positions, table, *at, **how, **store)) for r in rows],
+             T * left * (each + 2))
+        prep = dict(n_qk_heads=G, head_dim=d, n_v=H * d, n_small=H, n_low=low, low_pad=low, q_scale=d ** -0.5, unit_eps=1e-6, out_dtype=bf)
+        line(f"delta_prep, {T} rows", [(lambda r=r: ops.delta_prep(r[..., left:], wr, sr, *at, **how, **prep)) for r in rows],
+             T * (right * each + 2 * G * d * 4 + (H * d + H + low) * 2))
+        if splits == 1:
+            sc = torch.zeros(B, taps - 1, n_right, device=dev)
+            line(f"short_conv of as many channels, {T} rows",
+                 [(lambda r=r: ops.short_conv(r[:, left:left + n_right], wr.t().contiguous(), sc, *at, **how, activation="silu", residual=False, out_dtype=bf))
+                  for r in rows], T * n_right * 4)
+        q, k = torch.randn(T, G * d, device=dev) * d ** -0.5, torch.nn.functional.normalize(torch.randn(T, G, d, device=dev), dim=-1).flatten(1)
+        v, beta, z = torch.randn(T, H * d, device=dev).to(bf), torch.randn(T, H, device=dev).to(bf), torch.randn(T, 2 * H * d, device=dev).to(bf)
+        states = [torch.zeros(B, H, d, d, device=dev) for _ in range(copies)]
+        rate, bias = torch.rand(H, device=dev), torch.randn(H * d, device=dev) - 3.0
+        moved = T * (2 * G * d * 4 + H * d * 6) + B * H * d * d * (8 if B > 1 else 4)
+        line(f"recurrence, a decay per channel, {T} tokens of {B}",
+             [(lambda s=s: ops.linear_recurrence(q, k, v, s, *at, **how, beta_logits=beta, decay_logits=z[:, :H * d], decay_rate=rate, decay_bias=bias))
+              for s in states], moved + T * H * d * 2)
+        line(f"recurrence, a decay per head, {T} tokens of {B}",
+             [(lambda s=s: ops.linear_recurrence(q, k, v, s, *at, **how, beta_logits=beta, decay_logits=z[:, :H], decay_rate=rate, decay_bias=bias[:H]))
+              for s in states], moved)
+        line(f"recurrence, fixed decays, {T} tokens of {B}",
+             [(lambda s=s: ops.linear_recurrence(q, k, v, s, *at, **how, decay=rate)) for s in states], moved)
+        os, outs = [torch.randn(T, H * d, device=dev) for _ in range(copies)], torch.empty(T, 2 * H * d, device=dev, dtype=bf)
+        w = torch.randn(d, device=dev)
+        line(f"head_norm_gate, {T} rows", [(lambda o=o: ops.head_norm_gate(o, z[:, H * d:], w, 1e-6, head_dim=d, out_dtype=bf, activation="sigmoid",
+                                                                           out=outs[:, H * d:])) for o in os], T * H * d * 8)
+
+
 def main(argv=None) -> None:
     parser = argparse.ArgumentParser(description=__doc__, formatter_class=argparse.RawDescriptionHelpFormatter)
     sub = parser.add_subparsers(dest="case", required=True)
@@ -306,6 +365,10 @@ def main(argv=None) -> None:
     p = sub.add_parser("rows")
     p.add_argument("--tokens", type=int, default=2048)
     p.set_defaults(run=rows)
+    p = sub.add_parser("delta")
+    p.add_argument("--tokens", type=int, default=2048)
+    p.add_argument("--heads", type=int, default=16)
+    p.set_defaults(run=delta)
     p = sub.add_parser("elementwise")
     p.add_argument("--tokens", type=int, default=2048)
     p.set_defaults(run=elementwise)

@@ -134,6 +134,10 @@ class NativeOps:
         # bfloat16 value + bfloat16 remainder (2: a third slower, half the rounding error)
         self.prefill_probability_parts = int(os.environ.get("TORCHLLMS_B200_PREFILL_PARTS", "1"))
         self.use_fused_residual = os.environ.get("TORCHLLMS_B200_NO_FUSED_RESIDUAL", "") not in ("1", "true")
+        # independent branches of a layer on two streams (TORCHLLMS_B200_NO_SIDE_STREAM=1 keeps them on one, for comparisons)
+        self.use_side_stream = os.environ.get("TORCHLLMS_B200_NO_SIDE_STREAM", "") not in ("1", "true")
+        self._side_streams: Dict[int, torch.cuda.Stream] = {}
+        self._beside: Optional[torch.cuda.Stream] = None
         # attention with options (kept first keys, distance bias, gate, values of their own size) in bfloat16 on the
         # tensor cores; TORCHLLMS_B200_NO_MMA_OPTIONS=1 keeps such calls on the CUDA-core kernel, for comparisons
         self.use_mma_options = os.environ.get("TORCHLLMS_B200_NO_MMA_OPTIONS", "") not in ("1", "true")
@@ -179,6 +183,32 @@ class NativeOps:
                 entry[0] += 1
                 entry[1] += ms - inner.pop(depth + 1, 0.0)
                 inner[depth] = inner.get(depth, 0.0) + ms
+
+    # ------------------------------------------------------------- two chains of kernels at a time
+    @contextlib.contextmanager
+    def aside(self, max_q_len: int):
+        """What is issued inside the block runs on a stream of its own, after everything issued before it and beside what
+        is issued next, until :meth:`rejoin`.  Only in steps of short portions (``max_q_len``), whose kernels leave most
+        of the GPU idle: two long kernels side by side take each other's issue slots and are slower than one after the
+        other.  (Works in a graph's capture too; while a profile is being taken everything stays on one stream, so that
+        calls are timed alone.)"""
+        if self._profile is not None or not self.use_side_stream or max_q_len > 16:
+            yield
+            return
+        main = torch.cuda.current_stream()
+        side = self._side_streams.get(main.device_index)
+        if side is None:
+            side = self._side_streams[main.device_index] = torch.cuda.Stream()
+        side.wait_stream(main)
+        self._beside = side
+        with torch.cuda.stream(side):
+            yield
+
+    def rejoin(self) -> None:
+        """What is issued from here on waits for the work issued :meth:`aside`."""
+        if self._beside is not None:
+            torch.cuda.current_stream().wait_stream(self._beside)
+            self._beside = None
 
     # ------------------------------------------------------------- checks
     def check_attention_sizes(self, n_heads: int, n_kv_heads: int, head_dim: int, dtype: torch.dtype,
@@ -1015,7 +1045,7 @@ class NativeOps:
             _ptr(slot_mapping), _ptr(q), _ptr(extra), _ptr(k_pages), _ptr(v_pages), _DT[out_dtype], T, n_seqs, max_q_len, n_q_heads,
             n_k_heads, head_dim, v_head_dim, rot_dims, n_extra, ctypes.c_float(extra_scale), page_size, table.shape[0], _stream())
         _check(rc, "conv_rope_store")
-        self.launches += 2 if (max_q_len > 16 and w_conv.shape[0] > 1) else 1
+        self.launches += 2 if (max_q_len > 4 and w_conv.shape[0] > 1) else 1
         return q, extra
 
     @_timed
@@ -1045,7 +1075,7 @@ class NativeOps:
             _ptr(small), _ptr(low), _DT[out_dtype], T, n_seqs, max_q_len, n_qk_heads, head_dim, n_v, n_small, n_low, low_pad,
             ctypes.c_float(q_scale), ctypes.c_float(unit_eps), _stream())
         _check(rc, "delta_prep")
-        self.launches += 2 if (max_q_len > 16 and w_conv.shape[0] > 1) else 1
+        self.launches += 2 if (max_q_len > 4 and w_conv.shape[0] > 1) else 1
         return q, k, v, small, low
 
     BLOCKS_MIN_Q = 9      # steps with portions at least this long run a matrix recurrence four tokens at a time

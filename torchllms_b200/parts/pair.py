@@ -95,7 +95,7 @@ class SideBySideSum(_Pair):
     """``left(x) + right(x)``, each member scaled by what its own ``out_scale`` says, for members that run in halves
     (``Mixer.runs_in_halves``): their input products are one product over the stacked weights, each writes its result
     into its columns of one row, and ``[left's rows | right's rows]`` times ``[wo_l | wo_r]`` is the sum: one product, left to
-    the norm that follows."""
+    the norm that follows.  Between the two products the members of a step of short portions run on two streams."""
 
     def __init__(self, env: BuildEnv, *, dim: int, left: PartSpec, right: PartSpec, left_prefix: str = "left",
                  right_prefix: str = "right"):
@@ -123,8 +123,11 @@ class SideBySideSum(_Pair):
     def forward(self, x: torch.Tensor, ctx, cache) -> PendingProduct:
         proj = self.env.ops.linear(x, self.w_in, partials_ok=True)
         rows = torch.empty((x.shape[0], sum(self.inner)), dtype=self.env.dtype, device=x.device)
-        at = to = 0
-        for (prefix, m), width, inner in zip(self.members, self.widths, self.inner):
-            m.mix(proj[..., at:at + width], ctx, self._cache_of(prefix, m, cache), rows[:, to:to + inner])
-            at, to = at + width, to + inner
+        at, to = self.widths[0], self.inner[0]
+        (lp, left), (rp, right) = self.members
+        # the members know nothing of each other: their kernels may run side by side
+        with self.env.ops.aside(ctx.max_q_len):
+            right.mix(proj[..., at:], ctx, self._cache_of(rp, right, cache), rows[:, to:])
+        left.mix(proj[..., :at], ctx, self._cache_of(lp, left, cache), rows[:, :to])
+        self.env.ops.rejoin()
         return PendingProduct(rows, self.wo)
