@@ -43,6 +43,9 @@ template <int VEC> __device__ __forceinline__ Cols<VEC> load_cols(const float* p
     if constexpr (VEC == 4) {
         const float4 x = *reinterpret_cast<const float4*>(p);
         c.v[0] = x.x; c.v[1] = x.y; c.v[2] = x.z; c.v[3] = x.w;
+    } else if constexpr (VEC == 2) {
+        const float2 x = *reinterpret_cast<const float2*>(p);
+        c.v[0] = x.x; c.v[1] = x.y;
     } else c.v[0] = *p;
     return c;
 }
@@ -53,11 +56,15 @@ template <int VEC> __device__ __forceinline__ Cols<VEC> load_cols(const __nv_bfl
         const float2 a = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&raw.x));
         const float2 b = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&raw.y));
         c.v[0] = a.x; c.v[1] = a.y; c.v[2] = b.x; c.v[3] = b.y;
+    } else if constexpr (VEC == 2) {
+        const float2 a = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(p));
+        c.v[0] = a.x; c.v[1] = a.y;
     } else c.v[0] = __bfloat162float(*p);
     return c;
 }
 template <int VEC> __device__ __forceinline__ void store_cols(float* p, const Cols<VEC>& c) {
     if constexpr (VEC == 4) *reinterpret_cast<float4*>(p) = make_float4(c.v[0], c.v[1], c.v[2], c.v[3]);
+    else if constexpr (VEC == 2) *reinterpret_cast<float2*>(p) = make_float2(c.v[0], c.v[1]);
     else *p = c.v[0];
 }
 template <int VEC> __device__ __forceinline__ void store_cols(__nv_bfloat16* p, const Cols<VEC>& c) {
@@ -67,7 +74,8 @@ template <int VEC> __device__ __forceinline__ void store_cols(__nv_bfloat16* p, 
         raw.x = *reinterpret_cast<const unsigned*>(&a);
         raw.y = *reinterpret_cast<const unsigned*>(&b);
         *reinterpret_cast<uint2*>(p) = raw;
-    } else *p = __float2bfloat16_rn(c.v[0]);
+    } else if constexpr (VEC == 2) *reinterpret_cast<__nv_bfloat162*>(p) = __floats2bfloat162_rn(c.v[0], c.v[1]);
+    else *p = __float2bfloat16_rn(c.v[0]);
 }
 template <int VEC> __device__ __forceinline__ Cols<VEC> zero_cols() {
     Cols<VEC> c;
@@ -76,15 +84,18 @@ template <int VEC> __device__ __forceinline__ Cols<VEC> zero_cols() {
     return c;
 }
 
-// VEC columns of row t, planes added up
+// VEC columns of row t, planes added up (bfloat16 rows have one plane: without a loop behind every load, a thread's loads
+// go out together)
 template <int VEC, typename TI>
 __device__ __forceinline__ Cols<VEC> row_cols(const ConvInput& p, long long t, int c) {
     const TI* src = reinterpret_cast<const TI*>(p.proj) + t * p.ld + c;
     Cols<VEC> x = load_cols<VEC>(src);
-    for (int s = 1; s < p.splits; ++s) {
-        const Cols<VEC> y = load_cols<VEC>(src + s * p.plane);
+    if constexpr (sizeof(TI) == sizeof(float)) {
+        for (int s = 1; s < p.splits; ++s) {
+            const Cols<VEC> y = load_cols<VEC>(src + s * p.plane);
 #pragma unroll
-        for (int e = 0; e < VEC; ++e) x.v[e] += y.v[e];
+            for (int e = 0; e < VEC; ++e) x.v[e] += y.v[e];
+        }
     }
     return x;
 }
@@ -95,6 +106,18 @@ __device__ __forceinline__ Cols<VEC> conv_cols(const ConvInput& p, int start, in
     if (rel >= 0) return row_cols<VEC, TI>(p, (long long)start + rel, c);
     if (fresh || st == nullptr) return zero_cols<VEC>();
     return load_cols<VEC>(st + (size_t)(p.taps - 1 + rel) * p.C + c);
+}
+
+// VEC columns of the TOK rows from row t on, of which n are there (zeros behind them)
+template <int VEC, typename TI>
+__device__ __forceinline__ void rows_cols(const ConvInput& p, long long t, int n, int c, Cols<VEC> (&x)[TOK]) {
+    if (n == TOK) {
+#pragma unroll
+        for (int i = 0; i < TOK; ++i) x[i] = row_cols<VEC, TI>(p, t + i, c);
+    } else {
+#pragma unroll
+        for (int i = 0; i < TOK; ++i) x[i] = i < n ? row_cols<VEC, TI>(p, t + i, c) : zero_cols<VEC>();
+    }
 }
 
 // The last TM inputs of VEC channels and their taps (taps < TM: the oldest places weigh nothing and hold zeros).
@@ -109,6 +132,11 @@ struct Window {
         for (int j = 0; j < TM; ++j) w[j] = j >= off ? load_cols<VEC>(p.w + (size_t)(j - off) * p.C + c) : zero_cols<VEC>();
         // before the first push: the inputs r0 - (TM - 1) .. r0 - 1 lie in places 1 .. TM - 1
         in[0] = zero_cols<VEC>();
+        if (r0 >= TM - 1) {                             // (all of them inside the portion: loads without conditions)
+#pragma unroll
+            for (int j = 1; j < TM; ++j) in[j] = row_cols<VEC, TI>(p, (long long)start + r0 - TM + j, c);
+            return;
+        }
 #pragma unroll
         for (int j = 1; j < TM; ++j)
             in[j] = j > off ? conv_cols<VEC, TI>(p, start, r0 - TM + j, c, st, fresh) : zero_cols<VEC>();
@@ -167,9 +195,7 @@ __global__ void __launch_bounds__(NT) conv_rope_store_kernel(const StoreParams p
         const int c = (item - n_qk - n_v) * VEC;
         T* out = reinterpret_cast<T*>(p.extra_out);
         Cols<VEC> x[TOK];
-#pragma unroll
-        for (int i = 0; i < TOK; ++i)
-            x[i] = i < n ? row_cols<VEC, TI>(p.x, (long long)start + r0 + i, p.x.C + c) : zero_cols<VEC>();
+        rows_cols<VEC, TI>(p.x, (long long)start + r0, n, p.x.C + c, x);
 #pragma unroll
         for (int i = 0; i < TOK; ++i) {
             if (i >= n) break;
@@ -196,50 +222,55 @@ __global__ void __launch_bounds__(NT) conv_rope_store_kernel(const StoreParams p
         c0 = qk * p.hd + c;
         kind = 2;
     }
+    // where every token's angles and its place in the pages are: asked for ahead of the rows
+    int pos[TOK], slots[TOK];
+#pragma unroll
+    for (int i = 0; i < TOK; ++i) {
+        pos[i] = c1 >= 0 && i < n ? p.positions[start + r0 + i] : 0;
+        slots[i] = kind != 0 && i < n ? p.slot_mapping[start + r0 + i] : 0;
+    }
     const bool fresh = p.x.fresh[b] != 0;
     float* st = p.x.state != nullptr ? p.x.state + (size_t)p.x.state_slot[b] * p.x.state_pitch : nullptr;
     Window<VEC, TM> wa, wb;
     wa.template open<TI>(p.x, start, r0, c0, st, fresh);
     if (c1 >= 0) wb.template open<TI>(p.x, start, r0, c1, st, fresh);
-    {
-        Cols<VEC> xa[TOK], xb[TOK];
+    Cols<VEC> xa[TOK], xb[TOK];
+    rows_cols<VEC, TI>(p.x, (long long)start + r0, n, c0, xa);
+    if (c1 >= 0) rows_cols<VEC, TI>(p.x, (long long)start + r0, n, c1, xb);
+    float2 cs[TOK][VEC];
 #pragma unroll
-        for (int i = 0; i < TOK; ++i) {
-            const bool in = i < n;
-            xa[i] = in ? row_cols<VEC, TI>(p.x, (long long)start + r0 + i, c0) : zero_cols<VEC>();
-            xb[i] = in && c1 >= 0 ? row_cols<VEC, TI>(p.x, (long long)start + r0 + i, c1) : zero_cols<VEC>();
-        }
+    for (int i = 0; i < TOK; ++i) {
+        (void)TL_CHECK(pos[i] >= 0 && pos[i] < p.table_rows, TL_DBG_POSITION);
+        const int row = pos[i] < 0 ? 0 : (pos[i] >= p.table_rows ? p.table_rows - 1 : pos[i]);
 #pragma unroll
-        for (int i = 0; i < TOK; ++i) {
-            if (i >= n) break;
-            const int t = start + r0 + i;
-            Cols<VEC> ya = wa.push(xa[i]), yb;
-            if (c1 >= 0) {
-                yb = wb.push(xb[i]);
-                int pos = p.positions[t];
-                (void)TL_CHECK(pos >= 0 && pos < p.table_rows, TL_DBG_POSITION);
-                pos = pos < 0 ? 0 : (pos >= p.table_rows ? p.table_rows - 1 : pos);
-                const float* cs = p.table + (size_t)pos * p.rot + 2 * d0;
+        for (int e = 0; e < VEC; ++e)
+            cs[i][e] = c1 >= 0 ? *reinterpret_cast<const float2*>(p.table + (size_t)row * p.rot + 2 * (d0 + e)) : make_float2(0.f, 0.f);
+    }
 #pragma unroll
-                for (int e = 0; e < VEC; ++e) {
-                    const float2 a = *reinterpret_cast<const float2*>(cs + 2 * e);
-                    const float u = ya.v[e], v = yb.v[e];
-                    ya.v[e] = u * a.x - v * a.y;
-                    yb.v[e] = v * a.x + u * a.y;
-                }
+    for (int i = 0; i < TOK; ++i) {
+        if (i >= n) break;
+        const int t = start + r0 + i;
+        Cols<VEC> ya = wa.push(xa[i]), yb;
+        if (c1 >= 0) {
+            yb = wb.push(xb[i]);
+#pragma unroll
+            for (int e = 0; e < VEC; ++e) {
+                const float u = ya.v[e], v = yb.v[e];
+                ya.v[e] = u * cs[i][e].x - v * cs[i][e].y;
+                yb.v[e] = v * cs[i][e].x + u * cs[i][e].y;
             }
-            T* dst;
-            if (kind == 0) dst = reinterpret_cast<T*>(p.q_out) + ((size_t)t * p.n_q + head) * p.hd + d0;
-            else {
-                const int sm = p.slot_mapping[t];
-                const int page = sm / p.page_size, slot = sm - page * p.page_size;
-                if (!(TL_CHECK(sm >= 0, TL_DBG_SLOT) && tl_check_page(page))) continue;
-                const size_t at = ((size_t)page * p.n_k + head) * p.page_size + slot;
-                dst = kind == 1 ? reinterpret_cast<T*>(p.k_pages) + at * p.hd + d0 : reinterpret_cast<T*>(p.v_pages) + at * p.dv + d0;
-            }
-            store_cols<VEC>(dst, ya);
-            if (c1 >= 0) store_cols<VEC>(dst + half, yb);
         }
+        T* dst;
+        if (kind == 0) dst = reinterpret_cast<T*>(p.q_out) + ((size_t)t * p.n_q + head) * p.hd + d0;
+        else {
+            const int sm = slots[i];
+            const int page = sm / p.page_size, slot = sm - page * p.page_size;
+            if (!(TL_CHECK(sm >= 0, TL_DBG_SLOT) && tl_check_page(page))) continue;
+            const size_t at = ((size_t)page * p.n_k + head) * p.page_size + slot;
+            dst = kind == 1 ? reinterpret_cast<T*>(p.k_pages) + at * p.hd + d0 : reinterpret_cast<T*>(p.v_pages) + at * p.dv + d0;
+        }
+        store_cols<VEC>(dst, ya);
+        if (c1 >= 0) store_cols<VEC>(dst + half, yb);
     }
     if (p.x.n_chunks == 1 && st != nullptr) {                   // nobody else reads or writes these channels' state
         wa.leave(p.x, st, c0);
@@ -298,16 +329,14 @@ __global__ void __launch_bounds__(NT) delta_prep_kernel(const DeltaParams p) {
         for (int e = lane; e < UNIT; e += 32) {
             const int c = base + e;
             if (c >= p.n_small + p.low_pad) break;
-            float x[TOK];
-#pragma unroll
-            for (int i = 0; i < TOK; ++i)
-                x[i] = i < n && c < p.n_small + p.n_low ? row_cols<1, TI>(p.x, (long long)start + r0 + i, p.x.C + c).v[0] : 0.f;
+            Cols<1> x[TOK];
+            rows_cols<1, TI>(p.x, (long long)start + r0, c < p.n_small + p.n_low ? n : 0, p.x.C + c, x);
 #pragma unroll
             for (int i = 0; i < TOK; ++i) {
                 if (i >= n) break;
                 const size_t t = (size_t)start + r0 + i;
-                if (c < p.n_small) reinterpret_cast<T*>(p.small)[t * p.n_small + c] = from_float<T>(x[i]);
-                else reinterpret_cast<T*>(p.low)[t * p.low_pad + (c - p.n_small)] = from_float<T>(x[i]);
+                if (c < p.n_small) reinterpret_cast<T*>(p.small)[t * p.n_small + c] = from_float<T>(x[i].v[0]);
+                else reinterpret_cast<T*>(p.low)[t * p.low_pad + (c - p.n_small)] = from_float<T>(x[i].v[0]);
             }
         }
         return;
@@ -328,50 +357,45 @@ __global__ void __launch_bounds__(NT) delta_prep_kernel(const DeltaParams p) {
     const bool is_q = unit < p.heads;
     const float scale = is_q ? p.q_scale : 1.f;
     float* qk_out = is_q ? p.q + (size_t)unit * p.hd : p.k + (size_t)(unit - p.heads) * p.hd;
-    {
-        Cols<VEC> y[TOK][IT];
+    Cols<VEC> y[IT][TOK];
 #pragma unroll
-        for (int i = 0; i < TOK; ++i)
+    for (int it = 0; it < IT; ++it)
+        rows_cols<VEC, TI>(p.x, (long long)start + r0, mine[it] ? n : 0, c_lo + (it * 32 + lane) * VEC, y[it]);
+    float ssq[TOK];
 #pragma unroll
-            for (int it = 0; it < IT; ++it)
-                y[i][it] = i < n && mine[it] ? row_cols<VEC, TI>(p.x, (long long)start + r0 + i, c_lo + (it * 32 + lane) * VEC)
-                                                  : zero_cols<VEC>();
-        float ssq[TOK];
-#pragma unroll
-        for (int i = 0; i < TOK; ++i) {
-            ssq[i] = 0.f;
-            if (i < n) {
-#pragma unroll
-                for (int it = 0; it < IT; ++it) {
-                    if (!mine[it]) continue;
-                    y[i][it] = win[it].push(y[i][it]);
-#pragma unroll
-                    for (int e = 0; e < VEC; ++e) {
-                        const float a = silu_f(y[i][it].v[e]);
-                        y[i][it].v[e] = a;
-                        ssq[i] = fmaf(a, a, ssq[i]);
-                    }
-                }
-            }
-        }
-        if (!is_v) {
-#pragma unroll
-            for (int i = 0; i < TOK; ++i) ssq[i] = rsqrtf(warp_sum(ssq[i]) + p.unit_eps) * scale;
-        }
-#pragma unroll
-        for (int i = 0; i < TOK; ++i) {
-            if (i >= n) break;
-            const size_t t = (size_t)start + r0 + i;
+    for (int i = 0; i < TOK; ++i) {
+        ssq[i] = 0.f;
+        if (i < n) {
 #pragma unroll
             for (int it = 0; it < IT; ++it) {
                 if (!mine[it]) continue;
-                const int d = (it * 32 + lane) * VEC;
-                if (is_v) store_cols<VEC>(reinterpret_cast<T*>(p.v) + t * p.n_v + (c_lo - 2 * p.n_qk) + d, y[i][it]);
-                else {
+                y[it][i] = win[it].push(y[it][i]);
 #pragma unroll
-                    for (int e = 0; e < VEC; ++e) y[i][it].v[e] *= ssq[i];
-                    store_cols<VEC>(qk_out + t * p.n_qk + d, y[i][it]);
+                for (int e = 0; e < VEC; ++e) {
+                    const float a = silu_f(y[it][i].v[e]);
+                    y[it][i].v[e] = a;
+                    ssq[i] = fmaf(a, a, ssq[i]);
                 }
+            }
+        }
+    }
+    if (!is_v) {
+#pragma unroll
+        for (int i = 0; i < TOK; ++i) ssq[i] = rsqrtf(warp_sum(ssq[i]) + p.unit_eps) * scale;
+    }
+#pragma unroll
+    for (int i = 0; i < TOK; ++i) {
+        if (i >= n) break;
+        const size_t t = (size_t)start + r0 + i;
+#pragma unroll
+        for (int it = 0; it < IT; ++it) {
+            if (!mine[it]) continue;
+            const int d = (it * 32 + lane) * VEC;
+            if (is_v) store_cols<VEC>(reinterpret_cast<T*>(p.v) + t * p.n_v + (c_lo - 2 * p.n_qk) + d, y[it][i]);
+            else {
+#pragma unroll
+                for (int e = 0; e < VEC; ++e) y[it][i].v[e] *= ssq[i];
+                store_cols<VEC>(qk_out + t * p.n_qk + d, y[it][i]);
             }
         }
     }
@@ -400,15 +424,16 @@ int launch_state(const ConvInput& x, int in_dtype, int n_seqs, cudaStream_t s) {
                               : (int)tl_launch(conv_state_kernel<__nv_bfloat16>, grid, dim3(NT), 0, s, x);
 }
 
-bool good_input(const ConvInput& x, int n_seqs, int max_q_len) {
-    return x.taps >= 1 && x.taps <= MAX_TAPS && x.splits >= 1 && n_seqs <= 65535 && max_q_len > 0 && x.n_chunks <= 65535 &&
+bool good_input(const ConvInput& x, int in_dtype, int n_seqs, int max_q_len) {
+    return (x.splits == 1 || in_dtype == TL_F32) && x.taps >= 1 && x.taps <= MAX_TAPS && x.splits >= 1 && n_seqs <= 65535 && max_q_len > 0 && x.n_chunks <= 65535 &&
            (x.taps == 1 || x.state != nullptr);
 }
 
-// whether rows and state may be read four columns at a time (column offsets are the caller's to check)
-bool vector_input(const ConvInput& x, int in_dtype) {
-    const uintptr_t a = reinterpret_cast<uintptr_t>(x.proj);
-    return x.C % 4 == 0 && aligned16(x.w) && x.ld % 4 == 0 && x.plane % 4 == 0 && a % (in_dtype == TL_F32 ? 16 : 8) == 0 && x.state_pitch % 4 == 0 && aligned16(x.state);
+// whether rows, taps and state may be read so many columns at a time (column offsets are the caller's to check)
+bool vector_input(const ConvInput& x, int in_dtype, int vec) {
+    const uintptr_t a = reinterpret_cast<uintptr_t>(x.proj), w = reinterpret_cast<uintptr_t>(x.w), st = reinterpret_cast<uintptr_t>(x.state);
+    return x.C % vec == 0 && x.ld % vec == 0 && x.plane % vec == 0 && a % ((in_dtype == TL_F32 ? 4 : 2) * vec) == 0 && w % (4 * vec) == 0 &&
+           x.state_pitch % vec == 0 && st % (4 * vec) == 0;
 }
 
 }  // namespace
@@ -430,13 +455,14 @@ extern "C" int tl_conv_rope_store(const void* proj, int in_dtype, int splits, lo
     p.x.proj = proj; p.x.splits = splits; p.x.plane = plane; p.x.ld = ld; p.x.w = w; p.x.state = taps > 1 ? state : nullptr;
     p.x.state_pitch = taps > 1 ? state_pitch : 0; p.x.q_start = q_start; p.x.state_slot = state_slot; p.x.fresh = fresh;
     p.x.C = (n_q + n_k) * hd + n_k * dv; p.x.taps = taps; p.x.n_chunks = (max_q_len + TOK - 1) / TOK;
-    if (!good_input(p.x, n_seqs, max_q_len)) return TL_BAD_SIZE;
+    if (!good_input(p.x, in_dtype, n_seqs, max_q_len)) return TL_BAD_SIZE;
     p.positions = positions; p.table = table; p.slot_mapping = slot_mapping; p.q_out = q_out; p.extra_out = extra_out;
     p.k_pages = k_pages; p.v_pages = v_pages; p.n_q = n_q; p.n_k = n_k; p.hd = hd; p.dv = dv; p.rot = rot; p.n_extra = n_extra;
     p.page_size = page_size; p.table_rows = table_rows; p.extra_scale = extra_scale;
-    const bool vec = vector_input(p.x, in_dtype) && (rot / 2) % 4 == 0 && hd % 4 == 0 && dv % 4 == 0 && n_extra % 4 == 0 &&
+    // (two columns a thread: with more, a rotated pair's windows cost the registers of a third warp)
+    const bool vec = vector_input(p.x, in_dtype, 2) && (rot / 2) % 2 == 0 && hd % 2 == 0 && dv % 2 == 0 && n_extra % 2 == 0 &&
                      aligned16(q_out) && aligned16(extra_out) && aligned16(k_pages) && aligned16(v_pages) && aligned16(table);
-    const int V = vec ? 4 : 1;
+    const int V = vec ? 2 : 1;
     const long long items = (long long)(n_q + n_k) * (rot / 2 / V + (hd - rot) / V) + (long long)n_k * dv / V + n_extra / V;
     if (items > (1ll << 30)) return TL_BAD_SIZE;
     p.n_items = (int)items;
@@ -445,7 +471,7 @@ extern "C" int tl_conv_rope_store(const void* proj, int in_dtype, int splits, lo
     cudaError_t e;
 #define TL_STORE(TI, T, VEC, TM) tl_launch(conv_rope_store_kernel<TI, T, VEC, TM>, grid, block, 0, s, p)
 #define TL_STORE_PICK(TI, T)                                                                                   \
-    e = vec ? (taps <= 4 ? TL_STORE(TI, T, 4, 4) : TL_STORE(TI, T, 4, MAX_TAPS))                               \
+    e = vec ? (taps <= 4 ? TL_STORE(TI, T, 2, 4) : TL_STORE(TI, T, 2, MAX_TAPS))                               \
             : (taps <= 4 ? TL_STORE(TI, T, 1, 4) : TL_STORE(TI, T, 1, MAX_TAPS))
     if (in_dtype == TL_F32 && dtype == TL_F32) TL_STORE_PICK(float, float);
     else if (in_dtype == TL_F32 && dtype == TL_BF16) TL_STORE_PICK(float, __nv_bfloat16);
@@ -470,12 +496,12 @@ extern "C" int tl_delta_prep(const void* proj, int in_dtype, int splits, long lo
     p.x.proj = proj; p.x.splits = splits; p.x.plane = plane; p.x.ld = ld; p.x.w = w; p.x.state = taps > 1 ? state : nullptr;
     p.x.state_pitch = taps > 1 ? state_pitch : 0; p.x.q_start = q_start; p.x.state_slot = state_slot; p.x.fresh = fresh;
     p.x.C = 2 * heads * hd + n_v; p.x.taps = taps; p.x.n_chunks = (max_q_len + TOK - 1) / TOK;
-    if (!good_input(p.x, n_seqs, max_q_len)) return TL_BAD_SIZE;
+    if (!good_input(p.x, in_dtype, n_seqs, max_q_len)) return TL_BAD_SIZE;
     p.q = q; p.k = k; p.v = v; p.small = small; p.low = low; p.heads = heads; p.hd = hd; p.n_qk = heads * hd; p.n_v = n_v;
     p.n_small = n_small; p.n_low = n_low; p.low_pad = n_low > 0 ? low_pad : 0; p.q_scale = q_scale; p.unit_eps = unit_eps;
     p.v_units = (n_v + UNIT - 1) / UNIT;
     p.n_units = 2 * heads + p.v_units + (n_small + p.low_pad + UNIT - 1) / UNIT;
-    const bool vec = vector_input(p.x, in_dtype) && hd % 4 == 0 && n_v % 4 == 0 && aligned16(q) && aligned16(k) && aligned16(v);
+    const bool vec = vector_input(p.x, in_dtype, 4) && hd % 4 == 0 && n_v % 4 == 0 && aligned16(q) && aligned16(k) && aligned16(v);
     const dim3 grid((p.n_units + NT / 32 - 1) / (NT / 32), p.x.n_chunks, n_seqs), block(NT);
     cudaStream_t s = (cudaStream_t)stream;
     cudaError_t e;
