@@ -544,7 +544,7 @@ def test_results_that_are_columns_of_wider_rows(backend):
         torch.testing.assert_close(rows[:, 5:5 + H * d].cpu().double(), want, **tol)
         assert (rows[:, :5] == 3.0).all() and (rows[:, 5 + H * d:] == 3.0).all()
     page = 8
-    for H, G, d, dv, width in ((4, 2, 16, 24, 4 * 24 + 10), (2, 1, 9, 7, 2 * 7 + 3), (8, 2, 48, 96, 8 * 96 + 64)):
+    for H, G, d, dv, width in ((4, 2, 16, 24, 4 * 24 + 10), (2, 1, 9, 7, 2 * 7 + 3), (6, 2, 40, 80, 6 * 80 + 64)):
         for lens, total in (([1, 1], [700, 90]), ([40, 3], [60, 200])):
             T = sum(lens)
             n_pages = sum(-(-n // page) for n in total)

@@ -459,8 +459,9 @@ extern "C" int tl_conv_rope_store(const void* proj, int in_dtype, int splits, lo
     p.positions = positions; p.table = table; p.slot_mapping = slot_mapping; p.q_out = q_out; p.extra_out = extra_out;
     p.k_pages = k_pages; p.v_pages = v_pages; p.n_q = n_q; p.n_k = n_k; p.hd = hd; p.dv = dv; p.rot = rot; p.n_extra = n_extra;
     p.page_size = page_size; p.table_rows = table_rows; p.extra_scale = extra_scale;
-    // (two columns a thread: with more, a rotated pair's windows cost the registers of a third warp)
-    const bool vec = vector_input(p.x, in_dtype, 2) && (rot / 2) % 2 == 0 && hd % 2 == 0 && dv % 2 == 0 && n_extra % 2 == 0 &&
+    // (two columns a thread: with more, a rotated pair's windows cost the registers of a third warp; more than four taps
+    // go one column at a time)
+    const bool vec = taps <= 4 && vector_input(p.x, in_dtype, 2) && (rot / 2) % 2 == 0 && hd % 2 == 0 && dv % 2 == 0 && n_extra % 2 == 0 &&
                      aligned16(q_out) && aligned16(extra_out) && aligned16(k_pages) && aligned16(v_pages) && aligned16(table);
     const int V = vec ? 2 : 1;
     const long long items = (long long)(n_q + n_k) * (rot / 2 / V + (hd - rot) / V) + (long long)n_k * dv / V + n_extra / V;
@@ -471,7 +472,7 @@ extern "C" int tl_conv_rope_store(const void* proj, int in_dtype, int splits, lo
     cudaError_t e;
 #define TL_STORE(TI, T, VEC, TM) tl_launch(conv_rope_store_kernel<TI, T, VEC, TM>, grid, block, 0, s, p)
 #define TL_STORE_PICK(TI, T)                                                                                   \
-    e = vec ? (taps <= 4 ? TL_STORE(TI, T, 2, 4) : TL_STORE(TI, T, 2, MAX_TAPS))                               \
+    e = vec ? TL_STORE(TI, T, 2, 4)                                                                            \
             : (taps <= 4 ? TL_STORE(TI, T, 1, 4) : TL_STORE(TI, T, 1, MAX_TAPS))
     if (in_dtype == TL_F32 && dtype == TL_F32) TL_STORE_PICK(float, float);
     else if (in_dtype == TL_F32 && dtype == TL_BF16) TL_STORE_PICK(float, __nv_bfloat16);
@@ -501,19 +502,19 @@ extern "C" int tl_delta_prep(const void* proj, int in_dtype, int splits, long lo
     p.n_small = n_small; p.n_low = n_low; p.low_pad = n_low > 0 ? low_pad : 0; p.q_scale = q_scale; p.unit_eps = unit_eps;
     p.v_units = (n_v + UNIT - 1) / UNIT;
     p.n_units = 2 * heads + p.v_units + (n_small + p.low_pad + UNIT - 1) / UNIT;
-    const bool vec = vector_input(p.x, in_dtype, 4) && hd % 4 == 0 && n_v % 4 == 0 && aligned16(q) && aligned16(k) && aligned16(v);
+    const bool vec = taps <= 4 && vector_input(p.x, in_dtype, 4) && hd % 4 == 0 && n_v % 4 == 0 && aligned16(q) && aligned16(k) && aligned16(v);
     const dim3 grid((p.n_units + NT / 32 - 1) / (NT / 32), p.x.n_chunks, n_seqs), block(NT);
     cudaStream_t s = (cudaStream_t)stream;
     cudaError_t e;
 #define TL_PREP(TI, T, VEC, IT, TM) tl_launch(delta_prep_kernel<TI, T, VEC, IT, TM>, grid, block, 0, s, p)
-#define TL_PREP_TAPS(TI, T, VEC, IT) (taps <= 4 ? TL_PREP(TI, T, VEC, IT, 4) : TL_PREP(TI, T, VEC, IT, MAX_TAPS))
-#define TL_PREP_PICK(TI, T) e = vec ? (hd <= 128 ? TL_PREP_TAPS(TI, T, 4, 1) : TL_PREP_TAPS(TI, T, 4, 2)) : TL_PREP_TAPS(TI, T, 1, 8)
+#define TL_PREP_PICK(TI, T)                                                                                    \
+    e = vec ? (hd <= 128 ? TL_PREP(TI, T, 4, 1, 4) : TL_PREP(TI, T, 4, 2, 4))                                  \
+            : (taps <= 4 ? TL_PREP(TI, T, 1, 8, 4) : TL_PREP(TI, T, 1, 8, MAX_TAPS))
     if (in_dtype == TL_F32 && dtype == TL_F32) TL_PREP_PICK(float, float);
     else if (in_dtype == TL_F32 && dtype == TL_BF16) TL_PREP_PICK(float, __nv_bfloat16);
     else if (in_dtype == TL_BF16 && dtype == TL_BF16) TL_PREP_PICK(__nv_bfloat16, __nv_bfloat16);
     else return TL_BAD_DTYPE;
 #undef TL_PREP_PICK
-#undef TL_PREP_TAPS
 #undef TL_PREP
     if (e != cudaSuccess) return (int)e;
     return p.x.n_chunks > 1 && p.x.state != nullptr ? launch_state(p.x, in_dtype, n_seqs, s) : TL_OK;
